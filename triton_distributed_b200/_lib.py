@@ -20,6 +20,7 @@ import torch
 _PKG = Path(__file__).resolve().parent
 _DEBUG = os.environ.get("B200DIST_DEBUG_LIB", "0") == "1"   # the checking build (python -m ...build --debug)
 LIB_PATH = _PKG / "lib" / ("libb200dist_debug.so" if _DEBUG else "libb200dist.so")
+_serving = False   # see use_serving_library
 
 _lock = threading.Lock()
 _lib: ctypes.CDLL | None = None
@@ -33,6 +34,13 @@ class NativeError(RuntimeError):
         self.code = code
 
 
+def use_serving_library() -> None:
+    """For single-GPU programs, before the first kernel: unless the full library has been built already, build and load the
+    subset that serving one GPU needs (``build.SERVING_SOURCES``)."""
+    global _serving
+    _serving = True
+
+
 def lib_available() -> bool:
     return LIB_PATH.exists()
 
@@ -43,16 +51,18 @@ def load(build_if_missing: bool = True) -> ctypes.CDLL:
     with _lock:
         if _lib is not None:
             return _lib
+        path = LIB_PATH
         if not LIB_PATH.exists():
             if not build_if_missing or os.environ.get("B200DIST_NO_BUILD") == "1":
                 raise RuntimeError(
                     f"native library {LIB_PATH} is missing; run `python -m triton_distributed_b200.build`")
             from . import build as _build
-            _build.build(debug=_DEBUG)
-        lib = ctypes.CDLL(str(LIB_PATH))
+            path = _build.build(debug=_DEBUG, serving=_serving and not _DEBUG)
+        lib = ctypes.CDLL(str(path))
         lib.b200_last_error.restype = ctypes.c_char_p
         for name in ("b200_heap_base", "b200_heap_mc_base", "b200_heap_bytes", "b200_heap_live_bytes"):
-            getattr(lib, name).restype = ctypes.c_uint64
+            if hasattr(lib, name):  # not in the serving subset
+                getattr(lib, name).restype = ctypes.c_uint64
         _lib = lib
         return lib
 

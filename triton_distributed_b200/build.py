@@ -7,7 +7,10 @@ Compilation is incremental (source / header mtimes) and parallel.
 Role in the reference: CMake + setup.py building ``libtriton_distributed.so`` and the Triton
 backend (``CMakeLists.txt:15-26``, ``csrc/lib/CMakeLists.txt:47``, ``python/setup.py``).
 
-Usage: ``python -m triton_distributed_b200.build [--force] [--verbose] [--debug]``
+Usage: ``python -m triton_distributed_b200.build [--force] [--verbose] [--debug | --serving]``
+
+``--serving`` builds only what single-GPU serving needs into ``lib/libb200dist_serving.so``; programs that ask for it
+(``_lib.use_serving_library``) get it when the full library has not been built.
 
 ``--debug`` builds a second library, ``lib/libb200dist_debug.so``, with ``-DB200_DEBUG_CHECKS``: bounds-checked symmetric
 address translation and pseudo-random delays in front of every notify / wait / barrier (see ``b200/primitives.cuh``).
@@ -17,6 +20,7 @@ from __future__ import annotations
 
 import argparse
 import concurrent.futures
+import fcntl
 import os
 import shutil
 import subprocess
@@ -29,6 +33,12 @@ BUILD = PKG.parent / "build" / "b200dist"
 LIB_DIR = PKG / "lib"
 LIB_PATH = LIB_DIR / "libb200dist.so"
 DEBUG_LIB_PATH = LIB_DIR / "libb200dist_debug.so"
+SERVING_LIB_PATH = LIB_DIR / "libb200dist_serving.so"
+
+# sources of the single-GPU serving subset: no heap, no collectives, no expert kernels
+SERVING_SOURCES = ("runtime/host.cc", "kernels/decode_attn.cu", "kernels/elementwise.cu", "kernels/gemm_f32.cu",
+                   "kernels/gemm_skinny_sm100.cu", "kernels/gemm_sm100.cu", "kernels/latent_attn.cu",
+                   "kernels/prefill_attn_sm100.cu", "kernels/residual.cu", "kernels/sampling.cu")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -49,7 +59,9 @@ def _nvcc() -> str:
     return exe
 
 
-def sources() -> list[Path]:
+def sources(serving: bool = False) -> list[Path]:
+    if serving:
+        return [CSRC / name for name in SERVING_SOURCES]
     out = sorted(list(CSRC.glob("runtime/*.cc")) + list(CSRC.glob("runtime/*.cu")) + list(CSRC.glob("kernels/*.cu")))
     return out
 
@@ -69,14 +81,21 @@ def _compile(src: Path, obj: Path, verbose: bool, ptxas_v: bool, debug: bool = F
 
 
 def build(force: bool = False, verbose: bool = False, ptxas_v: bool = False, jobs: int | None = None,
-          debug: bool = False) -> Path:
-    """Compile what is out of date and link the shared library (the checking build with ``debug``). Returns its path."""
+          debug: bool = False, serving: bool = False) -> Path:
+    """Compile what is out of date and link the shared library (the checking build with ``debug``, the single-GPU subset with
+    ``serving``). Returns its path. Processes that build at the same time take turns."""
     BUILD.mkdir(parents=True, exist_ok=True)
     LIB_DIR.mkdir(parents=True, exist_ok=True)
+    with open(BUILD / ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return _build_locked(force, verbose, ptxas_v, jobs, debug, serving)
+
+
+def _build_locked(force: bool, verbose: bool, ptxas_v: bool, jobs: int | None, debug: bool, serving: bool) -> Path:
     hdr_time = max(_headers_mtime(), Path(__file__).stat().st_mtime)
-    lib_path = DEBUG_LIB_PATH if debug else LIB_PATH
+    lib_path = DEBUG_LIB_PATH if debug else SERVING_LIB_PATH if serving else LIB_PATH
     todo, objs = [], []
-    for src in sources():
+    for src in sources(serving):
         obj = BUILD / (src.parent.name + "_" + src.stem + (".dbg.o" if debug else ".o"))
         objs.append(obj)
         if force or not obj.exists() or obj.stat().st_mtime < max(src.stat().st_mtime, hdr_time):
@@ -88,12 +107,14 @@ def build(force: bool = False, verbose: bool = False, ptxas_v: bool = False, job
                 src, log = f.result()
                 if verbose or ptxas_v:
                     print(f"[build] {src.name}\n{log}", file=sys.stderr)
-    if todo or not lib_path.exists():
+    if todo or not lib_path.exists() or lib_path.stat().st_mtime < max(o.stat().st_mtime for o in objs):
+        part = lib_path.with_suffix(".part")  # renamed when complete: a reader never sees half a library
         cmd = [_nvcc(), "-shared", "-cudart", "static", "-gencode", "arch=compute_100a,code=sm_100a",
-               "-o", str(lib_path), *map(str, objs), "-lpthread", "-ldl", "-lrt"]
+               "-o", str(part), *map(str, objs), "-lpthread", "-ldl", "-lrt"]
         proc = subprocess.run(cmd, capture_output=True, text=True)
         if proc.returncode != 0:
             raise RuntimeError(f"link failed:\n{proc.stdout}\n{proc.stderr}")
+        os.replace(part, lib_path)
     return lib_path
 
 
@@ -121,8 +142,9 @@ def main() -> None:
     ap.add_argument("--verbose", action="store_true")
     ap.add_argument("--ptxas-v", action="store_true", help="print registers / spills / shared memory per kernel")
     ap.add_argument("--debug", action="store_true", help="build lib/libb200dist_debug.so with B200_DEBUG_CHECKS")
+    ap.add_argument("--serving", action="store_true", help="build only lib/libb200dist_serving.so (single-GPU serving)")
     args = ap.parse_args()
-    print(build(force=args.force, verbose=args.verbose, ptxas_v=args.ptxas_v, debug=args.debug))
+    print(build(force=args.force, verbose=args.verbose, ptxas_v=args.ptxas_v, debug=args.debug, serving=args.serving))
 
 
 if __name__ == "__main__":

@@ -1,17 +1,21 @@
-// Causal (or full) variable-length prefill attention for sm_100a, head dim 128, GQA, bf16 / f16.
+// Causal (or full) variable-length prefill attention for sm_100a, GQA, bf16 / f16, query / key sizes up to 256, any value
+// size, with an optional sink logit per head (one more term of the softmax denominator, without a value).
 //
 //   out[q, h, :] = softmax(scale * Q[q, h, :] . K[keys of q's sequence, kvh(h), :]^T) V[...]     (bottom-right causal mask)
 //
-// One CTA owns 128 query rows of one head and walks the keys in steps of 128:
-//   warp 0     TMA producer: the Q tile once, then K and V^T tiles through two-stage rings (128-byte swizzle)
+// One CTA owns 128 query rows of one head (and up to 128 columns of its values: wider values take more CTAs, each of which
+// computes the scores again) and walks the keys in steps of 128. The kernel is compiled for 1 to 4 column blocks of 64 in a
+// query / key row; columns beyond the row are zero-filled by TMA. Up to two blocks the K and V^T rings have two stages,
+// with three V^T has one and with four both have one, which is what shared memory holds.
+//   warp 0     TMA producer: the Q tile once, then K and V^T tiles through the rings (128-byte swizzle)
 //   warp 1     one elected thread issues tcgen05.mma: S = Q K^T into one of two 128-column TMEM buffers (so the
 //              scores of step j + 1 are computed while step j is in the softmax), then O_step = P V into a third
 //   warps 4-11 softmax, two threads per query row (each owns 64 of the 128 score / output columns; the row maximum is
 //              exchanged through shared memory): read S twice from TMEM (max, then exp2), write P as 16-bit into a
 //              swizzled shared-memory tile that is the A operand of the second MMA, and keep the running output row
 //              in 2 x 64 fp32 registers: O = O * exp2(m_old - m_new) + O_step, so tensor memory never has to be rescaled
-// V is the B operand of the second MMA and has to be K-major ([d, keys]); a small kernel transposes it once per call
-// into a zero-padded [batch x kv head, 128, padded keys] buffer, O(S d) work against the O(S^2 d) of the attention.
+// V is the B operand of the second MMA and has to be K-major ([d, keys]): callers that compute V with a GEMM produce it in
+// that layout (b200_prefill_attention_vt); for a row-major V a small kernel transposes it once per call into a zero-padded [batch x kv head, 128, padded keys] buffer, O(S d) work against the O(S^2 d) of the attention.
 // Every barrier wait is bounded; on expiry the CTA unwinds through an abort flag and reports a status.
 //
 // Role in the reference: flash_attn_with_kvcache in layers/nvidia/tp_attn.py:194-195 (prefill) and the Triton
@@ -24,20 +28,28 @@
 
 namespace b200 {
 
-constexpr int kPD = 128;                    // head dim
+constexpr int kPD = 128;                    // head dim of the row-major-V entry point; value columns per CTA
 constexpr int kPM = 128, kPN = 128;         // query rows per CTA, keys per step
 constexpr int kPAtom = 128 * 64 * 2;        // one 128-row x 64-column 16-bit swizzle atom: 16 KB
 constexpr int kPTile = 2 * kPAtom;          // a 128 x 128 tile: 32 KB
-constexpr int kPSmem = kPTile /*Q*/ + 2 * kPTile /*K*/ + 2 * kPTile /*V^T*/ + kPTile /*P*/ + 1024 + 256 + 3072 /*max / sum exchange*/;
+constexpr int prefill_k_stages(int dk_atoms) { return dk_atoms <= 3 ? 2 : 1; }
+constexpr int prefill_v_stages(int dk_atoms) { return dk_atoms <= 2 ? 2 : 1; }
+constexpr int prefill_smem(int dk_atoms) {
+  return dk_atoms * kPAtom /*Q*/ + prefill_k_stages(dk_atoms) * dk_atoms * kPAtom /*K*/ + prefill_v_stages(dk_atoms) * kPTile /*V^T*/ +
+         kPTile /*P*/ + 1024 + 256 + 3072 /*max / sum exchange*/;
+}
 constexpr int kPThreads = 384;
 
 struct PrefillParams {
   int Hq, Hkv, causal, bf16;
+  int dk, dv;           // query / key and value sizes of a head
+  int v_chunks;         // ceil(dv / 128): CTAs per (query block, head)
+  const float* sink;    // nullable [Hq]
   const int* cu_q;      // [B + 1] first packed query row of every sequence
   const int* cu_k;      // [B + 1] first key row of every sequence (only [0, B) is read when k_lens is given)
   const int* k_lens;    // nullable [B]: keys of every sequence; null = cu_k[b + 1] - cu_k[b] (packed sequences)
   float scale_log2e;    // softmax scale * log2(e)
-  void* out;            // [total_q, Hq, 128]
+  void* out;            // [total_q, Hq, dv]
   uint32_t* status;     // nullable: set non-zero when a pipeline wait expired
 };
 
@@ -71,10 +83,14 @@ __global__ void __launch_bounds__(256) transpose_v_kernel(const uint16_t* __rest
   }
 }
 
+template <int kDkAtoms>
 __global__ void __launch_bounds__(kPThreads, 1)
 prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                     const __grid_constant__ CUtensorMap tmVt, const PrefillParams p) {
-  const int m_blk = blockIdx.x, h = blockIdx.y, b = blockIdx.z;
+  constexpr int kKSt = prefill_k_stages(kDkAtoms), kVSt = prefill_v_stages(kDkAtoms);
+  constexpr int kQkTile = kDkAtoms * kPAtom;
+  const int m_blk = blockIdx.x, h = blockIdx.y / p.v_chunks, b = blockIdx.z;
+  const int v_col0 = (blockIdx.y - h * p.v_chunks) * kPD;  // first value column of this CTA
   const int q_start = p.cu_q[b], q_len = p.cu_q[b + 1] - q_start;
   const int k_start = p.cu_k[b], k_len = p.k_lens ? p.k_lens[b] : p.cu_k[b + 1] - k_start;
   if (m_blk * kPM >= q_len) return;  // uniform over the CTA, before anything is allocated
@@ -87,9 +103,9 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;
-  uint8_t* sK = sQ + kPTile;       // [2 stages][2 atoms]
-  uint8_t* sV = sK + 2 * kPTile;   // [2 stages][2 atoms], V^T: rows = d, columns = keys
-  uint8_t* sP = sV + 2 * kPTile;   // [2 atoms], rows = queries, columns = keys
+  uint8_t* sK = sQ + kQkTile;           // [stages][atoms]
+  uint8_t* sV = sK + kKSt * kQkTile;    // [stages][2 atoms], V^T: rows = d, columns = keys
+  uint8_t* sP = sV + kVSt * kPTile;     // [2 atoms], rows = queries, columns = keys
   uint64_t* bars = reinterpret_cast<uint64_t*>(sP + kPTile);
   uint64_t* q_full = bars;          // [1]
   uint64_t* k_full = bars + 1;      // [2]
@@ -137,20 +153,20 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   if (warp == 0) {
     // ------------------------------------------------------------------ TMA producer
     if (elect_one() && n_steps > 0) {  // nothing may be in flight into shared memory when nobody will wait for it
-      mbar_expect_tx(q_full, kPTile);
-      tma_load_3d(sQ, &tmQ, q_full, 0, h, q_start + m_blk * kPM);
-      tma_load_3d(sQ + kPAtom, &tmQ, q_full, 64, h, q_start + m_blk * kPM);
+      mbar_expect_tx(q_full, kQkTile);
+#pragma unroll
+      for (int a = 0; a < kDkAtoms; ++a) tma_load_3d(sQ + a * kPAtom, &tmQ, q_full, 64 * a, h, q_start + m_blk * kPM);
       for (int j = 0; j < n_steps; ++j) {
-        const int st = j & 1;
-        const uint32_t ph = (j >> 1) & 1;
-        if (!mbar_wait(k_empty + st, ph ^ 1, abort_flag, timeout_ns)) break;
-        mbar_expect_tx(k_full + st, kPTile);
-        tma_load_3d(sK + st * kPTile, &tmK, k_full + st, 0, kvh, k_start + j * kPN);
-        tma_load_3d(sK + st * kPTile + kPAtom, &tmK, k_full + st, 64, kvh, k_start + j * kPN);
-        if (!mbar_wait(v_empty + st, ph ^ 1, abort_flag, timeout_ns)) break;
-        mbar_expect_tx(v_full + st, kPTile);
-        tma_load_3d(sV + st * kPTile, &tmVt, v_full + st, j * kPN, 0, b * p.Hkv + kvh);
-        tma_load_3d(sV + st * kPTile + kPAtom, &tmVt, v_full + st, j * kPN + 64, 0, b * p.Hkv + kvh);
+        const int ks = j % kKSt, vs = j % kVSt;
+        if (!mbar_wait(k_empty + ks, ((j / kKSt) & 1) ^ 1, abort_flag, timeout_ns)) break;
+        mbar_expect_tx(k_full + ks, kQkTile);
+#pragma unroll
+        for (int a = 0; a < kDkAtoms; ++a)
+          tma_load_3d(sK + ks * kQkTile + a * kPAtom, &tmK, k_full + ks, 64 * a, kvh, k_start + j * kPN);
+        if (!mbar_wait(v_empty + vs, ((j / kVSt) & 1) ^ 1, abort_flag, timeout_ns)) break;
+        mbar_expect_tx(v_full + vs, kPTile);
+        tma_load_3d(sV + vs * kPTile, &tmVt, v_full + vs, j * kPN, v_col0, b * p.Hkv + kvh);
+        tma_load_3d(sV + vs * kPTile + kPAtom, &tmVt, v_full + vs, j * kPN + 64, v_col0, b * p.Hkv + kvh);
       }
     }
     __syncwarp();
@@ -160,18 +176,18 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       const uint32_t idesc = umma_idesc_f16(kPM, kPN, p.bf16 != 0);
       bool ok = mbar_wait(q_full, 0, abort_flag, timeout_ns);
       auto issue_scores = [&](int j) -> bool {
-        const int st = j & 1;
+        const int st = j & 1, ks = j % kKSt;
         const uint32_t ph = (j >> 1) & 1;
-        if (!mbar_wait(k_full + st, ph, abort_flag, timeout_ns)) return false;
+        if (!mbar_wait(k_full + ks, (j / kKSt) & 1, abort_flag, timeout_ns)) return false;
         if (!mbar_wait(s_empty + st, ph ^ 1, abort_flag, timeout_ns)) return false;
         tc_fence_after_sync();
 #pragma unroll
-        for (int kk = 0; kk < kPD / 16; ++kk) {
+        for (int kk = 0; kk < kDkAtoms * 4; ++kk) {
           const uint64_t da = umma_desc_sw128_kmajor(smem_u32(sQ + (kk >> 2) * kPAtom)) + 2 * (kk & 3);
-          const uint64_t db = umma_desc_sw128_kmajor(smem_u32(sK + st * kPTile + (kk >> 2) * kPAtom)) + 2 * (kk & 3);
+          const uint64_t db = umma_desc_sw128_kmajor(smem_u32(sK + ks * kQkTile + (kk >> 2) * kPAtom)) + 2 * (kk & 3);
           umma_f16(tmem_base + st * kPN, da, db, idesc, kk != 0 ? 1u : 0u);
         }
-        umma_commit(k_empty + st);
+        umma_commit(k_empty + ks);
         umma_commit(s_full + st);
         return true;
       };
@@ -179,18 +195,18 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       for (int j = 0; j < n_steps && ok; ++j) {
         if (j + 1 < n_steps) ok = issue_scores(j + 1);
         if (!ok) break;
-        const int st = j & 1;
+        const int vs = j % kVSt;
         if (!mbar_wait(p_full, j & 1, abort_flag, timeout_ns)) break;
-        if (!mbar_wait(v_full + st, (j >> 1) & 1, abort_flag, timeout_ns)) break;
+        if (!mbar_wait(v_full + vs, (j / kVSt) & 1, abort_flag, timeout_ns)) break;
         if (!mbar_wait(o_empty, (j & 1) ^ 1, abort_flag, timeout_ns)) break;
         tc_fence_after_sync();
 #pragma unroll
         for (int kk = 0; kk < kPN / 16; ++kk) {
           const uint64_t da = umma_desc_sw128_kmajor(smem_u32(sP + (kk >> 2) * kPAtom)) + 2 * (kk & 3);
-          const uint64_t db = umma_desc_sw128_kmajor(smem_u32(sV + st * kPTile + (kk >> 2) * kPAtom)) + 2 * (kk & 3);
+          const uint64_t db = umma_desc_sw128_kmajor(smem_u32(sV + vs * kPTile + (kk >> 2) * kPAtom)) + 2 * (kk & 3);
           umma_f16(tmem_base + 2 * kPN, da, db, idesc, kk != 0 ? 1u : 0u);
         }
-        umma_commit(v_empty + st);
+        umma_commit(v_empty + vs);
         umma_commit(o_full);
       }
     }
@@ -313,11 +329,13 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     xsum[half * kPM + row] = l_run;
     softmax_bar();
     l_run += xsum[(half ^ 1) * kPM + row];
+    if (p.sink != nullptr) l_run += exp2f(p.sink[h] * 1.4426950408889634f - m_run);  // the sink counts once, unscaled
     if (ok && q_pos < q_len) {
       const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-      uint8_t* dst = static_cast<uint8_t*>(p.out) + ((static_cast<size_t>(q_start + q_pos) * p.Hq + h) * kPD + col0) * 2;
+      uint8_t* dst = static_cast<uint8_t*>(p.out) + ((static_cast<size_t>(q_start + q_pos) * p.Hq + h) * p.dv + v_col0 + col0) * 2;
 #pragma unroll
       for (int c = 0; c < 8; ++c) {
+        if (v_col0 + col0 + c * 8 >= p.dv) break;
         float f[8];
 #pragma unroll
         for (int i = 0; i < 8; ++i) f[i] = o[c * 8 + i] * inv;
@@ -334,6 +352,48 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   __syncthreads();
   if (warp == 2) tmem_dealloc(tmem_base, 512);
   if (threadIdx.x == 0 && *abort_flag != 0u && p.status != nullptr) atomicMax(p.status, static_cast<uint32_t>(kStatusPipeTimeout));
+}
+
+template <int kDkAtoms>
+static int launch_prefill_atoms(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const PrefillParams& p, dim3 grid,
+                                cudaStream_t s) {
+  static bool configured[64] = {false};
+  int dev = 0;
+  B200_CHECK_CUDA(cudaGetDevice(&dev));
+  if (!configured[dev & 63]) {
+    B200_CHECK_CUDA(cudaFuncSetAttribute(prefill_attn_kernel<kDkAtoms>, cudaFuncAttributeMaxDynamicSharedMemorySize, prefill_smem(kDkAtoms)));
+    configured[dev & 63] = true;
+  }
+  prefill_attn_kernel<kDkAtoms><<<grid, kPThreads, prefill_smem(kDkAtoms), s>>>(tq, tk, tv, p);
+  B200_CHECK_CUDA(cudaGetLastError());
+  return kOk;
+}
+
+static int prefill_launch(const void* q, int64_t ldq, const void* k, const void* vt, int s_pad, const int* cu_q, const int* cu_k,
+                          const int* k_lens, int B, int total_q, int total_k, int max_q, int Hq, int Hkv, int dk, int dv, float scale,
+                          int causal, const float* sink, void* out, int dtype, uint32_t* status, cudaStream_t s) {
+  CUtensorMap tq, tk, tv;
+  int rc = make_tma_3d(&tq, q, dtype, dk, Hq, total_q, dk, static_cast<uint64_t>(ldq), 64, 1, kPM, true);
+  if (rc != kOk) return rc;
+  rc = make_tma_3d(&tk, k, dtype, dk, Hkv, total_k, dk, static_cast<uint64_t>(Hkv) * dk, 64, 1, kPN, true);
+  if (rc != kOk) return rc;
+  rc = make_tma_3d(&tv, vt, dtype, s_pad, dv, static_cast<uint64_t>(B) * Hkv, s_pad, static_cast<uint64_t>(dv) * s_pad, 64, kPD, 1, true);
+  if (rc != kOk) return rc;
+  PrefillParams p;
+  memset(&p, 0, sizeof(p));
+  p.Hq = Hq; p.Hkv = Hkv; p.causal = causal; p.bf16 = dtype == kBF16;
+  p.dk = dk; p.dv = dv; p.v_chunks = (dv + kPD - 1) / kPD; p.sink = sink;
+  p.cu_q = cu_q; p.cu_k = cu_k; p.k_lens = k_lens;
+  p.scale_log2e = scale * 1.4426950408889634f;
+  p.out = out; p.status = status;
+  const dim3 grid((max_q + kPM - 1) / kPM, Hq * p.v_chunks, B);
+  B200_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "prefill attention grid is too large");
+  switch ((dk + 63) / 64) {
+    case 1: return launch_prefill_atoms<1>(tq, tk, tv, p, grid, s);
+    case 2: return launch_prefill_atoms<2>(tq, tk, tv, p, grid, s);
+    case 3: return launch_prefill_atoms<3>(tq, tk, tv, p, grid, s);
+    default: return launch_prefill_atoms<4>(tq, tk, tv, p, grid, s);
+  }
 }
 
 }  // namespace b200
@@ -368,29 +428,24 @@ B200_API int b200_prefill_attention(const void* q, const void* k, const void* v,
   transpose_v_kernel<<<dim3(s_pad / 32, kPD / 32, B * Hkv), 256, 0, s>>>(static_cast<const uint16_t*>(v),
                                                                           static_cast<uint16_t*>(vt_scratch), cu_k, k_lens, Hkv, s_pad);
   B200_CHECK_CUDA(cudaGetLastError());
-  CUtensorMap tq, tk, tv;
-  int rc = make_tma_3d(&tq, q, dtype, kPD, Hq, total_q, kPD, static_cast<uint64_t>(Hq) * kPD, 64, 1, kPM, true);
-  if (rc != kOk) return rc;
-  rc = make_tma_3d(&tk, k, dtype, kPD, Hkv, total_k, kPD, static_cast<uint64_t>(Hkv) * kPD, 64, 1, kPN, true);
-  if (rc != kOk) return rc;
-  rc = make_tma_3d(&tv, vt_scratch, dtype, s_pad, kPD, static_cast<uint64_t>(B) * Hkv, s_pad,
-                   static_cast<uint64_t>(kPD) * s_pad, 64, kPD, 1, true);
-  if (rc != kOk) return rc;
-  static bool configured[64] = {false};
-  int dev = 0;
-  B200_CHECK_CUDA(cudaGetDevice(&dev));
-  if (!configured[dev & 63]) {
-    B200_CHECK_CUDA(cudaFuncSetAttribute(prefill_attn_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kPSmem));
-    configured[dev & 63] = true;
-  }
-  PrefillParams p;
-  memset(&p, 0, sizeof(p));
-  p.Hq = Hq; p.Hkv = Hkv; p.causal = causal; p.bf16 = dtype == kBF16;
-  p.cu_q = cu_q; p.cu_k = cu_k; p.k_lens = k_lens;
-  p.scale_log2e = scale * 1.4426950408889634f;
-  p.out = out; p.status = status;
-  dim3 grid((max_q + kPM - 1) / kPM, Hq, B);
-  prefill_attn_kernel<<<grid, kPThreads, kPSmem, s>>>(tq, tk, tv, p);
-  B200_CHECK_CUDA(cudaGetLastError());
-  return kOk;
+  return prefill_launch(q, static_cast<int64_t>(Hq) * kPD, k, vt_scratch, s_pad, cu_q, cu_k, k_lens, B, total_q, total_k, max_q, Hq,
+                        Hkv, kPD, kPD, scale, causal, nullptr, out, dtype, status, s);
+}
+
+// As b200_prefill_attention for head sizes other than 128 and values that are already transposed:
+//   q [total_q, Hq, dk] with ldq elements between two tokens; k [total_k, Hkv, dk] contiguous; vt [B * Hkv, dv, s_pad] with the
+//   keys of a sequence in its first columns (columns up to the next multiple of 128 below s_pad are read and must be finite);
+//   sink: nullable fp32 [Hq] on the device, a logit that joins every row's softmax denominator unscaled and has no value;
+//   out [total_q, Hq, dv]. dk, dv, ldq and s_pad are multiples of 8, dk <= 256.
+B200_API int b200_prefill_attention_vt(const void* q, long long ldq, const void* k, const void* vt, int s_pad, const int* cu_q,
+                                       const int* cu_k, const int* k_lens, int B, int total_q, int total_k, int max_q, int Hq,
+                                       int Hkv, int dk, int dv, float scale, int causal, const float* sink, void* out, int dtype,
+                                       uint32_t* status, void* stream) {
+  B200_REQUIRE(dtype == kBF16 || dtype == kF16, "prefill attention supports bf16/f16");
+  B200_REQUIRE(Hkv > 0 && Hq % Hkv == 0, "Hq (%d) must be a multiple of Hkv (%d)", Hq, Hkv);
+  B200_REQUIRE(B >= 1 && max_q >= 1 && total_q >= 1 && total_k >= 1 && s_pad >= 1, "empty problem");
+  B200_REQUIRE(dk >= 8 && dk % 8 == 0 && dk <= 256 && dv >= 8 && dv % 8 == 0 && ldq % 8 == 0 && s_pad % 8 == 0,
+               "prefill attention needs dk (%d) <= 256, and dk, dv (%d), ldq, s_pad (%d) in multiples of 8", dk, dv, s_pad);
+  return prefill_launch(q, ldq, k, vt, s_pad, cu_q, cu_k, k_lens, B, total_q, total_k, max_q, Hq, Hkv, dk, dv, scale, causal, sink,
+                        out, dtype, status, static_cast<cudaStream_t>(stream));
 }

@@ -1,0 +1,252 @@
+// The residual stream of decoders that keep it in fp32: embedding, gated sublayer sums, a weighted average over the
+// states of all earlier layers ("depth average"), and the norm whose output the next layer's GEMMs read. One CTA per
+// token, one pass: everything a layer does between its last GEMM and the next layer's first one is one kernel.
+//
+//   embed_norm       x = table[id] * scale;  state_0 = x;  h = norm(x)
+//   residual_norm    s = x + mult * (sigmoid(ga + ba) * a + sigmoid(gb + bb) * b)     (gates and b optional)
+//                    state_n = s;  x = w_0 state_0 + ... + w_{n-1} state_{n-1} + w_n s (with weights; else x = s)
+//                    h = norm(x)
+// norm is layer norm (center = 1: mean removed, variance = mean of squared deviations) or RMS norm (center = 0), with a
+// gain and an optional bias. The stream, the states and all arithmetic are fp32; a, b, the gates and h have the model's
+// storage type (bf16 / f16 / fp32). Rows are `pitch` wide: columns in [width, pitch) are padding, which carries zeros and
+// is left out of the statistics.
+#include "b200/elem.cuh"
+#include "b200/host.h"
+
+#include <cstring>
+
+namespace b200 {
+
+constexpr int kRnThreads = 512;
+
+struct NormParams {
+  int width, pitch, center;
+  float eps;
+  const void* gain;   // [pitch]; null: no norm, h is not written
+  const void* bias;   // [pitch] or null
+  void* h;            // [T, pitch]
+};
+
+struct ResidualParams {
+  const void *a, *b;              // sublayer results [T, pitch]; b nullable
+  const void *gate_a, *gate_b;    // gate logits [T, *] with row pitch ldg; null = no gate
+  const void *bias_a, *bias_b;    // [pitch] or null
+  int ldg;
+  float mult;
+  float* x;                       // [T, pitch] in / out
+  float* states;                  // [*, T, pitch] states 0 .. n_prev - 1 are read; null without weights
+  long long state_stride;         // elements between two states
+  const float* weights;           // [n_prev + 1] or null
+  int n_prev;
+  int keep;                       // store the new state at index n_prev
+  NormParams norm;
+};
+
+struct EmbedParams {
+  const long long* ids;
+  const void* table;   // [V, pitch]
+  long long V;
+  float scale;
+  float* x;            // [T, pitch]
+  float* state0;       // [T, pitch] or null
+  NormParams norm;
+};
+
+__device__ __forceinline__ float block_sum(float v, float* red) {
+  v = warp_sum(v);
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  const int nw = blockDim.x >> 5;
+  return warp_sum((threadIdx.x & 31) < nw ? red[threadIdx.x & 31] : 0.f);
+}
+
+// U groups of four columns per thread: group u of a thread starts at column 4 * (threadIdx.x + u * blockDim.x)
+template <typename T, int U>
+__device__ __forceinline__ void norm_row(const NormParams& n, size_t row, const float4 (&v)[U], const float4 (&gain)[U],
+                                         const float4 (&bias)[U], float* red) {
+  if (n.gain == nullptr) return;
+  float mean = 0.f;
+  if (n.center) {
+    float s = 0.f;
+#pragma unroll
+    for (int u = 0; u < U; ++u) s += (v[u].x + v[u].y) + (v[u].z + v[u].w);
+    mean = block_sum(s, red) / n.width;
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    const int c = 4 * (threadIdx.x + u * blockDim.x);
+    const float d[4] = {v[u].x - mean, v[u].y - mean, v[u].z - mean, v[u].w - mean};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) ss += c + e < n.width ? d[e] * d[e] : 0.f;
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / n.width + n.eps);
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    const int c = 4 * (threadIdx.x + u * blockDim.x);
+    if (c < n.pitch) {
+      float4 o;
+      o.x = (v[u].x - mean) * inv * gain[u].x + bias[u].x;
+      o.y = (v[u].y - mean) * inv * gain[u].y + bias[u].y;
+      o.z = (v[u].z - mean) * inv * gain[u].z + bias[u].z;
+      o.w = (v[u].w - mean) * inv * gain[u].w + bias[u].w;
+      store4(static_cast<T*>(n.h) + row * n.pitch + c, o);
+    }
+  }
+}
+
+// the gain and bias are weights: read before the dependency wait
+template <typename T, int U>
+__device__ __forceinline__ void load_norm_weights(const NormParams& n, float4 (&gain)[U], float4 (&bias)[U]) {
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    const int c = 4 * (threadIdx.x + u * blockDim.x);
+    gain[u] = bias[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (n.gain != nullptr && c < n.pitch) {
+      gain[u] = load4(static_cast<const T*>(n.gain) + c);
+      if (n.bias != nullptr) bias[u] = load4(static_cast<const T*>(n.bias) + c);
+    }
+  }
+}
+
+template <typename T, int U>
+__global__ void __launch_bounds__(kRnThreads) embed_norm_kernel(const EmbedParams p) {
+  __shared__ float red[32];
+  const size_t t = blockIdx.x;
+  const int pitch = p.norm.pitch;
+  griddep_launch_dependents();
+  float4 gain[U], bias[U], v[U];
+  load_norm_weights<T, U>(p.norm, gain, bias);
+  griddep_wait();
+  const long long id = p.ids[t];
+  const bool ok = id >= 0 && id < p.V;   // an id outside the table reads as a zero row
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    const int c = 4 * (threadIdx.x + u * blockDim.x);
+    v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < pitch) {
+      if (ok) v[u] = load4(static_cast<const T*>(p.table) + static_cast<size_t>(id) * pitch + c);
+      v[u].x *= p.scale; v[u].y *= p.scale; v[u].z *= p.scale; v[u].w *= p.scale;
+      store4(p.x + t * pitch + c, v[u]);
+      if (p.state0 != nullptr) store4(p.state0 + t * pitch + c, v[u]);
+    }
+  }
+  norm_row<T, U>(p.norm, t, v, gain, bias, red);
+}
+
+__device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+
+template <typename T>
+__device__ __forceinline__ float4 gated(const void* val, const void* gate, const void* bias, size_t row, int pitch, int ldg, int c) {
+  float4 a = load4(static_cast<const T*>(val) + row * pitch + c);
+  if (gate != nullptr) {
+    float4 z = load4(static_cast<const T*>(gate) + row * ldg + c);
+    if (bias != nullptr) {
+      const float4 b = load4(static_cast<const T*>(bias) + c);
+      z.x += b.x; z.y += b.y; z.z += b.z; z.w += b.w;
+    }
+    a.x *= sigmoid(z.x); a.y *= sigmoid(z.y); a.z *= sigmoid(z.z); a.w *= sigmoid(z.w);
+  }
+  return a;
+}
+
+template <typename T, int U>
+__global__ void __launch_bounds__(kRnThreads) residual_norm_kernel(const ResidualParams p) {
+  __shared__ float red[32];
+  const size_t t = blockIdx.x;
+  const int pitch = p.norm.pitch;
+  griddep_launch_dependents();
+  float4 gain[U], bias[U], x[U];
+  load_norm_weights<T, U>(p.norm, gain, bias);
+  griddep_wait();
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    const int c = 4 * (threadIdx.x + u * blockDim.x);
+    x[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c >= pitch) continue;
+    const size_t at = t * pitch + c;
+    float4 r = load4(p.x + at);
+    const float4 a = gated<T>(p.a, p.gate_a, p.bias_a, t, pitch, p.ldg, c);
+    float4 s = a;
+    if (p.b != nullptr) {
+      const float4 b = gated<T>(p.b, p.gate_b, p.bias_b, t, pitch, p.ldg, c);
+      s.x += b.x; s.y += b.y; s.z += b.z; s.w += b.w;
+    }
+    r.x = fmaf(p.mult, s.x, r.x); r.y = fmaf(p.mult, s.y, r.y); r.z = fmaf(p.mult, s.z, r.z); r.w = fmaf(p.mult, s.w, r.w);
+    if (p.weights != nullptr) {
+      if (p.keep) store4(p.states + p.n_prev * p.state_stride + at, r);
+      const float wn = __ldg(p.weights + p.n_prev);
+      r.x *= wn; r.y *= wn; r.z *= wn; r.w *= wn;
+      const float* st = p.states + at;
+#pragma unroll 8
+      for (int j = 0; j < p.n_prev; ++j) {
+        const float w = __ldg(p.weights + j);
+        const float4 o = load4(st + j * p.state_stride);
+        r.x = fmaf(w, o.x, r.x); r.y = fmaf(w, o.y, r.y); r.z = fmaf(w, o.z, r.z); r.w = fmaf(w, o.w, r.w);
+      }
+    }
+    x[u] = r;
+    store4(p.x + at, r);
+  }
+  norm_row<T, U>(p.norm, t, x, gain, bias, red);
+}
+
+static int check_norm(const NormParams& n) {
+  B200_REQUIRE(n.width > 0 && n.pitch % 4 == 0 && n.pitch >= n.width, "row pitch (%d) must be a multiple of 4 and >= width (%d)",
+               n.pitch, n.width);
+  B200_REQUIRE(n.pitch <= 4 * 8 * kRnThreads, "width (%d) is limited to %d", n.width, 4 * 8 * kRnThreads);
+  B200_REQUIRE(n.gain == nullptr || n.h != nullptr, "the norm needs an output");
+  return kOk;
+}
+static int row_threads(int pitch) {
+  const int t = (pitch / 4 + 31) / 32 * 32;
+  return t < kRnThreads ? t : kRnThreads;
+}
+
+template <typename T, typename P>
+static int launch_rows(void (*k1)(P), void (*k2)(P), void (*k4)(P), void (*k8)(P), const P& p, int T_rows, cudaStream_t s) {
+  const int threads = row_threads(p.norm.pitch);
+  const int groups = (p.norm.pitch / 4 + threads - 1) / threads;
+  B200_CHECK_CUDA(launch_pdl(groups == 1 ? k1 : groups == 2 ? k2 : groups <= 4 ? k4 : k8, dim3(T_rows), dim3(threads), 0, s, p));
+  return kOk;
+}
+
+}  // namespace b200
+
+using namespace b200;
+
+B200_API int b200_embed_norm(const long long* ids, const void* table, int rows, long long V, int width, int pitch, float scale,
+                             float* x, float* state0, const void* gain, const void* bias, float eps, int center, void* h,
+                             int dtype, void* stream) {
+  if (rows <= 0) return kOk;
+  EmbedParams p;
+  memset(&p, 0, sizeof(p));
+  p.ids = ids; p.table = table; p.V = V; p.scale = scale; p.x = x; p.state0 = state0;
+  p.norm = NormParams{width, pitch, center, eps, gain, bias, h};
+  int rc = check_norm(p.norm);
+  if (rc != kOk) return rc;
+  B200_DISPATCH_FLOAT(dtype, return launch_rows<T>(embed_norm_kernel<T, 1>, embed_norm_kernel<T, 2>, embed_norm_kernel<T, 4>,
+                                                   embed_norm_kernel<T, 8>, p, rows, static_cast<cudaStream_t>(stream)););
+}
+
+// `states` holds n_prev earlier states of [rows, pitch] each, state_stride elements apart; with keep != 0 the new state
+// is stored behind them. weights [n_prev + 1] fp32 on the device, null = no depth average.
+B200_API int b200_residual_norm(const void* a, const void* gate_a, const void* bias_a, const void* b, const void* gate_b,
+                                const void* bias_b, int ldg, float mult, float* x, float* states, long long state_stride,
+                                const float* weights, int n_prev, int keep, int rows, int width, int pitch, const void* gain,
+                                const void* bias, float eps, int center, void* h, int dtype, void* stream) {
+  if (rows <= 0) return kOk;
+  B200_REQUIRE(a != nullptr && x != nullptr, "residual_norm needs a sublayer result and the stream");
+  B200_REQUIRE(weights == nullptr || (states != nullptr && n_prev >= 1), "the depth average needs the earlier states");
+  B200_REQUIRE(ldg % 4 == 0, "the gates' row pitch (%d) must be a multiple of 4", ldg);
+  ResidualParams p;
+  memset(&p, 0, sizeof(p));
+  p.a = a; p.b = b; p.gate_a = gate_a; p.gate_b = gate_b; p.bias_a = bias_a; p.bias_b = bias_b; p.ldg = ldg; p.mult = mult;
+  p.x = x; p.states = states; p.state_stride = state_stride; p.weights = weights; p.n_prev = n_prev; p.keep = keep;
+  p.norm = NormParams{width, pitch, center, eps, gain, bias, h};
+  int rc = check_norm(p.norm);
+  if (rc != kOk) return rc;
+  B200_DISPATCH_FLOAT(dtype, return launch_rows<T>(residual_norm_kernel<T, 1>, residual_norm_kernel<T, 2>, residual_norm_kernel<T, 4>,
+                                                   residual_norm_kernel<T, 8>, p, rows, static_cast<cudaStream_t>(stream)););
+}

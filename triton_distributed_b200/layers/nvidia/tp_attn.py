@@ -124,7 +124,7 @@ class TP_Attn:
         cu_q = torch.arange(0, (bsz + 1) * seqlen, seqlen, dtype=torch.int32, device=qkv.device)
         cu_k = torch.arange(0, (bsz + 1) * L, L, dtype=torch.int32, device=qkv.device)
         o = ops.prefill_attention(q, kp.view(-1, self.kv_heads_local, self.head_dim), vp.view(-1, self.kv_heads_local, self.head_dim),
-                                  cu_q, cu_k, seqlen, min(L, kv_cache.max_length), self.scale, True, seqlens_k=step["kv_lens"])
+                                  cu_q, cu_k, seqlen, min(L, step.get("kv_len") or kv_cache.max_length), self.scale, True, seqlens_k=step["kv_lens"])
         return o.reshape(bsz * seqlen, -1)
 
     def _attn_torch(self, qkv, position_ids, cos_sin_cache, kv_cache, layer_idx, bsz, seqlen):

@@ -3,7 +3,8 @@
 API parity with ``python/triton_dist/models/engine.py:37-187``: ``Engine(model_config, temperature, top_p,
 verbose, group)``, attributes ``backend`` / ``no_graph`` / ``enable_profile``, and ``serve(input_ids, gen_len)``.
 The decode graph contains the whole forward (embedding to logits); sampling runs after each replay, as
-in the reference (:164-177).
+in the reference (:164-177). ``start`` / ``extend`` are the step function underneath: the next tokens of every sequence in,
+logits of any of them out, from the cache that earlier steps left.
 """
 from __future__ import annotations
 
@@ -13,16 +14,16 @@ import torch
 import torch.distributed as dist
 
 from ..kernels.allreduce import AllReduceMethod
+from .auto import AutoLLM
 from .config import ModelConfig
-from .kv_cache import KV_Cache
-from .qwen import Qwen3
+from .kv_cache import PagedCache
 from .utils import logger, sample_token
 
 
 class Engine:
 
     def __init__(self, model_config: ModelConfig, temperature: float = 0.6, top_p: float = 0.95, verbose: bool = False,
-                 group=None, model: Qwen3 | None = None):
+                 group=None, model=None):
         self.model_config = model_config
         self.temperature, self.top_p, self.verbose, self.group = temperature, top_p, verbose, group
         self.backend = "triton_dist_AR"      # decode backend: torch | triton_dist | triton_dist_AR
@@ -30,18 +31,20 @@ class Engine:
         self.no_graph = False
         self.enable_profile = False
         self.ar_method: AllReduceMethod | None = None
-        self.model = model if model is not None else Qwen3(model_config, group)
-        self.kv_cache: KV_Cache | None = None
+        self.model = model if model is not None else AutoLLM.from_pretrained(model_config, group)
+        self.kv_cache: PagedCache | None = None
         self.graph = None
         self.bsz = None
+        self.length = 0                      # tokens every sequence holds in the cache (host copy of its offsets)
+        self._decode_cache = None            # the cache the decode step was prepared for
 
     # ------------------------------------------------------------------ set-up
     def _init_kv_cache(self, bsz: int) -> None:
-        a = self.model.arch
         if self.kv_cache is None or self.kv_cache.batch_size != bsz:
-            self.kv_cache = KV_Cache(a.num_hidden_layers, bsz, self.model_config.max_length, a.num_key_value_heads,
-                                     a.head_dim, self.model_config.dtype, self.model_config.world_size)
+            self.graph = self._decode_cache = None
+            self.kv_cache = self.model.make_cache(bsz, self.model_config.max_length)
         self.kv_cache.clear()
+        self.length = 0
 
     def _set_backend(self, backend: str, max_M: int) -> None:
         m = self.model
@@ -76,17 +79,47 @@ class Engine:
         torch.cuda.synchronize()
 
     # ------------------------------------------------------------------ steps
-    @torch.no_grad()
-    def prefill(self, input_ids: torch.Tensor) -> torch.Tensor:
-        bsz, plen = input_ids.shape
+    def start(self, bsz: int) -> None:
+        """Begin `bsz` new sequences; what earlier ones held in the cache is given back."""
         self.bsz = bsz
         self._init_kv_cache(bsz)
-        backend = self.prefill_backend or self.backend
-        self._set_backend(backend, max(bsz * plen, bsz))
-        pos = torch.arange(plen, device=input_ids.device, dtype=torch.int64)[None, :].expand(bsz, plen).contiguous()
-        logits = self.model.inference(input_ids, pos, self.kv_cache)
-        self.kv_cache.kv_offset.fill_(plen)
-        return sample_token(logits, self.temperature, self.top_p)
+
+    @torch.no_grad()
+    def extend(self, input_ids: torch.Tensor, want: list[int] | None = None) -> torch.Tensor | None:
+        """Run the next tokens [B, S] of every sequence. Returns fp32 logits [B, len(want), V] at the places `want` among
+        these tokens (None: the last one; empty: the head is skipped and None returned). One token per sequence takes the
+        captured decode step, several take the prefill path. The logits of a decode step are valid until the next one."""
+        bsz, S = input_ids.shape
+        if self.kv_cache is None or bsz != self.bsz:
+            raise ValueError("start() the sequences first")
+        if self.length + S > self.model_config.max_length:
+            raise ValueError("the sequences would exceed max_length")
+        logits = None
+        if S == 1:
+            if self._decode_cache is not self.kv_cache:
+                self.prepare_decode(input_ids)
+            elif self.graph is None:
+                self._set_backend(self.backend, max(bsz, self.model_config.world_size))
+            logits = self._run_decode(input_ids)
+            if want is not None:
+                logits = logits.expand(-1, len(want), -1) if want else None
+        else:
+            self._set_backend(self.prefill_backend or self.backend, bsz * S)
+            pos = torch.arange(self.length, self.length + S, device=input_ids.device, dtype=torch.int64)[None, :].expand(bsz, S).contiguous()
+            kw = {"kv_len": self.length + S}
+            if want is None:
+                logits = self.model.inference(input_ids, pos, self.kv_cache, **kw)
+            else:
+                hidden = self.model.inference(input_ids, pos, self.kv_cache, wo_lm_head=True, **kw)
+                logits = self.model.lm_logits(hidden[:, want]) if want else None
+        self.kv_cache.inc_offset(S)
+        self.length += S
+        return logits
+
+    @torch.no_grad()
+    def prefill(self, input_ids: torch.Tensor) -> torch.Tensor:
+        self.start(input_ids.shape[0])
+        return sample_token(self.extend(input_ids), self.temperature, self.top_p)
 
     @torch.no_grad()
     def prepare_decode(self, first_token: torch.Tensor) -> None:
@@ -95,19 +128,25 @@ class Engine:
         self._static_ids = first_token.clone()
         self._static_pos = torch.zeros((bsz, 1), dtype=torch.int64, device=first_token.device)
         self._static_logits = None
+        self._decode_cache = self.kv_cache
         self._init_cuda_graph()
 
-    @torch.no_grad()
-    def decode_one(self, token: torch.Tensor | None = None) -> torch.Tensor:
-        """One decode step: feed `token` (default: the previously sampled one), return the next token ids [B, 1]."""
+    def _run_decode(self, token: torch.Tensor | None) -> torch.Tensor:
+        """One decode step on the static buffers (`token` None: the ids already there); logits [B, 1, V]."""
         if token is not None:
             self._static_ids.copy_(token, non_blocking=True)
         if self.graph is not None:
             self.graph.replay()
         else:
             self._decode_step()
-        nxt = sample_token(self._static_logits, self.temperature, self.top_p)
+        return self._static_logits
+
+    @torch.no_grad()
+    def decode_one(self, token: torch.Tensor | None = None) -> torch.Tensor:
+        """One decode step: feed `token` (default: the previously sampled one), return the next token ids [B, 1]."""
+        nxt = sample_token(self._run_decode(token), self.temperature, self.top_p)
         self.kv_cache.inc_offset()
+        self.length += 1
         self._static_ids.copy_(nxt)
         return nxt
 

@@ -1,42 +1,58 @@
-"""Paged KV cache, head-sharded over the tensor-parallel ranks.
+"""Paged caches: keys and values head-sharded over the tensor-parallel ranks, or one latent row per token and layer.
 
 Same interface as the reference's dense cache (``python/triton_dist/models/kv_cache.py:29-66``:
 ``update_kv_cache``, ``rand_fill_kv_cache``, ``inc_offset``, ``clear``, ``get_kv_len``) but stored as pages
 ``[layers, num_blocks, page, kv_heads / world, head_dim]`` with a block table, which is the layout the
 decode-attention kernel reads. Sequence b owns blocks ``b * blocks_per_seq ...`` so the table is static
-and a decode step can be captured in a CUDA graph.
+and a decode step can be captured in a CUDA graph. ``PagedCache`` owns the pages' bookkeeping (slots, block table,
+offsets), the subclasses own what a page holds.
 """
 from __future__ import annotations
 
 import torch
 
 
-class KV_Cache:
+class PagedCache:
 
-    def __init__(self, num_layers: int = 32, batch_size: int = 1, max_length: int = 32 * 1024, kv_heads: int = 8,
-                 head_dim: int = 128, dtype=torch.bfloat16, world_size: int = 8, page_size: int = 64,
-                 device="cuda") -> None:
+    def __init__(self, num_layers: int, batch_size: int, max_length: int, dtype, page_size: int = 64, device="cuda") -> None:
         self.num_layers, self.batch_size, self.max_length = num_layers, batch_size, max_length
-        self.kv_heads, self.head_dim, self.dtype, self.world_size = kv_heads, head_dim, dtype, world_size
-        self.page_size = page_size
-        self.local_kv_heads = max(1, kv_heads // world_size)
+        self.dtype, self.page_size = dtype, page_size
         self.blocks_per_seq = (max_length + page_size - 1) // page_size
-        nblk = batch_size * self.blocks_per_seq
-        shape = (num_layers, nblk, page_size, self.local_kv_heads, head_dim)
-        self.k_cache = torch.zeros(shape, device=device, dtype=dtype)
-        self.v_cache = torch.zeros(shape, device=device, dtype=dtype)
+        self.num_blocks = batch_size * self.blocks_per_seq
         self.kv_offset = torch.zeros(batch_size, dtype=torch.int32, device=device)
-        self.block_table = torch.arange(nblk, dtype=torch.int32, device=device).view(batch_size, self.blocks_per_seq)
-
-    def layer(self, layer_idx: int):
-        """(k pages, v pages) of one layer: [num_blocks, page, kv_heads_local, head_dim]."""
-        return self.k_cache[layer_idx], self.v_cache[layer_idx]
+        self.block_table = torch.arange(self.num_blocks, dtype=torch.int32, device=device).view(batch_size, self.blocks_per_seq)
 
     def slots(self, positions: torch.Tensor) -> torch.Tensor:
         """Flat slot index (block * page + offset) of token position [B, S] of every sequence -> int64 [B*S]."""
         B, S = positions.shape
         base = torch.arange(B, device=positions.device, dtype=torch.int64)[:, None] * (self.blocks_per_seq * self.page_size)
         return (base + positions.to(torch.int64)).reshape(-1)
+
+    def inc_offset(self, n: int = 1) -> None:
+        self.kv_offset += n
+
+    def clear(self) -> None:
+        self.kv_offset.zero_()
+
+    def get_kv_len(self) -> torch.Tensor:
+        return self.kv_offset
+
+
+class KV_Cache(PagedCache):
+
+    def __init__(self, num_layers: int = 32, batch_size: int = 1, max_length: int = 32 * 1024, kv_heads: int = 8,
+                 head_dim: int = 128, dtype=torch.bfloat16, world_size: int = 8, page_size: int = 64,
+                 device="cuda") -> None:
+        super().__init__(num_layers, batch_size, max_length, dtype, page_size, device)
+        self.kv_heads, self.head_dim, self.world_size = kv_heads, head_dim, world_size
+        self.local_kv_heads = max(1, kv_heads // world_size)
+        shape = (num_layers, self.num_blocks, page_size, self.local_kv_heads, head_dim)
+        self.k_cache = torch.zeros(shape, device=device, dtype=dtype)
+        self.v_cache = torch.zeros(shape, device=device, dtype=dtype)
+
+    def layer(self, layer_idx: int):
+        """(k pages, v pages) of one layer: [num_blocks, page, kv_heads_local, head_dim]."""
+        return self.k_cache[layer_idx], self.v_cache[layer_idx]
 
     def update_kv_cache(self, new_k: torch.Tensor, new_v: torch.Tensor, layer_idx: int):
         """Append [B, S, kv_heads_local, D] at the current offsets (the fused rope kernel normally does this)."""
@@ -52,11 +68,21 @@ class KV_Cache:
         self.v_cache.copy_(torch.rand_like(self.v_cache) / 10)
         self.kv_offset.fill_(offset)
 
-    def inc_offset(self, n: int = 1) -> None:
-        self.kv_offset += n
 
-    def clear(self) -> None:
-        self.kv_offset.zero_()
+class LatentCache(PagedCache):
+    """Latent attention's cache: layer i keeps one row of ``widths[i]`` elements per token (shared by all heads, so it is
+    replicated over tensor-parallel ranks), as pages ``[num_blocks, page, widths[i]]``."""
 
-    def get_kv_len(self) -> torch.Tensor:
-        return self.kv_offset
+    def __init__(self, widths: list[int], batch_size: int, max_length: int, dtype=torch.bfloat16, page_size: int = 64,
+                 device="cuda") -> None:
+        super().__init__(len(widths), batch_size, max_length, dtype, page_size, device)
+        self.c_cache = [torch.zeros((self.num_blocks, page_size, w), device=device, dtype=dtype) for w in widths]
+
+    def layer(self, layer_idx: int) -> torch.Tensor:
+        """Pages of one layer: [num_blocks, page, width]."""
+        return self.c_cache[layer_idx]
+
+    def rows(self, layer_idx: int, seq: int, count: int) -> torch.Tensor:
+        """The first `count` latent rows of sequence `seq` as one matrix (its pages are consecutive)."""
+        c = self.c_cache[layer_idx].view(self.batch_size, self.blocks_per_seq * self.page_size, -1)
+        return c[seq, :count]

@@ -90,6 +90,8 @@ class Qwen3Layer:
 
 class Qwen3:
 
+    dtypes = (torch.bfloat16, torch.float16)
+
     def __init__(self, model_config: ModelConfig, group=None, source: WeightSource | None = None):
         self.model_config = model_config
         self.group = group
@@ -146,6 +148,11 @@ class Qwen3:
         self.mode = mode
         for layer in self.layers:
             layer.set_fwd(mode)
+
+    def make_cache(self, batch_size: int, max_length: int | None = None) -> KV_Cache:
+        a = self.arch
+        return KV_Cache(a.num_hidden_layers, batch_size, max_length or self.max_length, a.num_key_value_heads, a.head_dim,
+                        self.dtype, self.world_size)
 
     # ------------------------------------------------------------------ contexts (shared by all layers)
     def init_triton_dist_ctx(self, max_M: int) -> None:
@@ -228,10 +235,10 @@ class Qwen3:
         return ops.rmsnorm(partial, gamma, self.eps, residual=residual)
 
     @torch.no_grad()
-    def _inference_AR(self, input_ids, position_ids, kv_cache):
+    def _inference_AR(self, input_ids, position_ids, kv_cache, kv_len=None):
         """Returns the final-normed hidden states [B, S, H]."""
         bsz, seqlen = input_ids.shape
-        step = {"pos": position_ids.reshape(-1).to(torch.int32), "slots": kv_cache.slots(position_ids),
+        step = {"pos": position_ids.reshape(-1).to(torch.int32), "slots": kv_cache.slots(position_ids), "kv_len": kv_len,
                 "kv_lens": (position_ids[:, -1] + 1).to(torch.int32)}
         residual = ops.embedding(input_ids.reshape(-1), self.embed_tokens)  # [T, H], becomes the residual stream
         x = ops.rmsnorm(residual, self.layers[0].input_norm_w, self.eps)
@@ -245,13 +252,14 @@ class Qwen3:
 
     @torch.no_grad()
     def inference(self, input_ids: torch.Tensor, position_ids: torch.Tensor, kv_cache: KV_Cache,
-                  wo_lm_head: bool = False) -> torch.Tensor:
+                  wo_lm_head: bool = False, kv_len: int | None = None) -> torch.Tensor:
         """input_ids / position_ids [B, S] (full batch on every rank). Returns fp32 logits [B, 1, V] of the last
-        position (or the normed hidden states with ``wo_lm_head``). ``triton_dist`` mode needs B % world == 0."""
+        position (or the normed hidden states with ``wo_lm_head``). ``triton_dist`` mode needs B % world == 0. `kv_len`: the
+        longest sequence after this step when the host knows it (bounds the work of a prefill)."""
         bsz, seqlen = input_ids.shape
         native_gather = self.world_size > 1 and self.gather_ctx is not None and bsz <= self.gather_rows
         if self.mode == "triton_dist_AR":
-            hidden = self._inference_AR(input_ids, position_ids, kv_cache)
+            hidden = self._inference_AR(input_ids, position_ids, kv_cache, kv_len)
         else:
             native = self.mode == "triton_dist"
             hidden = ops.embedding(input_ids, self.embed_tokens) if native else F.embedding(input_ids, self.embed_tokens)
@@ -278,7 +286,15 @@ class Qwen3:
                     hidden = full
         if wo_lm_head:
             return hidden
-        last = hidden[:, -1, :].contiguous()
+        return self._logits(hidden[:, -1, :].contiguous(), native_gather)
+
+    def lm_logits(self, hidden: torch.Tensor) -> torch.Tensor:
+        """fp32 logits [B, n, V] of normed hidden states [B, n, H]."""
+        return self._logits(hidden.reshape(-1, hidden.shape[-1]).contiguous(), False).view(*hidden.shape[:-1], -1)
+
+    def _logits(self, last: torch.Tensor, native_gather: bool) -> torch.Tensor:
+        """Head over rows [B, H] -> fp32 [B, 1, V]; the vocabulary shards are gathered over ranks."""
+        bsz = last.shape[0]
         if self.mode == "torch":
             local = F.linear(last, self.lm_head)
         elif native_gather:

@@ -13,7 +13,29 @@ import os
 
 import torch
 
-from .config import ArchConfig
+from .config import ArchConfig, LikosunConfig
+
+
+def likosun_param_shapes(arch: LikosunConfig) -> dict[str, tuple[int, ...]]:
+    """Names and shapes of a Likosun checkpoint (linear weights [out, in])."""
+    W = arch.hidden_size
+    out = {"embed": (arch.vocab_size, W)}
+    for i, layer in enumerate(arch.layers):
+        p, m = f"l{i}.", layer.mixer
+        out.update({p + "norm1": (W,), p + "norm1.b": (W,), p + "mix.q": (m.heads * m.dim, W), p + "mix.dkv": (m.kv_rank, W),
+                    p + "mix.dkv.norm": (m.kv_rank,), p + "mix.uk": (m.heads * m.dim, m.kv_rank),
+                    p + "mix.uv": (m.heads * m.vdim, m.kv_rank), p + "mix.sink": (m.heads,), p + "mix.o": (W, m.heads * m.vdim)})
+        if layer.mlp is not None:
+            out.update({p + "mlp.up": (layer.mlp.ff, W), p + "mlp.down": (W, layer.mlp.ff)})
+        for g in ("rg1", "rg2") if layer.mlp is not None else ("rg1",):
+            out.update({p + g: (W, W), p + g + ".b": (W,)})
+        out[p + "dwa"] = (i + 2,)
+    out.update({"final.norm": (W,), "final.norm.b": (W,), "head": (arch.vocab_size, W)})
+    return out
+
+
+def param_shapes(arch: ArchConfig | LikosunConfig) -> dict[str, tuple[int, ...]]:
+    return likosun_param_shapes(arch) if isinstance(arch, LikosunConfig) else hf_param_shapes(arch)
 
 
 def hf_param_shapes(arch: ArchConfig) -> dict[str, tuple[int, ...]]:
@@ -46,21 +68,51 @@ def hf_param_shapes(arch: ArchConfig) -> dict[str, tuple[int, ...]]:
     return out
 
 
-def _init_tensor(name: str, shape: tuple[int, ...], dtype: torch.dtype, seed: int, device="cpu") -> torch.Tensor:
-    """N(0, 0.02) for matrices, ones for norm gains; the stream depends only on (seed, name)."""
-    if name.endswith("norm.weight") or name.endswith("layernorm.weight"):
+def _constant_init(name: str, shape: tuple[int, ...], dtype: torch.dtype, device) -> torch.Tensor | None:
+    if name.endswith(("norm.weight", "layernorm.weight", ".norm", ".norm1")):
         return torch.ones(shape, dtype=dtype, device=device)
+    if name.endswith((".b", ".sink")):
+        return torch.zeros(shape, dtype=dtype, device=device)
+    if name.endswith(".dwa"):
+        t = torch.zeros(shape, dtype=dtype, device=device)
+        t[-1] = 1
+        return t
+    return None
+
+
+def _init_tensor(name: str, shape: tuple[int, ...], dtype: torch.dtype, seed: int, device="cpu") -> torch.Tensor:
+    """N(0, 0.02) for matrices, ones for norm gains, zeros for biases and sinks, the newest state alone for depth-average
+    weights; the stream depends only on (seed, name)."""
+    const = _constant_init(name, shape, dtype, device)
+    if const is not None:
+        return const
     g = torch.Generator(device=device)
     g.manual_seed((seed * 1000003 + sum(ord(c) * (i + 1) for i, c in enumerate(name))) % (2**31 - 1))
     return (torch.randn(shape, generator=g, dtype=torch.float32, device=device) * 0.02).to(dtype)
 
 
-def write_random_checkpoint(path: str, arch: ArchConfig, dtype: torch.dtype = torch.bfloat16, seed: int = 0,
+def _config_dict(arch: ArchConfig | LikosunConfig, dtype: torch.dtype) -> dict:
+    """Contents of config.json."""
+    if isinstance(arch, LikosunConfig):
+        return arch.to_dict()
+    return {
+        "architectures": ["Qwen3MoeForCausalLM" if arch.num_experts else "Qwen3ForCausalLM"],
+        "hidden_size": arch.hidden_size, "intermediate_size": arch.intermediate_size,
+        "num_hidden_layers": arch.num_hidden_layers, "num_attention_heads": arch.num_attention_heads,
+        "num_key_value_heads": arch.num_key_value_heads, "head_dim": arch.head_dim, "vocab_size": arch.vocab_size,
+        "rms_norm_eps": arch.rms_norm_eps, "rope_theta": arch.rope_theta,
+        "tie_word_embeddings": arch.tie_word_embeddings, "num_experts": arch.num_experts,
+        "num_experts_per_tok": arch.num_experts_per_tok, "moe_intermediate_size": arch.moe_intermediate_size,
+        "norm_topk_prob": arch.norm_topk_prob, "torch_dtype": str(dtype).replace("torch.", ""),
+    }
+
+
+def write_random_checkpoint(path: str, arch: ArchConfig | LikosunConfig, dtype: torch.dtype = torch.bfloat16, seed: int = 0,
                             max_shard_bytes: int = 2 << 30) -> None:
     """Write ``config.json``, ``model.safetensors.index.json`` and ``model-XXXXX-of-YYYYY.safetensors``."""
     from safetensors.torch import save_file
     os.makedirs(path, exist_ok=True)
-    shapes = hf_param_shapes(arch)
+    shapes = param_shapes(arch)
     shards: list[dict[str, torch.Tensor]] = [{}]
     size = 0
     for name, shape in shapes.items():
@@ -78,23 +130,17 @@ def write_random_checkpoint(path: str, arch: ArchConfig, dtype: torch.dtype = to
         weight_map.update({k: fname for k in shard})
     with open(os.path.join(path, "model.safetensors.index.json"), "w") as f:
         json.dump({"metadata": {}, "weight_map": weight_map}, f)
-    cfg = {
-        "architectures": ["Qwen3MoeForCausalLM" if arch.num_experts else "Qwen3ForCausalLM"],
-        "hidden_size": arch.hidden_size, "intermediate_size": arch.intermediate_size,
-        "num_hidden_layers": arch.num_hidden_layers, "num_attention_heads": arch.num_attention_heads,
-        "num_key_value_heads": arch.num_key_value_heads, "head_dim": arch.head_dim, "vocab_size": arch.vocab_size,
-        "rms_norm_eps": arch.rms_norm_eps, "rope_theta": arch.rope_theta,
-        "tie_word_embeddings": arch.tie_word_embeddings, "num_experts": arch.num_experts,
-        "num_experts_per_tok": arch.num_experts_per_tok, "moe_intermediate_size": arch.moe_intermediate_size,
-        "norm_topk_prob": arch.norm_topk_prob, "torch_dtype": str(dtype).replace("torch.", ""),
-    }
     with open(os.path.join(path, "config.json"), "w") as f:
-        json.dump(cfg, f, indent=1)
+        json.dump(_config_dict(arch, dtype), f, indent=1)
 
 
-def read_arch_from_checkpoint(path: str) -> ArchConfig:
+def read_arch_from_checkpoint(path: str) -> ArchConfig | LikosunConfig:
     with open(os.path.join(path, "config.json")) as f:
         c = json.load(f)
+    if c.get("architecture") == LikosunConfig.architecture:
+        return LikosunConfig.from_dict(c)
+    if "hidden_size" not in c:
+        raise ValueError(f"unknown architecture in {path}/config.json: {c.get('architecture', c.get('architectures'))!r}")
     return ArchConfig(
         hidden_size=c["hidden_size"], intermediate_size=c["intermediate_size"],
         num_hidden_layers=c["num_hidden_layers"], num_attention_heads=c["num_attention_heads"],
@@ -156,7 +202,7 @@ class SafetensorsSource(WeightSource):
 
 
 class RandomSource(WeightSource):
-    """Random initialisation in HF layout.
+    """Random initialisation under the checkpoint's names (HF layout for Qwen3).
 
     ``consistent=True`` draws every full tensor from a stream keyed by (seed, name) and slices it, so any
     tensor-parallel split sees the same model (tests). ``consistent=False`` draws only the requested slice,
@@ -164,8 +210,8 @@ class RandomSource(WeightSource):
     seconds; the result is a valid random-init model, just not the same one for different world sizes.
     """
 
-    def __init__(self, arch: ArchConfig, dtype: torch.dtype, seed: int = 0, device="cuda", consistent: bool = True):
-        self.shapes = hf_param_shapes(arch)
+    def __init__(self, arch: ArchConfig | LikosunConfig, dtype: torch.dtype, seed: int = 0, device="cuda", consistent: bool = True):
+        self.shapes = param_shapes(arch)
         self.dtype, self.seed, self.device, self.consistent = dtype, seed, device, consistent
 
     def has(self, name: str) -> bool:

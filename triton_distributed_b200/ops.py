@@ -49,10 +49,12 @@ def gemm(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor | None = None, max_
 
 
 class _SkinnyScratch:
-    """Per-device split-K scratch shared by all skinny GEMM calls of a stream (each call re-zeroes it)."""
+    """Per-device split-K scratch shared by all skinny GEMM calls of a stream (each call re-zeroes it). Buffers that were
+    outgrown stay allocated: a captured CUDA graph may hold their addresses."""
 
     def __init__(self):
         self.bufs: dict[int, tuple[torch.Tensor, torch.Tensor]] = {}
+        self.outgrown: list[tuple[torch.Tensor, torch.Tensor]] = []
 
     def get(self, device: torch.device, floats: int, tiles: int):
         key = device.index if device.index is not None else torch.cuda.current_device()
@@ -60,6 +62,7 @@ class _SkinnyScratch:
         if cur is None or cur[0].numel() < floats or cur[1].numel() < tiles:
             if cur is not None:
                 torch.cuda.synchronize()
+                self.outgrown.append(cur)
             nf = max(floats, 4 << 20, 0 if cur is None else cur[0].numel())
             nt = max(tiles, 4096, 0 if cur is None else cur[1].numel())
             cur = (torch.zeros(nf, dtype=torch.float32, device=device), torch.zeros(nt, dtype=torch.int32, device=device))
@@ -176,12 +179,30 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = Non
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
-    """``x @ w.T`` for any leading shape, routed to the skinny kernel for <= 256 rows, else the tiled one."""
+    """``x @ w.T`` for any leading shape: the skinny kernel for <= 256 rows, else the tiled one; fp32 has its own kernel."""
     lead = x.shape[:-1]
     x2 = x.reshape(-1, x.shape[-1])
     o2 = out.reshape(-1, w.shape[0]) if out is not None else None
-    y = gemm_skinny(x2, w, o2) if x2.shape[0] <= 256 else gemm(x2, w, o2)
+    if x2.dtype == torch.float32:
+        y = gemm_f32(x2, w, o2)
+    else:
+        y = gemm_skinny(x2, w, o2) if x2.shape[0] <= 256 else gemm(x2, w, o2)
     return y.reshape(*lead, w.shape[0])
+
+
+def gemm_f32(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+    """``a[M,K] @ b[N,K].T`` in true fp32 (no TF32), for the models' 32-bit mode."""
+    _lib.require_cuda()
+    _check_2d(a, "a"), _check_2d(b, "b")
+    M, K = a.shape
+    N = b.shape[0]
+    if b.shape[1] != K or a.dtype != torch.float32 or b.dtype != torch.float32:
+        raise ValueError("gemm_f32: shape/dtype mismatch")
+    if out is None:
+        out = torch.empty((M, N), dtype=a.dtype, device=a.device)
+    _lib.call("b200_gemm_f32", ptr(a), ptr(b), ptr(out), M, N, K, a.stride(0), b.stride(0), out.stride(0), stream_ptr())
+    _count()
+    return out
 
 
 def rmsnorm(x: torch.Tensor, gamma: torch.Tensor, eps: float, residual: torch.Tensor | None = None,
@@ -447,5 +468,148 @@ def combine_partials(o_part: torch.Tensor, lse_part: torch.Tensor, out_dtype: to
     _lib.call("b200_decode_combine", ptr(o_part), ptr(lse_part), ctypes.c_longlong(o_part.stride(1)),
               ctypes.c_longlong(o_part.stride(0)), ctypes.c_longlong(lse_part.stride(1)),
               ctypes.c_longlong(lse_part.stride(0)), BH, R, ptr(out), None, None, dtype_code(out_dtype), stream_ptr())
+    _count()
+    return out
+
+
+# ---- fp32 residual stream (csrc/kernels/residual.cu) ------------------------------------------
+def _norm_args(width, gain, bias, eps, center, h):
+    return ptr(gain), ptr(bias), c_float(eps), 1 if center else 0, ptr(h)
+
+
+def embed_norm(ids: torch.Tensor, table: torch.Tensor, scale: float, width: int, gain: torch.Tensor, bias: torch.Tensor | None,
+               eps: float, center: bool, state0: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
+    """``x = table[ids] * scale`` in fp32 and ``h = norm(x)`` in the table's type, one kernel. ids int64 [T]; table [V, P]
+    with P >= width columns (padding columns zero). ``center``: layer norm, else RMS norm. ``state0`` fp32 [T, P]
+    receives a copy of x. Returns (x fp32 [T, P], h [T, P])."""
+    _lib.require_cuda()
+    flat = ids.reshape(-1).to(torch.int64).contiguous()
+    T, P = flat.numel(), table.shape[1]
+    x = torch.empty((T, P), dtype=torch.float32, device=table.device)
+    h = torch.empty((T, P), dtype=table.dtype, device=table.device)
+    _lib.call("b200_embed_norm", ptr(flat), ptr(table), T, ctypes.c_longlong(table.shape[0]), width, P, c_float(scale), ptr(x),
+              ptr(state0), *_norm_args(width, gain, bias, eps, center, h), dtype_code(table.dtype), stream_ptr())
+    _count()
+    return x, h
+
+
+def residual_norm(x: torch.Tensor, width: int, mult: float, a: torch.Tensor, gate_a: torch.Tensor | None = None,
+                  bias_a: torch.Tensor | None = None, b: torch.Tensor | None = None, gate_b: torch.Tensor | None = None,
+                  bias_b: torch.Tensor | None = None, states: torch.Tensor | None = None, weights: torch.Tensor | None = None,
+                  keep: bool = False, gain: torch.Tensor | None = None, bias: torch.Tensor | None = None, eps: float = 0.0,
+                  center: bool = True) -> torch.Tensor | None:
+    """One pass over the fp32 residual stream ``x`` [T, P] (updated in place):
+    ``s = x + mult * (sigmoid(gate_a + bias_a) * a + sigmoid(gate_b + bias_b) * b)``; with ``weights`` (fp32 [n + 1])
+    ``x = sum_j weights[j] * states[j] + weights[n] * s`` over the n earlier states (``states`` fp32 [>= n, T, P]; s is stored
+    as state n with ``keep``), else ``x = s``; returns ``norm(x)`` when ``gain`` is given. a, b [T, P]; the gate logits may be
+    column slices of a wider GEMM output (same row pitch)."""
+    _lib.require_cuda()
+    T, P = x.shape
+    if x.dtype != torch.float32 or a.shape != x.shape or not a.is_contiguous() or (b is not None and (b.shape != x.shape or not b.is_contiguous())):
+        raise ValueError("residual_norm: x must be fp32 [T, P] and the sublayer results contiguous [T, P]")
+    ldg = gate_a.stride(0) if gate_a is not None else 0
+    if gate_b is not None and gate_a is not None and gate_b.stride(0) != ldg:
+        raise ValueError("residual_norm: the gates need one row pitch")
+    if gate_b is not None and gate_a is None:
+        ldg = gate_b.stride(0)
+    n = weights.numel() - 1 if weights is not None else 0
+    if weights is not None and (weights.dtype != torch.float32 or states is None or states.shape[0] < n + (1 if keep else 0)
+                                or states.shape[1:] != x.shape or not states.is_contiguous()):
+        raise ValueError("residual_norm: weights fp32 [n + 1] need contiguous fp32 states [>= n, T, P]")
+    h = torch.empty((T, P), dtype=a.dtype, device=a.device) if gain is not None else None
+    _lib.call("b200_residual_norm", ptr(a), ptr(gate_a), ptr(bias_a), ptr(b), ptr(gate_b), ptr(bias_b), ldg, c_float(mult), ptr(x),
+              ptr(states), ctypes.c_longlong(T * P), ptr(weights), n, 1 if keep else 0, T, width, P,
+              *_norm_args(width, gain, bias, eps, center, h), dtype_code(a.dtype), stream_ptr())
+    _count()
+    return h
+
+
+# ---- latent attention (csrc/kernels/latent_attn.cu, prefill_attn_sm100.cu) --------------------
+def latent_prep(latent_in: torch.Tensor | None, gain: torch.Tensor | None, cache: torch.Tensor | None, slots: torch.Tensor | None,
+                rank: int, eps: float, up: torch.Tensor | None = None) -> torch.Tensor | None:
+    """RMS norm of ``latent_in`` [T, >= rank] into rows ``slots`` (int64 [T]) of ``cache`` [..., P], and squared relu of ``up``
+    [T, I] (returned), in one launch. Both inputs may be column slices of the same GEMM output."""
+    _lib.require_cuda()
+    src = latent_in if latent_in is not None else up
+    T, ld = src.shape[0], src.stride(0)
+    if latent_in is not None and up is not None and up.stride(0) != ld:
+        raise ValueError("latent_prep: both inputs need one row pitch")
+    inter = up.shape[1] if up is not None else 0
+    act = torch.empty((T, inter), dtype=up.dtype, device=up.device) if up is not None else None
+    pitch = cache.shape[-1] if cache is not None else 0
+    _lib.call("b200_latent_prep", ptr(latent_in), ptr(gain), ptr(cache), ptr(slots), rank, pitch, c_float(eps), ptr(up), ptr(act),
+              inter, ld, T, dtype_code(src.dtype), stream_ptr())
+    _count()
+    return act
+
+
+def head_linear(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """Per-head GEMM ``y[t, h, :] = w[h] @ x[t, h, :]``: x [T, H, K] (unit inner stride), w [H, N, K] -> y [T, H, N]."""
+    _lib.require_cuda()
+    T, H, K = x.shape
+    N = w.shape[1]
+    if w.shape != (H, N, K) or not w.is_contiguous() or x.stride(2) != 1 or x.dtype != w.dtype:
+        raise ValueError("head_linear: shape/layout mismatch")
+    y = torch.empty((T, H, N), dtype=x.dtype, device=x.device)
+    ll = ctypes.c_longlong
+    _lib.call("b200_head_linear", ptr(x), ptr(w), ptr(y), T, H, N, K, ll(x.stride(0)), ll(x.stride(1)), ll(y.stride(0)),
+              ll(y.stride(1)), dtype_code(x.dtype), stream_ptr())
+    _count()
+    return y
+
+
+def choose_latent_splits(batch: int, rows: int, max_kv_len: int, sm_count: int = 148) -> int:
+    """Splits of the absorbed latent attention: one wave of CTAs (a CTA owns up to 32 rows and keeps most of an SM's shared
+    memory), at least two 64-token tiles each."""
+    ctas = batch * ((rows + 31) // 32)
+    return int(max(1, min(sm_count // max(ctas, 1), (max_kv_len + 127) // 128, 64)))
+
+
+def latent_attention(q: torch.Tensor, cache: torch.Tensor, kv_lens: torch.Tensor, block_table: torch.Tensor, tokens: int,
+                     scale: float, sink: torch.Tensor | None = None, num_splits: int = 1, plain: bool = False) -> torch.Tensor:
+    """Attention of absorbed queries over paged latents that are both keys and values. q [B * tokens, H, P]; cache
+    [blocks, page, P]; kv_lens int32 [B] (the new tokens included); block_table int32 [B, *]; query token i of a sequence attends
+    keys j <= kv_len - tokens + i. ``sink`` fp32 [H]. Returns [B * tokens, H, P].
+
+    16-bit ranks up to 512 take the split tensor-core kernel; fp32, wider ranks and ``plain=True`` the one-warp-per-row one."""
+    _lib.require_cuda()
+    T, H, P = q.shape
+    B = kv_lens.numel()
+    if T != B * tokens or cache.shape[-1] != P or not (q.is_contiguous() and cache.is_contiguous()) or block_table.stride(1) != 1:
+        raise ValueError("latent_attention: shape/layout mismatch")
+    if sink is not None and (sink.dtype != torch.float32 or sink.numel() != H):
+        raise ValueError("latent_attention: sink must be fp32 [H]")
+    page = cache.shape[1]
+    out = torch.empty_like(q)
+    common = (ptr(q), ptr(cache), ptr(block_table), block_table.stride(0), ptr(kv_lens), B, tokens, H, P, page, c_float(scale))
+    if plain or q.dtype == torch.float32 or P > 512 or page % 64 != 0:
+        _lib.call("b200_latent_attention_plain", *common, ptr(sink), ptr(out), dtype_code(q.dtype), stream_ptr())
+        _count()
+        return out
+    o_part = torch.empty((T * H, num_splits, P), dtype=torch.float32, device=q.device)
+    lse_part = torch.empty((T * H, num_splits), dtype=torch.float32, device=q.device)
+    _lib.call("b200_latent_attention", *common, num_splits, ptr(o_part), ptr(lse_part), dtype_code(q.dtype), stream_ptr())
+    _lib.call("b200_latent_combine", ptr(o_part), ptr(lse_part), ptr(sink), T * H, H, num_splits, P, ptr(out), dtype_code(q.dtype),
+              stream_ptr())
+    _count(2)
+    return out
+
+
+def prefill_attention_vt(q: torch.Tensor, k: torch.Tensor, vt: torch.Tensor, cu_seqlens_q: torch.Tensor, cu_seqlens_k: torch.Tensor,
+                         seqlens_k: torch.Tensor, max_seqlen_q: int, scale: float, causal: bool = True,
+                         sink: torch.Tensor | None = None) -> torch.Tensor:
+    """``prefill_attention`` for other head sizes, transposed values and an optional sink logit per head. q [total_q, Hq, dk]
+    (rows may be strided), k [total_k, Hkv, dk], vt [B, Hkv, dv, S] (keys of a sequence in its first columns), sink fp32 [Hq]
+    or None; dk <= 256, dk, dv and S multiples of 8. Returns [total_q, Hq, dv]."""
+    _lib.require_cuda()
+    total_q, Hq, dk = q.shape
+    total_k, Hkv, _ = k.shape
+    B, _, dv, s_pad = vt.shape
+    if q.stride(2) != 1 or q.stride(1) != dk or not (k.is_contiguous() and vt.is_contiguous()) or vt.shape[1] != Hkv:
+        raise ValueError("prefill_attention_vt: shape/layout mismatch")
+    out = torch.empty((total_q, Hq, dv), dtype=q.dtype, device=q.device)
+    _lib.call("b200_prefill_attention_vt", ptr(q), ctypes.c_longlong(q.stride(0)), ptr(k), ptr(vt), s_pad, ptr(cu_seqlens_q),
+              ptr(cu_seqlens_k), ptr(seqlens_k), B, total_q, total_k, int(max_seqlen_q), Hq, Hkv, dk, dv, c_float(scale),
+              1 if causal else 0, ptr(sink), ptr(out), dtype_code(q.dtype), ptr(_pipeline_status(q.device)), stream_ptr())
     _count()
     return out
