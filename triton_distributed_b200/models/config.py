@@ -130,8 +130,8 @@ ARCHS: dict[str, ArchConfig | LikosunConfig] = {
         LayerSpec(LatentAttentionSpec(8, 32, 48, 56, 0.15), None),
         LayerSpec(LatentAttentionSpec(2, 72, 136, 96, 0.1), DenseMlpSpec(200))), 1e-5, 12.0, 0.4),
     # shapes of real layers (random weights; benchmarks): a small, a middle and a large model
-    "likosun-2b": _likosun(32768, 2048, 24, 16, 128, 128, 512, 8192),
-    "likosun-8b": _likosun(65536, 4096, 32, 32, 128, 128, 512, 16384),
+    "likosun-1b": _likosun(32768, 2048, 24, 16, 128, 128, 512, 8192),
+    "likosun-7b": _likosun(65536, 4096, 32, 32, 128, 128, 512, 16384),
     "likosun-20b": _likosun(65536, 5120, 48, 64, 128, 128, 512, 25600),
 }
 

@@ -11,5 +11,7 @@ from .moe import (ag_group_gemm_ref, grouped_gemm_ref, grouped_gemm_fp8_ref, deq
                   fp8_dequant_ref, fp8_quant_ref, moe_align_block_size_ref, moe_reduce_rs_ref, select_experts_ref,
                   ag_moe_tile_schedule_ref, calc_gather_scatter_index_ref)
 from .attention import paged_decode_attention_ref, combine_partials_ref, sp_flash_decode_ref
+from .likosun import (depth_average_ref, gated_residual_ref, greedy_ref, latent_attention_ref, layer_norm_ref, likosun_layer_ref,
+                      likosun_ref, rms_norm_ref, sink_softmax_ref, squared_relu_ref)
 
 __all__ = [n for n in dir() if n.endswith("_ref")]
