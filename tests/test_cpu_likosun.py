@@ -62,8 +62,11 @@ def test_latent_cache_pages():
     assert c.layer(1).shape == (9, 64, 40) and c.blocks_per_seq == 3
     pos = torch.tensor([[0, 63], [64, 65], [128, 129]])
     c.layer(1).view(-1, 40)[c.slots(pos)] = torch.arange(6.0)[:, None].expand(6, 40)
-    assert c.rows(1, 0, 64)[:, 0].tolist() == [0.0] + [0.0] * 62 + [1.0]
-    assert c.rows(1, 1, 66)[64:, 3].tolist() == [2.0, 3.0] and c.rows(1, 2, 130)[128:, 39].tolist() == [4.0, 5.0]
+    rows = c.rows(1, 130).view(3, 130, 40)
+    assert rows[0, :64, 0].tolist() == [0.0] * 63 + [1.0]
+    assert rows[1, 64:66, 3].tolist() == [2.0, 3.0] and rows[2, 128:, 39].tolist() == [4.0, 5.0]
+    c.blank(1, 65, 129)
+    assert c.rows(1, 192).view(3, 192, 40)[:, :, 7].nonzero().tolist() == [[0, 63], [1, 64], [2, 129]]
     page = c.block_table[2, 128 // 64]
     assert c.layer(1)[page, 1, 0] == 5.0
 

@@ -135,11 +135,11 @@ def test_head_linear(dtype, T, H, N, K):
 
 
 def _paged(seqs, pitch, page, dtype, seed=0):
-    """Latents of several sequences in shuffled pages; unused slots hold large garbage that must not be read as keys."""
+    """Latents of several sequences in shuffled pages; unused slots hold NaN, which must not reach any result."""
     g = torch.Generator().manual_seed(seed)
     nb = [(s.shape[0] + page - 1) // page for s in seqs]
     perm = torch.randperm(sum(nb) + 3, generator=g)
-    cache = torch.full((sum(nb) + 3, page, pitch), 300.0)
+    cache = torch.full((sum(nb) + 3, page, pitch), torch.nan)
     table = torch.zeros(len(seqs), max(nb) + 1, dtype=torch.int32)
     used = 0
     for b, s in enumerate(seqs):
@@ -159,11 +159,13 @@ def _absorbed_ref(q, c, sink, scale, first):
     return ref.latent_attention_ref(q, c, eye, eye, sink, scale, first)
 
 
-@pytest.mark.parametrize("dtype,plain", [(torch.bfloat16, False), (torch.float16, False), (torch.bfloat16, True), (torch.float32, True)])
+@pytest.mark.parametrize("dtype,variant", [(torch.bfloat16, "tc"), (torch.float16, "tc"), (torch.bfloat16, "mma"), (torch.float16, "mma"),
+                                           (torch.bfloat16, "plain"), (torch.float32, "plain")])
 @pytest.mark.parametrize("H,S,rank,lens,splits,page", [
     (1, 1, 8, [1, 2, 63, 64, 65], 1, 64), (6, 1, 72, [300, 17, 128, 129], 3, 64), (16, 1, 512, [700, 64, 1], 5, 128),
-    (3, 2, 40, [2, 65, 66, 130], 2, 64), (5, 7, 136, [7, 8, 70, 134], 2, 192), (33, 3, 264, [200, 3], 4, 64), (4, 31, 384, [31, 95], 1, 64)])
-def test_latent_attention(dtype, plain, H, S, rank, lens, splits, page):
+    (3, 2, 40, [2, 65, 66, 130], 2, 64), (5, 7, 136, [7, 8, 70, 134], 2, 192), (33, 3, 264, [200, 3], 4, 64), (4, 31, 384, [31, 95], 1, 64),
+    (64, 1, 512, [1000, 257, 129], 3, 64), (20, 2, 200, [500, 2, 256], 2, 64), (40, 1, 448, [128, 384, 770], 6, 64)])
+def test_latent_attention(dtype, variant, H, S, rank, lens, splits, page):
     from triton_distributed_b200 import ops
     pitch = rank
     seqs = [torch.randn(n, rank).to(dtype) for n in lens]
@@ -172,20 +174,45 @@ def test_latent_attention(dtype, plain, H, S, rank, lens, splits, page):
     sink = torch.randn(H) + 2
     scale = 1.3 / rank ** 0.5
     out = ops.latent_attention(q.cuda(), cache, torch.tensor(lens, dtype=torch.int32, device="cuda"), table, S, scale, sink.cuda(),
-                               splits, plain=plain)
+                               splits, variant=variant)
     want = torch.cat([_absorbed_ref(q[b * S:(b + 1) * S].double(), seqs[b].double(), sink.double(), scale, n - S)
                       for b, n in enumerate(lens)])
     _close(out, want, dtype, factor=2.0)
     no_sink = ops.latent_attention(q.cuda(), cache, torch.tensor(lens, dtype=torch.int32, device="cuda"), table, S, scale, None,
-                                   splits, plain=plain)
+                                   splits, variant=variant)
     want0 = torch.cat([_absorbed_ref(q[b * S:(b + 1) * S].double(), seqs[b].double(), torch.full((H,), -1e30, dtype=torch.float64),
                                      scale, n - S) for b, n in enumerate(lens)])
     _close(no_sink, want0, dtype, factor=2.0)
+    if variant == "tc":
+        for rows in (16, 32, 64):
+            other = ops.latent_attention(q.cuda(), cache, torch.tensor(lens, dtype=torch.int32, device="cuda"), table, S, scale,
+                                         sink.cuda(), 1, rows_per_cta=rows, variant="tc")
+            _close(other, want, dtype, factor=2.0)
+    ops.check_pipeline_status()
 
 
-@pytest.mark.parametrize("plain", [False, True])
+def test_latent_attention_with_scores_that_grow():
+    """Scores that rise tile after tile make the running maximum move again and again, for each row at its own pace."""
+    from triton_distributed_b200 import ops
+    H, rank, n = 20, 128, 1500
+    c = torch.randn(n, rank) * 0.3
+    c[:, 0] = torch.linspace(-40, 60, n)
+    q = torch.randn(1, H, rank) * 0.3
+    q[0, :, 0] = torch.linspace(-1.5, 1.5, H)
+    c, q = c.bfloat16(), q.bfloat16()
+    cache, table = _paged([c], rank, 64, torch.bfloat16)
+    want = _absorbed_ref(q.double(), c.double(), torch.zeros(H, dtype=torch.float64), 1.0, n - 1)
+    for variant in ("tc", "mma", "plain"):
+        for splits in (1, 3):
+            out = ops.latent_attention(q.cuda(), cache, torch.tensor([n], dtype=torch.int32, device="cuda"), table, 1, 1.0,
+                                       torch.zeros(H, device="cuda"), splits, variant=variant)
+            _close(out, want, torch.bfloat16, factor=2.0)
+    ops.check_pipeline_status()
+
+
+@pytest.mark.parametrize("variant", ["tc", "mma", "plain"])
 @pytest.mark.parametrize("kv_len,S", [(1, 1), (64, 1), (65, 1), (128, 5), (190, 3), (321, 1)])
-def test_latent_attention_sees_exactly_the_keys_up_to_its_own(plain, kv_len, S):
+def test_latent_attention_sees_exactly_the_keys_up_to_its_own(variant, kv_len, S):
     """One key at a time gets a score that dwarfs the others: rows whose position is at or after it return its latent, rows
     before it must not notice it. Places: first key, page and tile borders, the tokens of the step themselves."""
     from triton_distributed_b200 import ops
@@ -200,7 +227,7 @@ def test_latent_attention_sees_exactly_the_keys_up_to_its_own(plain, kv_len, S):
         c[j, 0] = 8.0                                    # score 64 against about 0.4
         cache, table = _paged([c.to(torch.bfloat16)], rank, 64, torch.bfloat16, seed=j)
         out = ops.latent_attention(q.to(torch.bfloat16).cuda(), cache, torch.tensor([kv_len], dtype=torch.int32, device="cuda"), table,
-                                   S, 1.0, torch.zeros(H, device="cuda"), 3, plain=plain).float().cpu()
+                                   S, 1.0, torch.zeros(H, device="cuda"), 3, variant=variant).float().cpu()
         want = c.to(torch.bfloat16).float()[j]
         for i in range(S):
             seen = kv_len - S + i >= j
@@ -221,17 +248,17 @@ def test_prefill_attention_vt(dtype, H, dk, dv, q_lens, prefix, sink_on):
     wide = torch.randn(total, H * dk + 16).to(dtype)
     q = wide.cuda()[:, 8:8 + H * dk].unflatten(1, (H, dk))
     k = torch.full((B, kv8, H, dk), 100.0)               # slots beyond a sequence hold garbage
-    vt = torch.full((B, H, dv, kv8), 100.0)
+    vt = torch.full((H, dv, B, kv8), 100.0)
     ks, vs = [], []
     for b, n in enumerate(k_lens):
         kb, vb = torch.randn(n, H, dk).to(dtype), torch.randn(n, H, dv).to(dtype)
-        k[b, :n], vt[b, :, :, :n] = kb.float(), vb.permute(1, 2, 0).float()
+        k[b, :n], vt[:, :, b, :n] = kb.float(), vb.permute(1, 2, 0).float()
         ks.append(kb), vs.append(vb)
     sink = (torch.randn(H) + 3) if sink_on else None
     scale = 2.0 / dk ** 0.5
     cu_q = torch.tensor([0] + list(torch.tensor(q_lens).cumsum(0)), dtype=torch.int32, device="cuda")
     cu_k = torch.arange(B + 1, dtype=torch.int32, device="cuda") * kv8
-    out = ops.prefill_attention_vt(q, k.to(dtype).cuda().view(B * kv8, H, dk), vt.to(dtype).cuda(), cu_q, cu_k,
+    out = ops.prefill_attention_vt(q, k.to(dtype).cuda().view(B * kv8, H, dk), vt.to(dtype).cuda().view(H, dv, B * kv8), cu_q, cu_k,
                                    torch.tensor(k_lens, dtype=torch.int32, device="cuda"), max(q_lens), scale, True,
                                    sink.cuda() if sink_on else None)
     ops.check_pipeline_status()
@@ -259,7 +286,7 @@ def test_prefill_attention_sees_exactly_the_keys_up_to_its_own():
         k[:, :, 0] = 0.0
         k[j, :, 0] = 8.0
         v[j] = 1.0
-        out = ops.prefill_attention_vt(q.bfloat16().cuda(), k.bfloat16().cuda(), v.permute(1, 2, 0)[None].contiguous().bfloat16().cuda(),
+        out = ops.prefill_attention_vt(q.bfloat16().cuda(), k.bfloat16().cuda(), v.permute(1, 2, 0).contiguous().bfloat16().cuda(),
                                        torch.tensor([0, S], dtype=torch.int32, device="cuda"),
                                        torch.tensor([0, kv8], dtype=torch.int32, device="cuda"),
                                        torch.tensor([n], dtype=torch.int32, device="cuda"), S, 1.0, True, torch.zeros(H, device="cuda"))

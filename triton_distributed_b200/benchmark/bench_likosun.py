@@ -117,8 +117,8 @@ def kernels(name: str, batch: int = 8, prompt: int = 2048) -> list[dict]:
         pages = batch * kv // 64
         table = torch.arange(pages, dtype=torch.int32, device=dev).view(batch, -1)
         cache, qc, sink = rnd(pages, 64, r), rnd(batch, H, r), torch.zeros(H, device=dev)
-        splits = ops.choose_latent_splits(batch, H, kv)
-        new = _row(f"latent attention + combine, kv {kv}", lambda: ops.latent_attention(qc, cache, lens, table, 1, 0.1, sink, splits),
+        splits, rows = ops.choose_latent_splits(batch, H, kv)
+        new = _row(f"latent attention + combine, kv {kv}", lambda: ops.latent_attention(qc, cache, lens, table, 1, 0.1, sink, splits, rows),
                    2.0 * batch * kv * r, 4.0 * batch * H * kv * r)
         kc, vc, qq = rnd(pages, 64, Hkv, 128), rnd(pages, 64, Hkv, 128), rnd(batch, H, 128)
         ws: dict = {}
@@ -158,14 +158,15 @@ def kernels(name: str, batch: int = 8, prompt: int = 2048) -> list[dict]:
         new = _row(f"embed_norm, {T} tokens", lambda: ops.embed_norm(ids, tab, 2.0, W, g, b, 1e-6, True, state0=st0), T * W * 12.0)
         pair(new, _row(f"embedding, {T} tokens", lambda: ops.embedding(ids, tab), 4.0 * T * W))
     S, B = prompt, batch                                                              # ---- prompts
-    c, uk, uv = rnd(S, r), rnd(H * d, r), rnd(H * v, r)
-    xp = rnd(S, W)
+    R = B * S
+    c, uk, uv = rnd(R, r), rnd(H * d, r), rnd(H * v, r)
+    xp = rnd(R, W)
     w_like = rnd(H * 128, W)
-    like = _row(f"gemm {S} x {H * 128} x {W}", lambda: ops.linear(xp, w_like),
-                2.0 * (S * W + S * H * 128 + H * 128 * W), 2.0 * S * H * 128 * W)
-    pair(_row(f"expand keys: gemm {S} x {H * d} x {r}", lambda: ops.linear(c, uk), 2.0 * (S * r + H * d * r + S * H * d), 2.0 * S * H * d * r), like)
-    pair(_row(f"expand values: gemm {H * v} x {S} x {r}", lambda: ops.linear(uv, c), 2.0 * (S * r + H * v * r + S * H * v), 2.0 * S * H * v * r), like)
-    qp, kp, vt = rnd(B * S, H, d), rnd(B * S, H, d), rnd(B, H, v, S)
+    like = _row(f"gemm {R} x {H * 128} x {W}", lambda: ops.linear(xp, w_like),
+                2.0 * (R * W + R * H * 128 + H * 128 * W), 2.0 * R * H * 128 * W)
+    pair(_row(f"expand keys: gemm {R} x {H * d} x {r}", lambda: ops.linear(c, uk), 2.0 * (R * r + H * d * r + R * H * d), 2.0 * R * H * d * r), like)
+    pair(_row(f"expand values: gemm {H * v} x {R} x {r}", lambda: ops.linear(uv, c), 2.0 * (R * r + H * v * r + R * H * v), 2.0 * R * H * v * r), like)
+    qp, kp, vt = rnd(B * S, H, d), rnd(B * S, H, d), rnd(H, v, B * S)
     cu = torch.arange(0, (B + 1) * S, S, dtype=torch.int32, device=dev)
     lens = torch.full((B,), S, dtype=torch.int32, device=dev)
     sink = torch.zeros(H, device=dev)

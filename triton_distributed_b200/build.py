@@ -37,7 +37,7 @@ SERVING_LIB_PATH = LIB_DIR / "libb200dist_serving.so"
 
 # sources of the single-GPU serving subset: no heap, no collectives, no expert kernels
 SERVING_SOURCES = ("runtime/host.cc", "kernels/decode_attn.cu", "kernels/elementwise.cu", "kernels/gemm_f32.cu",
-                   "kernels/gemm_skinny_sm100.cu", "kernels/gemm_sm100.cu", "kernels/latent_attn.cu",
+                   "kernels/gemm_skinny_sm100.cu", "kernels/gemm_sm100.cu", "kernels/latent_attn.cu", "kernels/latent_decode_sm100.cu",
                    "kernels/prefill_attn_sm100.cu", "kernels/residual.cu", "kernels/sampling.cu")
 
 NVCC_FLAGS = [

@@ -1,0 +1,411 @@
+// Absorbed latent attention for sm_100a on the tensor cores: one cached row per token is key and value of all heads.
+//
+// The roles of the operands are swapped so that the few query rows (query token x head, N of them) are the narrow side of
+// every tcgen05.mma and no tensor-core row is padding:
+//   scores   S^T [128 keys, N]  = C [128 keys, rank] . Q [N, rank]^T        (C and Q K-major)
+//   values   O^T [rank, N]     += C^T [rank, 128 keys] . P [N, 128 keys]^T  (C^T is the same shared-memory tile read MN-major)
+// so a latent row is loaded once and used twice, and the running output stays in tensor memory: lane = column of the latent
+// (in chunks of 128), column = query row.
+//
+// One CTA owns N query rows of a sequence and a range of 128-key tiles (split-KV; latent_combine merges, and adds the sink):
+//   warp 0     TMA producer: the Q tile once, then the tiles in slots of 128 keys x 128 columns (two 64-column swizzle atoms)
+//   warp 1     MMA issuer; a slot is given back as soon as its chunk of the output has been accumulated, so the next tile
+//              streams in while the rest of this one is still being multiplied
+//   warps 4-7  softmax, one thread per key of the tile: column maxima by warp-wide redux + shared memory, exponentials, P as
+//              16-bit into a swizzled tile. The reference maximum of a row only moves when it is exceeded by more than 2^8, so
+//              the output in tensor memory is rescaled a few times per sequence at most; sums and output use the same reference,
+//              which cancels in the end.
+// Every barrier wait is bounded; on expiry the CTA unwinds through an abort flag and reports a status.
+#include "b200/host.h"
+#include "b200/primitives.cuh"
+#include "b200/tcgen05.cuh"
+
+#include <cstring>
+
+namespace b200 {
+
+constexpr int kLdKeys = 128;              // keys per tile
+constexpr int kLdAtom = kLdKeys * 128;    // 128 keys x 64 columns: 16 KB
+constexpr int kLdSlot = 2 * kLdAtom;      // 128 keys x 128 columns
+constexpr int kLdThreads = 256;
+constexpr float kLdSlack = 8.f;           // how far (log2) a score may exceed the reference before it moves
+constexpr int kLdSmemMax = 226 * 1024;
+
+constexpr int ld_fixed_bytes(int n, int rk) { return (rk / 64 + 2) * n * 128 + 1024 + 512 + n * 44; }
+constexpr int ld_slots(int n, int rk) {
+  const int fit = (kLdSmemMax - ld_fixed_bytes(n, rk)) / kLdSlot, want = 2 * (rk / 128) + 1;
+  return fit < want ? fit : want;
+}
+constexpr int ld_smem_bytes(int n, int rk) { return ld_fixed_bytes(n, rk) + ld_slots(n, rk) * kLdSlot; }
+
+struct LatentDecodeParams {
+  const int* block_table;  // [B, bt_stride]
+  const int* kv_lens;      // [B]
+  float* o_part;           // [B * S * H, splits, pitch]
+  float* lse_part;         // [B * S * H, splits]
+  int bt_stride, page, H, S, pitch, splits, bf16;
+  float scale_log2e;       // positive
+  uint32_t* status;
+};
+
+// MN-major operand in 128-byte-swizzled atoms of 64 (MN) x 8 (K): 8-row K groups 1024 bytes apart, the next 64 MN elements
+// `mn_stride` bytes away
+__device__ __forceinline__ uint64_t umma_desc_sw128_mnmajor(uint32_t smem_addr, uint32_t mn_stride) {
+  uint64_t d = umma_desc_sw128_kmajor(smem_addr);
+  d &= ~(static_cast<uint64_t>(0x3FFF) << 16);
+  d |= static_cast<uint64_t>(mn_stride >> 4) << 16;
+  return d;
+}
+__device__ __forceinline__ float redux_max(float v) {
+  float r;
+  asm volatile("redux.sync.max.f32 %0, %1, 0xffffffff;" : "=f"(r) : "f"(v));
+  return r;
+}
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void tmem_st_32x16(uint32_t taddr, const uint32_t (&r)[16]) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], "
+      "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};" ::"r"(taddr),
+      "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]),
+      "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
+      : "memory");
+}
+__device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+__device__ __forceinline__ void ld_softmax_bar() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+
+// N: query rows per CTA (16, 32 or 64); RK: rank rounded up to a multiple of 128 (TMA fills the padding columns with zeros)
+template <int N, int RK>
+__global__ void __launch_bounds__(kLdThreads, 1)
+latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant__ CUtensorMap tmQ, const LatentDecodeParams p) {
+  constexpr int kPairs = RK / 128, kSlots = ld_slots(N, RK), kRowAtom = N * 128;
+  static_assert(kSlots >= kPairs && kSlots <= 16, "a tile must fit in the ring, the ring in the barrier layout");
+  constexpr uint32_t kTmemNeed = N * (1 + kPairs);
+  constexpr uint32_t kTmemCols = kTmemNeed <= 32 ? 32 : kTmemNeed <= 64 ? 64 : kTmemNeed <= 128 ? 128 : kTmemNeed <= 256 ? 256 : 512;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* ring = smem;                             // [kSlots][2 atoms][128 keys][128 B]
+  uint8_t* sQ = ring + kSlots * kLdSlot;            // [RK / 64 atoms][N rows][128 B]
+  uint8_t* sP = sQ + (RK / 64) * kRowAtom;          // [2 atoms][N rows][128 B], columns = keys
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + 2 * kRowAtom);
+  uint64_t* full = bars;                // [kSlots]
+  uint64_t* empty = bars + 16;          // [kSlots]
+  uint64_t* q_full = bars + 32;
+  uint64_t* s_full = bars + 33;
+  uint64_t* p_full = bars + 34;
+  uint64_t* o_full = bars + 35;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 36);
+  volatile uint32_t* abort_flag = tmem_slot + 1;
+  volatile int* moved = reinterpret_cast<volatile int*>(tmem_slot + 2);  // last tile at which a reference maximum moved
+  float* xmax = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(bars) + 512);  // [4 warps][N]
+  float* mref = xmax + 4 * N;                                                      // [N]
+  float* corr = mref + N;                                                          // [N]; at the end 1 / row sum
+  float* xsum = corr + N;                                                          // [4][N]
+  int* limit = reinterpret_cast<int*>(xsum + 4 * N);                               // [N] last key a row attends
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int split = blockIdx.x, r0 = blockIdx.y * N, b = blockIdx.z;
+  const int n_rows = p.S * p.H;
+  const uint64_t timeout_ns = 4000000000ull;
+  griddep_launch_dependents();
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < kSlots; ++i) {
+      mbar_init(full + i, 1);
+      mbar_init(empty + i, 1);
+    }
+    mbar_init(q_full, 1);
+    mbar_init(s_full, 1);
+    mbar_init(p_full, 4);
+    mbar_init(o_full, 1);
+    *abort_flag = 0;
+    *moved = -1;
+    mbar_fence_init();
+    tma_prefetch_desc(&tmC);
+    tma_prefetch_desc(&tmQ);
+  }
+  if (warp == 2) tmem_alloc(tmem_slot, kTmemCols);
+  griddep_wait();
+  const int kv_len = p.kv_lens[b];
+  const int first_limit = kv_len - p.S;  // last key of token 0; token i adds i
+  const int n_keys = max(0, min(kv_len, first_limit + (min(r0 + N, n_rows) - 1) / p.H + 1));
+  const int n_tiles = (n_keys + kLdKeys - 1) / kLdKeys;
+  const int per = (n_tiles + p.splits - 1) / p.splits;
+  const int tile0 = min(n_tiles, split * per), tile1 = min(n_tiles, tile0 + per);
+  const int row_base = b * n_rows + r0;
+  for (int n = threadIdx.x; n < N; n += kLdThreads) {
+    limit[n] = r0 + n < n_rows ? first_limit + (r0 + n) / p.H : -1;
+    mref[n] = -INFINITY;
+    corr[n] = 1.f;
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem_base = *tmem_slot;  // columns [0, N) S^T, then kPairs x N columns of O^T
+
+  if (warp == 0) {
+    if (elect_one() && tile0 < tile1) {
+      fence_proxy_async();  // queries and latents were written by earlier kernels through the generic proxy
+      mbar_expect_tx(q_full, (RK / 64) * kRowAtom);
+      for (int a = 0; a < RK / 64; ++a) tma_load_2d(sQ + a * kRowAtom, &tmQ, q_full, a * 64, row_base);
+      const int* table = p.block_table + static_cast<size_t>(b) * p.bt_stride;
+      int it = 0;
+      bool ok = true;
+      for (int tile = tile0; tile < tile1 && ok; ++tile) {
+        int row[2];
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {  // 64 keys lie in one page; a half beyond the last key repeats the first
+          int key = tile * kLdKeys + 64 * half;
+          if (key >= n_keys) key = tile * kLdKeys;
+          row[half] = table[key / p.page] * p.page + key % p.page;
+        }
+        for (int pr = 0; pr < kPairs && ok; ++pr, ++it) {
+          const int slot = it % kSlots;
+          ok = mbar_wait(empty + slot, ((it / kSlots) & 1) ^ 1, abort_flag, timeout_ns);
+          if (!ok) break;
+          mbar_expect_tx(full + slot, kLdSlot);
+#pragma unroll
+          for (int a = 0; a < 2; ++a)
+#pragma unroll
+            for (int half = 0; half < 2; ++half)
+              tma_load_2d(ring + slot * kLdSlot + a * kLdAtom + half * (kLdAtom / 2), &tmC, full + slot, pr * 128 + a * 64, row[half]);
+        }
+      }
+    }
+    __syncwarp();
+  } else if (warp == 1) {
+    if (elect_one() && tile0 < tile1) {
+      const uint32_t idesc_s = umma_idesc_f16(128, N, p.bf16 != 0);
+      const uint32_t idesc_o = idesc_s | (1u << 15);  // A is MN-major
+      bool ok = mbar_wait(q_full, 0, abort_flag, timeout_ns);
+      int it = 0;
+      for (int tile = tile0; tile < tile1 && ok; ++tile, it += kPairs) {
+        for (int pr = 0; pr < kPairs && ok; ++pr) {
+          const int slot = (it + pr) % kSlots;
+          ok = mbar_wait(full + slot, ((it + pr) / kSlots) & 1, abort_flag, timeout_ns);
+          if (!ok) break;
+          tc_fence_after_sync();
+#pragma unroll
+          for (int kk = 0; kk < 8; ++kk) {
+            const uint64_t da = umma_desc_sw128_kmajor(smem_u32(ring + slot * kLdSlot + (kk >> 2) * kLdAtom)) + 2 * (kk & 3);
+            const uint64_t db = umma_desc_sw128_kmajor(smem_u32(sQ + (2 * pr + (kk >> 2)) * kRowAtom)) + 2 * (kk & 3);
+            umma_f16(tmem_base, da, db, idesc_s, (pr | kk) != 0 ? 1u : 0u);
+          }
+        }
+        if (!ok) break;
+        umma_commit(s_full);  // also: every product of the tile before has been accumulated
+        ok = mbar_wait(p_full, (tile - tile0) & 1, abort_flag, timeout_ns);
+        if (!ok) break;
+        tc_fence_after_sync();
+        for (int pr = 0; pr < kPairs; ++pr) {
+          const int slot = (it + pr) % kSlots;
+#pragma unroll
+          for (int kk = 0; kk < kLdKeys / 16; ++kk) {
+            const uint64_t da = umma_desc_sw128_mnmajor(smem_u32(ring + slot * kLdSlot + kk * 16 * 128), kLdAtom);
+            const uint64_t db = umma_desc_sw128_kmajor(smem_u32(sP + (kk >> 2) * kRowAtom)) + 2 * (kk & 3);
+            umma_f16(tmem_base + N * (1 + pr), da, db, idesc_o, (tile != tile0 || kk != 0) ? 1u : 0u);
+          }
+          umma_commit(empty + slot);
+        }
+      }
+      if (ok) umma_commit(o_full);
+    }
+    __syncwarp();
+  } else if (warp >= 4) {
+    const int w4 = warp & 3, t = threadIdx.x - 128;  // t: key of the tile = TMEM lane
+    const uint32_t lane_base = tmem_base + (static_cast<uint32_t>(w4 * 32) << 16);
+    float l[N];  // this key's share of every row sum
+#pragma unroll
+    for (int n = 0; n < N; ++n) l[n] = 0.f;
+    const int all_below = r0 + N <= n_rows ? first_limit + r0 / p.H : -1;  // keys up to here are visible to all rows
+    uint8_t* p_col = sP + (t >> 6) * kRowAtom + (t & 7) * 2;
+    const int p_chunk = (t & 63) >> 3;
+    bool ok = true;
+    int it = 0;
+    // every thread meets the barriers of every tile, also after a pipeline wait has failed
+    for (int tile = tile0; tile < tile1; ++tile, it += kPairs) {
+      if (ok) ok = mbar_wait(s_full, (tile - tile0) & 1, abort_flag, timeout_ns);
+      ok = __all_sync(0xffffffffu, ok);
+      tc_fence_after_sync();
+      const int key = tile * kLdKeys + t;
+      const bool masked = tile * kLdKeys + kLdKeys - 1 > all_below;
+      if (ok) {
+#pragma unroll
+        for (int c = 0; c < N / 16; ++c) {
+          uint32_t r[16];
+          tmem_ld_32x16(lane_base + c * 16, r);
+          tmem_ld_wait();
+          float mine = 0.f;
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            float v = __uint_as_float(r[i]);
+            if (masked) v = key <= limit[c * 16 + i] ? v : -INFINITY;
+            const float m = redux_max(v);
+            mine = lane == i ? m : mine;
+          }
+          if (lane < 16) xmax[w4 * N + c * 16 + lane] = mine;
+        }
+      }
+      ld_softmax_bar();
+      if (t < N) {
+        const float mx = fmaxf(fmaxf(xmax[t], xmax[N + t]), fmaxf(xmax[2 * N + t], xmax[3 * N + t])) * p.scale_log2e;
+        const float old = mref[t];
+        if (mx > old + kLdSlack) {  // (always when the row has no reference yet and sees a key)
+          corr[t] = ex2(old - mx);
+          mref[t] = mx;
+          *moved = tile;
+        } else {
+          corr[t] = 1.f;
+        }
+      }
+      ld_softmax_bar();
+      if (!ok) continue;
+      if (*moved == tile && tile != tile0) {
+#pragma unroll
+        for (int n = 0; n < N; ++n) l[n] *= corr[n];
+#pragma unroll 1
+        for (int c = 0; c < kPairs * (N / 16); ++c) {
+          uint32_t r[16];
+          const uint32_t at = lane_base + N + c * 16;
+          tmem_ld_32x16(at, r);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 16; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * corr[(c % (N / 16)) * 16 + i]);
+          tmem_st_32x16(at, r);
+        }
+        tmem_st_wait();
+      }
+#pragma unroll
+      for (int c = 0; c < N / 16; ++c) {
+        uint32_t r[16];
+        tmem_ld_32x16(lane_base + c * 16, r);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const int n = c * 16 + i;
+          float pr = ex2(fmaf(__uint_as_float(r[i]), p.scale_log2e, -mref[n]));
+          if (masked) pr = key <= limit[n] ? pr : 0.f;
+          l[n] += pr;
+          const uint16_t h = p.bf16 ? __bfloat16_as_ushort(__float2bfloat16(pr)) : __half_as_ushort(__float2half(pr));
+          *reinterpret_cast<uint16_t*>(p_col + n * 128 + ((p_chunk ^ (n & 7)) << 4)) = h;
+        }
+      }
+      if (key >= n_keys) {  // slots beyond the sequence may hold anything: their weight is zero, make the value zero too
+        for (int pr = 0; pr < kPairs; ++pr)
+          for (int a = 0; a < 2; ++a) {
+            uint4* dst = reinterpret_cast<uint4*>(ring + ((it + pr) % kSlots) * kLdSlot + a * kLdAtom + t * 128);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) dst[i] = make_uint4(0, 0, 0, 0);
+          }
+      }
+      tc_fence_before_sync();     // this thread's TMEM accesses are done
+      fence_view_async_shared();  // its shared-memory writes are visible to the tensor core
+      __syncwarp();
+      if (lane == 0) mbar_arrive(p_full);
+    }
+    // ---- row sums over the keys, then the normalised partial output and its log-sum-exp
+#pragma unroll
+    for (int c = 0; c < N / 16; ++c) {
+      float mine = 0.f;
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        const float s = warp_sum(l[c * 16 + i]);
+        mine = lane == i ? s : mine;
+      }
+      if (lane < 16) xsum[w4 * N + c * 16 + lane] = mine;
+    }
+    ld_softmax_bar();
+    if (t < N) {
+      const float s = (xsum[t] + xsum[N + t]) + (xsum[2 * N + t] + xsum[3 * N + t]);
+      corr[t] = s > 0.f ? 1.f / s : 0.f;
+      if (r0 + t < n_rows)
+        p.lse_part[static_cast<size_t>(row_base + t) * p.splits + split] =
+            s > 0.f ? (mref[t] + log2f(s)) * 0.6931471805599453f : -INFINITY;
+    }
+    ld_softmax_bar();
+    if (tile0 < tile1) {
+      if (ok) ok = mbar_wait(o_full, 0, abort_flag, timeout_ns);
+      ok = __all_sync(0xffffffffu, ok);
+      tc_fence_after_sync();
+      if (ok) {
+#pragma unroll 1
+        for (int pr = 0; pr < kPairs; ++pr) {
+          const int col = pr * 128 + t;
+#pragma unroll
+          for (int c = 0; c < N / 16; ++c) {
+            uint32_t r[16];
+            tmem_ld_32x16(lane_base + N * (1 + pr) + c * 16, r);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 16; ++i) {
+              const int n = c * 16 + i;
+              if (r0 + n < n_rows && col < p.pitch)
+                p.o_part[(static_cast<size_t>(row_base + n) * p.splits + split) * p.pitch + col] = __uint_as_float(r[i]) * corr[n];
+            }
+          }
+        }
+      }
+    }
+  }
+
+  tc_fence_before_sync();
+  __syncthreads();
+  if (warp == 2) tmem_dealloc(tmem_base, kTmemCols);
+  if (threadIdx.x == 0 && *abort_flag != 0u && p.status != nullptr) atomicMax(p.status, static_cast<uint32_t>(kStatusPipeTimeout));
+}
+
+template <int N, int RK>
+static int launch_latent_decode(const CUtensorMap& tc, const CUtensorMap& tq, const LatentDecodeParams& p, int B, cudaStream_t s) {
+  static bool configured[64] = {false};
+  int dev = 0;
+  B200_CHECK_CUDA(cudaGetDevice(&dev));
+  if (!configured[dev & 63]) {
+    B200_CHECK_CUDA(cudaFuncSetAttribute(latent_decode_kernel<N, RK>, cudaFuncAttributeMaxDynamicSharedMemorySize, ld_smem_bytes(N, RK)));
+    configured[dev & 63] = true;
+  }
+  const dim3 grid(p.splits, (p.S * p.H + N - 1) / N, B);
+  B200_CHECK_CUDA(launch_pdl(latent_decode_kernel<N, RK>, grid, dim3(kLdThreads), ld_smem_bytes(N, RK), s, tc, tq, p));
+  return kOk;
+}
+template <int N>
+static int launch_latent_decode_rank(const CUtensorMap& tc, const CUtensorMap& tq, const LatentDecodeParams& p, int B, cudaStream_t s) {
+  if (p.pitch <= 128) return launch_latent_decode<N, 128>(tc, tq, p, B, s);
+  if (p.pitch <= 256) return launch_latent_decode<N, 256>(tc, tq, p, B, s);
+  if (p.pitch <= 384) return launch_latent_decode<N, 384>(tc, tq, p, B, s);
+  return launch_latent_decode<N, 512>(tc, tq, p, B, s);
+}
+
+}  // namespace b200
+
+using namespace b200;
+
+// q [B * S * H, pitch]; cache [num_slots, pitch] in pages of `page` slots (a multiple of 64); partial results as in
+// b200_latent_combine. rows_per_cta: 16, 32 or 64.
+B200_API int b200_latent_decode(const void* q, const void* cache, long long num_slots, const int* block_table, int bt_stride,
+                                const int* kv_lens, int B, int S, int H, int pitch, int page, float scale, int splits,
+                                int rows_per_cta, float* o_part, float* lse_part, int dtype, uint32_t* status, void* stream) {
+  B200_REQUIRE(dtype == kBF16 || dtype == kF16, "latent decode attention supports bf16 / f16");
+  B200_REQUIRE(rows_per_cta == 16 || rows_per_cta == 32 || rows_per_cta == 64, "rows_per_cta must be 16, 32 or 64, got %d", rows_per_cta);
+  B200_REQUIRE(B >= 1 && S >= 1 && H >= 1 && B <= 65535 && num_slots >= 64, "bad latent attention shape");
+  B200_REQUIRE(pitch >= 8 && pitch % 8 == 0 && pitch <= 512, "the latent row (%d elements) must be a multiple of 8 and at most 512", pitch);
+  B200_REQUIRE(page >= 64 && page % 64 == 0, "the page size (%d) must be a multiple of 64", page);
+  B200_REQUIRE(scale > 0.f, "the score scale must be positive");
+  B200_REQUIRE(splits >= 1 && o_part && lse_part, "latent attention needs its partial buffers");
+  B200_REQUIRE((S * H + rows_per_cta - 1) / rows_per_cta <= 65535, "too many query rows (%d)", S * H);
+  CUtensorMap tc, tq;
+  int rc = make_tma_2d(&tc, cache, dtype, num_slots, pitch, pitch, 64, 64, true);
+  if (rc != kOk) return rc;
+  rc = make_tma_2d(&tq, q, dtype, static_cast<uint64_t>(B) * S * H, pitch, pitch, rows_per_cta, 64, true);
+  if (rc != kOk) return rc;
+  LatentDecodeParams p;
+  memset(&p, 0, sizeof(p));
+  p.block_table = block_table; p.kv_lens = kv_lens; p.o_part = o_part; p.lse_part = lse_part; p.bt_stride = bt_stride; p.page = page;
+  p.H = H; p.S = S; p.pitch = pitch; p.splits = splits; p.bf16 = dtype == kBF16; p.scale_log2e = scale * 1.4426950408889634f;
+  p.status = status;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (rows_per_cta == 16) return launch_latent_decode_rank<16>(tc, tq, p, B, s);
+  if (rows_per_cta == 32) return launch_latent_decode_rank<32>(tc, tq, p, B, s);
+  return launch_latent_decode_rank<64>(tc, tq, p, B, s);
+}

@@ -44,6 +44,7 @@ struct PrefillParams {
   int Hq, Hkv, causal, bf16;
   int dk, dv;           // query / key and value sizes of a head
   int v_chunks;         // ceil(dv / 128): CTAs per (query block, head)
+  int v_packed;         // V^T is [Hkv, dv, total_k], a sequence's keys at columns cu_k[b] ...; else [B * Hkv, dv, s_pad]
   const float* sink;    // nullable [Hq]
   const int* cu_q;      // [B + 1] first packed query row of every sequence
   const int* cu_k;      // [B + 1] first key row of every sequence (only [0, B) is read when k_lens is given)
@@ -153,6 +154,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   if (warp == 0) {
     // ------------------------------------------------------------------ TMA producer
     if (elect_one() && n_steps > 0) {  // nothing may be in flight into shared memory when nobody will wait for it
+      const int v_key0 = p.v_packed ? k_start : 0, v_row = p.v_packed ? kvh : b * p.Hkv + kvh;
       mbar_expect_tx(q_full, kQkTile);
 #pragma unroll
       for (int a = 0; a < kDkAtoms; ++a) tma_load_3d(sQ + a * kPAtom, &tmQ, q_full, 64 * a, h, q_start + m_blk * kPM);
@@ -165,8 +167,8 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           tma_load_3d(sK + ks * kQkTile + a * kPAtom, &tmK, k_full + ks, 64 * a, kvh, k_start + j * kPN);
         if (!mbar_wait(v_empty + vs, ((j / kVSt) & 1) ^ 1, abort_flag, timeout_ns)) break;
         mbar_expect_tx(v_full + vs, kPTile);
-        tma_load_3d(sV + vs * kPTile, &tmVt, v_full + vs, j * kPN, v_col0, b * p.Hkv + kvh);
-        tma_load_3d(sV + vs * kPTile + kPAtom, &tmVt, v_full + vs, j * kPN + 64, v_col0, b * p.Hkv + kvh);
+        tma_load_3d(sV + vs * kPTile, &tmVt, v_full + vs, v_key0 + j * kPN, v_col0, v_row);
+        tma_load_3d(sV + vs * kPTile + kPAtom, &tmVt, v_full + vs, v_key0 + j * kPN + 64, v_col0, v_row);
       }
     }
     __syncwarp();
@@ -369,20 +371,21 @@ static int launch_prefill_atoms(const CUtensorMap& tq, const CUtensorMap& tk, co
   return kOk;
 }
 
-static int prefill_launch(const void* q, int64_t ldq, const void* k, const void* vt, int s_pad, const int* cu_q, const int* cu_k,
-                          const int* k_lens, int B, int total_q, int total_k, int max_q, int Hq, int Hkv, int dk, int dv, float scale,
+static int prefill_launch(const void* q, int64_t ldq, const void* k, const void* vt, int s_pad, int v_packed, const int* cu_q,
+                          const int* cu_k, const int* k_lens, int B, int total_q, int total_k, int max_q, int Hq, int Hkv, int dk, int dv, float scale,
                           int causal, const float* sink, void* out, int dtype, uint32_t* status, cudaStream_t s) {
   CUtensorMap tq, tk, tv;
   int rc = make_tma_3d(&tq, q, dtype, dk, Hq, total_q, dk, static_cast<uint64_t>(ldq), 64, 1, kPM, true);
   if (rc != kOk) return rc;
   rc = make_tma_3d(&tk, k, dtype, dk, Hkv, total_k, dk, static_cast<uint64_t>(Hkv) * dk, 64, 1, kPN, true);
   if (rc != kOk) return rc;
-  rc = make_tma_3d(&tv, vt, dtype, s_pad, dv, static_cast<uint64_t>(B) * Hkv, s_pad, static_cast<uint64_t>(dv) * s_pad, 64, kPD, 1, true);
+  rc = make_tma_3d(&tv, vt, dtype, s_pad, dv, static_cast<uint64_t>(v_packed ? 1 : B) * Hkv, s_pad, static_cast<uint64_t>(dv) * s_pad, 64,
+                   kPD, 1, true);
   if (rc != kOk) return rc;
   PrefillParams p;
   memset(&p, 0, sizeof(p));
   p.Hq = Hq; p.Hkv = Hkv; p.causal = causal; p.bf16 = dtype == kBF16;
-  p.dk = dk; p.dv = dv; p.v_chunks = (dv + kPD - 1) / kPD; p.sink = sink;
+  p.dk = dk; p.dv = dv; p.v_chunks = (dv + kPD - 1) / kPD; p.v_packed = v_packed; p.sink = sink;
   p.cu_q = cu_q; p.cu_k = cu_k; p.k_lens = k_lens;
   p.scale_log2e = scale * 1.4426950408889634f;
   p.out = out; p.status = status;
@@ -428,24 +431,25 @@ B200_API int b200_prefill_attention(const void* q, const void* k, const void* v,
   transpose_v_kernel<<<dim3(s_pad / 32, kPD / 32, B * Hkv), 256, 0, s>>>(static_cast<const uint16_t*>(v),
                                                                           static_cast<uint16_t*>(vt_scratch), cu_k, k_lens, Hkv, s_pad);
   B200_CHECK_CUDA(cudaGetLastError());
-  return prefill_launch(q, static_cast<int64_t>(Hq) * kPD, k, vt_scratch, s_pad, cu_q, cu_k, k_lens, B, total_q, total_k, max_q, Hq,
+  return prefill_launch(q, static_cast<int64_t>(Hq) * kPD, k, vt_scratch, s_pad, 0, cu_q, cu_k, k_lens, B, total_q, total_k, max_q, Hq,
                         Hkv, kPD, kPD, scale, causal, nullptr, out, dtype, status, s);
 }
 
 // As b200_prefill_attention for head sizes other than 128 and values that are already transposed:
-//   q [total_q, Hq, dk] with ldq elements between two tokens; k [total_k, Hkv, dk] contiguous; vt [B * Hkv, dv, s_pad] with the
-//   keys of a sequence in its first columns (columns up to the next multiple of 128 below s_pad are read and must be finite);
+//   q [total_q, Hq, dk] with ldq elements between two tokens; k [total_k, Hkv, dk] contiguous; vt [Hkv, dv, total_k], the keys of
+//   a sequence at columns cu_k[b] ... (multiples of 8). Whole tiles of 128 keys are read: what follows a sequence must be finite;
 //   sink: nullable fp32 [Hq] on the device, a logit that joins every row's softmax denominator unscaled and has no value;
-//   out [total_q, Hq, dv]. dk, dv, ldq and s_pad are multiples of 8, dk <= 256.
-B200_API int b200_prefill_attention_vt(const void* q, long long ldq, const void* k, const void* vt, int s_pad, const int* cu_q,
+//   out [total_q, Hq, dv]. dk, dv, ldq and total_k are multiples of 8, dk <= 256.
+B200_API int b200_prefill_attention_vt(const void* q, long long ldq, const void* k, const void* vt, const int* cu_q,
                                        const int* cu_k, const int* k_lens, int B, int total_q, int total_k, int max_q, int Hq,
                                        int Hkv, int dk, int dv, float scale, int causal, const float* sink, void* out, int dtype,
                                        uint32_t* status, void* stream) {
   B200_REQUIRE(dtype == kBF16 || dtype == kF16, "prefill attention supports bf16/f16");
   B200_REQUIRE(Hkv > 0 && Hq % Hkv == 0, "Hq (%d) must be a multiple of Hkv (%d)", Hq, Hkv);
-  B200_REQUIRE(B >= 1 && max_q >= 1 && total_q >= 1 && total_k >= 1 && s_pad >= 1, "empty problem");
-  B200_REQUIRE(dk >= 8 && dk % 8 == 0 && dk <= 256 && dv >= 8 && dv % 8 == 0 && ldq % 8 == 0 && s_pad % 8 == 0,
-               "prefill attention needs dk (%d) <= 256, and dk, dv (%d), ldq, s_pad (%d) in multiples of 8", dk, dv, s_pad);
-  return prefill_launch(q, ldq, k, vt, s_pad, cu_q, cu_k, k_lens, B, total_q, total_k, max_q, Hq, Hkv, dk, dv, scale, causal, sink,
+  B200_REQUIRE(B >= 1 && max_q >= 1 && total_q >= 1 && total_k >= 1, "empty problem");
+  B200_REQUIRE(dk >= 8 && dk % 8 == 0 && dk <= 256 && dv >= 8 && dv % 8 == 0 && ldq % 8 == 0 && total_k % 8 == 0,
+               "prefill attention needs dk (%d) <= 256, and dk, dv (%d), ldq, total_k (%d) in multiples of 8", dk, dv, total_k);
+  B200_REQUIRE(scale > 0.f, "the score scale must be positive");
+  return prefill_launch(q, ldq, k, vt, total_k, 1, cu_q, cu_k, k_lens, B, total_q, total_k, max_q, Hq, Hkv, dk, dv, scale, causal, sink,
                         out, dtype, status, static_cast<cudaStream_t>(stream));
 }

@@ -199,16 +199,22 @@ static int check_norm(const NormParams& n) {
   B200_REQUIRE(n.gain == nullptr || n.h != nullptr, "the norm needs an output");
   return kOk;
 }
+// groups of four columns per thread, from the kernels' instantiations, and the threads that then cover a row
+static int row_groups(int pitch) {
+  const int g = (pitch / 4 + kRnThreads - 1) / kRnThreads;
+  return g <= 4 ? g : 8;
+}
 static int row_threads(int pitch) {
-  const int t = (pitch / 4 + 31) / 32 * 32;
-  return t < kRnThreads ? t : kRnThreads;
+  const int g = row_groups(pitch);
+  return ((pitch / 4 + g - 1) / g + 31) / 32 * 32;
 }
 
 template <typename T, typename P>
-static int launch_rows(void (*k1)(P), void (*k2)(P), void (*k4)(P), void (*k8)(P), const P& p, int T_rows, cudaStream_t s) {
-  const int threads = row_threads(p.norm.pitch);
-  const int groups = (p.norm.pitch / 4 + threads - 1) / threads;
-  B200_CHECK_CUDA(launch_pdl(groups == 1 ? k1 : groups == 2 ? k2 : groups <= 4 ? k4 : k8, dim3(T_rows), dim3(threads), 0, s, p));
+static int launch_rows(void (*k1)(P), void (*k2)(P), void (*k3)(P), void (*k4)(P), void (*k8)(P), const P& p, int T_rows,
+                       cudaStream_t s) {
+  const int groups = row_groups(p.norm.pitch);
+  B200_CHECK_CUDA(launch_pdl(groups == 1 ? k1 : groups == 2 ? k2 : groups == 3 ? k3 : groups == 4 ? k4 : k8, dim3(T_rows),
+                             dim3(row_threads(p.norm.pitch)), 0, s, p));
   return kOk;
 }
 
@@ -226,7 +232,7 @@ B200_API int b200_embed_norm(const long long* ids, const void* table, int rows, 
   p.norm = NormParams{width, pitch, center, eps, gain, bias, h};
   int rc = check_norm(p.norm);
   if (rc != kOk) return rc;
-  B200_DISPATCH_FLOAT(dtype, return launch_rows<T>(embed_norm_kernel<T, 1>, embed_norm_kernel<T, 2>, embed_norm_kernel<T, 4>,
+  B200_DISPATCH_FLOAT(dtype, return launch_rows<T>(embed_norm_kernel<T, 1>, embed_norm_kernel<T, 2>, embed_norm_kernel<T, 3>, embed_norm_kernel<T, 4>,
                                                    embed_norm_kernel<T, 8>, p, rows, static_cast<cudaStream_t>(stream)););
 }
 
@@ -247,6 +253,6 @@ B200_API int b200_residual_norm(const void* a, const void* gate_a, const void* b
   p.norm = NormParams{width, pitch, center, eps, gain, bias, h};
   int rc = check_norm(p.norm);
   if (rc != kOk) return rc;
-  B200_DISPATCH_FLOAT(dtype, return launch_rows<T>(residual_norm_kernel<T, 1>, residual_norm_kernel<T, 2>, residual_norm_kernel<T, 4>,
+  B200_DISPATCH_FLOAT(dtype, return launch_rows<T>(residual_norm_kernel<T, 1>, residual_norm_kernel<T, 2>, residual_norm_kernel<T, 3>, residual_norm_kernel<T, 4>,
                                                    residual_norm_kernel<T, 8>, p, rows, static_cast<cudaStream_t>(stream)););
 }

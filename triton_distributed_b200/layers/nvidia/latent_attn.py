@@ -91,24 +91,22 @@ class LatentAttention:
     def _attend_absorbed(self, q3, kv_cache, layer_idx, step):
         cache = kv_cache.layer(layer_idx)
         qc = ops.head_linear(q3, self.uk_t)
-        splits = ops.choose_latent_splits(step["bsz"], step["seqlen"] * self.heads, step["kv_len"] or kv_cache.max_length)
-        ctx = ops.latent_attention(qc, cache, step["kv_lens"], kv_cache.block_table, step["seqlen"], self.scale, self.sink, splits)
+        splits, rows = ops.choose_latent_splits(step["bsz"], step["seqlen"] * self.heads, step["kv_len"] or kv_cache.max_length)
+        ctx = ops.latent_attention(qc, cache, step["kv_lens"], kv_cache.block_table, step["seqlen"], self.scale, self.sink, splits, rows)
         return ops.head_linear(ctx, self.uv.view(self.heads, self.vdim, self.pitch))
 
     def _attend_expanded(self, q3, kv_cache, layer_idx, step):
         B, S, kv = step["bsz"], step["seqlen"], step["kv_len"]
-        kv8 = pad_up(kv)  # rows between kv and kv8 are unused cache slots: finite, and masked
-        k = torch.empty((B, kv8, self.heads, self.dim), dtype=q3.dtype, device=q3.device)
-        vt = torch.empty((B, self.heads, self.vdim, kv8), dtype=q3.dtype, device=q3.device)
-        for b in range(B):
-            c = kv_cache.rows(layer_idx, b, kv8)
-            ops.linear(c, self.uk, out=k[b].view(kv8, -1))
-            ops.linear(self.uv, c, out=vt[b].view(-1, kv8))
+        kv8 = pad_up(kv)
+        kv_cache.blank(layer_idx, kv, kv8)  # the rows in between are unused slots: masked, and must be finite
+        c = kv_cache.rows(layer_idx, kv8)   # [B * kv8, pitch]
+        k = ops.linear(c, self.uk)
+        vt = ops.linear(self.uv, c)         # values already transposed: [heads * vdim, B * kv8]
         if "cu_q" not in step:  # the same for every layer of the step
             step["cu_q"] = torch.arange(0, (B + 1) * S, S, dtype=torch.int32, device=q3.device)
             step["cu_k"] = torch.arange(0, (B + 1) * kv8, kv8, dtype=torch.int32, device=q3.device)
-        return ops.prefill_attention_vt(q3, k.view(B * kv8, self.heads, self.dim), vt, step["cu_q"], step["cu_k"], step["kv_lens"],
-                                        S, self.scale, True, self.sink)
+        return ops.prefill_attention_vt(q3, k.view(B * kv8, self.heads, self.dim), vt.view(self.heads, self.vdim, B * kv8), step["cu_q"],
+                                        step["cu_k"], step["kv_lens"], S, self.scale, True, self.sink)
 
     @torch.no_grad()
     def partial_fwd(self, q, kv_cache, layer_idx: int, step, out: torch.Tensor | None = None) -> torch.Tensor:

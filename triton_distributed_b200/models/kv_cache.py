@@ -82,7 +82,13 @@ class LatentCache(PagedCache):
         """Pages of one layer: [num_blocks, page, width]."""
         return self.c_cache[layer_idx]
 
-    def rows(self, layer_idx: int, seq: int, count: int) -> torch.Tensor:
-        """The first `count` latent rows of sequence `seq` as one matrix (its pages are consecutive)."""
-        c = self.c_cache[layer_idx].view(self.batch_size, self.blocks_per_seq * self.page_size, -1)
-        return c[seq, :count]
+    def rows(self, layer_idx: int, count: int) -> torch.Tensor:
+        """The first `count` latent rows of every sequence as one matrix [batch * count, width] (a sequence's pages are
+        consecutive; a view where the rows of the batch are, else a copy)."""
+        c = self.c_cache[layer_idx].view(self.batch_size, self.blocks_per_seq * self.page_size, -1)[:, :count]
+        return c.reshape(self.batch_size * count, -1)
+
+    def blank(self, layer_idx: int, start: int, stop: int) -> None:
+        """Zero the unused rows [start, stop) of every sequence."""
+        if stop > start:
+            self.c_cache[layer_idx].view(self.batch_size, self.blocks_per_seq * self.page_size, -1)[:, start:stop].zero_()

@@ -558,20 +558,23 @@ def head_linear(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return y
 
 
-def choose_latent_splits(batch: int, rows: int, max_kv_len: int, sm_count: int = 148) -> int:
-    """Splits of the absorbed latent attention: one wave of CTAs (a CTA owns up to 32 rows and keeps most of an SM's shared
-    memory), at least two 64-token tiles each."""
-    ctas = batch * ((rows + 31) // 32)
-    return int(max(1, min(sm_count // max(ctas, 1), (max_kv_len + 127) // 128, 64)))
+def choose_latent_splits(batch: int, rows: int, max_kv_len: int, sm_count: int = 148) -> tuple[int, int]:
+    """(splits, query rows per CTA) of the absorbed latent attention: one wave of CTAs (a CTA keeps most of an SM's shared
+    memory) over 128-key tiles."""
+    per_cta = 16 if rows <= 16 else 32 if rows <= 32 else 64
+    ctas = batch * ((rows + per_cta - 1) // per_cta)
+    return int(max(1, min(sm_count // max(ctas, 1), (max_kv_len + 255) // 256, 64))), per_cta
 
 
 def latent_attention(q: torch.Tensor, cache: torch.Tensor, kv_lens: torch.Tensor, block_table: torch.Tensor, tokens: int,
-                     scale: float, sink: torch.Tensor | None = None, num_splits: int = 1, plain: bool = False) -> torch.Tensor:
+                     scale: float, sink: torch.Tensor | None = None, num_splits: int = 1, rows_per_cta: int = 0,
+                     variant: str | None = None) -> torch.Tensor:
     """Attention of absorbed queries over paged latents that are both keys and values. q [B * tokens, H, P]; cache
     [blocks, page, P]; kv_lens int32 [B] (the new tokens included); block_table int32 [B, *]; query token i of a sequence attends
     keys j <= kv_len - tokens + i. ``sink`` fp32 [H]. Returns [B * tokens, H, P].
 
-    16-bit ranks up to 512 take the split tensor-core kernel; fp32, wider ranks and ``plain=True`` the one-warp-per-row one."""
+    ``variant``: "tc" (tcgen05 tiles, 16-bit, ranks up to 512), "mma" (warp-level products, same limits) or "plain" (one warp per
+    row, any type and rank); None picks the first that handles the operands."""
     _lib.require_cuda()
     T, H, P = q.shape
     B = kv_lens.numel()
@@ -581,14 +584,22 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, kv_lens: torch.Tensor
         raise ValueError("latent_attention: sink must be fp32 [H]")
     page = cache.shape[1]
     out = torch.empty_like(q)
-    common = (ptr(q), ptr(cache), ptr(block_table), block_table.stride(0), ptr(kv_lens), B, tokens, H, P, page, c_float(scale))
-    if plain or q.dtype == torch.float32 or P > 512 or page % 64 != 0:
-        _lib.call("b200_latent_attention_plain", *common, ptr(sink), ptr(out), dtype_code(q.dtype), stream_ptr())
+    if variant is None:
+        variant = "plain" if q.dtype == torch.float32 or P > 512 or page % 64 != 0 else "tc"
+    shape = (ptr(block_table), block_table.stride(0), ptr(kv_lens), B, tokens, H, P, page, c_float(scale))
+    if variant == "plain":
+        _lib.call("b200_latent_attention_plain", ptr(q), ptr(cache), *shape, ptr(sink), ptr(out), dtype_code(q.dtype), stream_ptr())
         _count()
         return out
     o_part = torch.empty((T * H, num_splits, P), dtype=torch.float32, device=q.device)
     lse_part = torch.empty((T * H, num_splits), dtype=torch.float32, device=q.device)
-    _lib.call("b200_latent_attention", *common, num_splits, ptr(o_part), ptr(lse_part), dtype_code(q.dtype), stream_ptr())
+    if variant == "tc":
+        per_cta = rows_per_cta or (16 if tokens * H <= 16 else 32 if tokens * H <= 32 else 64)
+        _lib.call("b200_latent_decode", ptr(q), ptr(cache), ctypes.c_longlong(cache.shape[0] * page), *shape, num_splits, per_cta,
+                  ptr(o_part), ptr(lse_part), dtype_code(q.dtype), ptr(_pipeline_status(q.device)), stream_ptr())
+    else:
+        _lib.call("b200_latent_attention", ptr(q), ptr(cache), *shape, num_splits, ptr(o_part), ptr(lse_part), dtype_code(q.dtype),
+                  stream_ptr())
     _lib.call("b200_latent_combine", ptr(o_part), ptr(lse_part), ptr(sink), T * H, H, num_splits, P, ptr(out), dtype_code(q.dtype),
               stream_ptr())
     _count(2)
@@ -599,16 +610,17 @@ def prefill_attention_vt(q: torch.Tensor, k: torch.Tensor, vt: torch.Tensor, cu_
                          seqlens_k: torch.Tensor, max_seqlen_q: int, scale: float, causal: bool = True,
                          sink: torch.Tensor | None = None) -> torch.Tensor:
     """``prefill_attention`` for other head sizes, transposed values and an optional sink logit per head. q [total_q, Hq, dk]
-    (rows may be strided), k [total_k, Hkv, dk], vt [B, Hkv, dv, S] (keys of a sequence in its first columns), sink fp32 [Hq]
-    or None; dk <= 256, dk, dv and S multiples of 8. Returns [total_q, Hq, dv]."""
+    (rows may be strided), k [total_k, Hkv, dk], vt [Hkv, dv, total_k]: the keys of a sequence are rows ``cu_seqlens_k[b]`` ... of k and
+    the same columns of vt (``seqlens_k[b]`` of them; multiples of 8 apart; what lies between must be finite). sink fp32 [Hq] or
+    None; dk <= 256, dk, dv and total_k multiples of 8. Returns [total_q, Hq, dv]."""
     _lib.require_cuda()
     total_q, Hq, dk = q.shape
     total_k, Hkv, _ = k.shape
-    B, _, dv, s_pad = vt.shape
-    if q.stride(2) != 1 or q.stride(1) != dk or not (k.is_contiguous() and vt.is_contiguous()) or vt.shape[1] != Hkv:
+    B, dv = seqlens_k.numel(), vt.shape[1]
+    if q.stride(2) != 1 or q.stride(1) != dk or not (k.is_contiguous() and vt.is_contiguous()) or vt.shape != (Hkv, dv, total_k):
         raise ValueError("prefill_attention_vt: shape/layout mismatch")
     out = torch.empty((total_q, Hq, dv), dtype=q.dtype, device=q.device)
-    _lib.call("b200_prefill_attention_vt", ptr(q), ctypes.c_longlong(q.stride(0)), ptr(k), ptr(vt), s_pad, ptr(cu_seqlens_q),
+    _lib.call("b200_prefill_attention_vt", ptr(q), ctypes.c_longlong(q.stride(0)), ptr(k), ptr(vt), ptr(cu_seqlens_q),
               ptr(cu_seqlens_k), ptr(seqlens_k), B, total_q, total_k, int(max_seqlen_q), Hq, Hkv, dk, dv, c_float(scale),
               1 if causal else 0, ptr(sink), ptr(out), dtype_code(q.dtype), ptr(_pipeline_status(q.device)), stream_ptr())
     _count()
