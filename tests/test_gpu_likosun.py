@@ -33,7 +33,7 @@ def test_gemm_f32_is_true_fp32(M, N, K):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16, torch.float16])
-@pytest.mark.parametrize("width,center,with_bias", [(75, True, True), (1000, False, False), (2048, True, False), (5120, True, True), (9001, True, True)])
+@pytest.mark.parametrize("width,center,with_bias", [(75, True, True), (1030, True, True), (2052, False, True), (1000, False, False), (2048, True, False), (5120, True, True), (9001, True, True)])
 def test_embed_norm(dtype, width, center, with_bias):
     from triton_distributed_b200 import ops
     P, V = (width + 7) // 8 * 8, 50
@@ -50,17 +50,19 @@ def test_embed_norm(dtype, width, center, with_bias):
     assert torch.equal(x, state0) and torch.all(x[:, width:] == 0) and torch.all(h[:, width:] == 0)
     _close(x[:, :width], rows, torch.float32)
     g, b = gain[:width].double().cpu(), bias[:width].double().cpu() * (1.0 if with_bias else 0.0)
-    want = ref.layer_norm_ref(rows, g, b, 1e-3) if center else ref.rms_norm_ref(rows, g, 1e-3)
+    want = ref.layer_norm_ref(rows, g, b, 1e-3) if center else ref.rms_norm_ref(rows, g, 1e-3) + b
     _close(h[:, :width], want, dtype)
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("width,n_prev,two,gates,keep,norm", [
     (75, 1, True, True, True, True), (264, 7, False, True, True, True), (2048, 3, True, False, False, True),
-    (4100, 12, True, True, True, True), (16, 0, True, True, False, True), (640, 2, True, True, True, False)])
-def test_residual_norm(dtype, width, n_prev, two, gates, keep, norm):
+    (4100, 12, True, True, True, True), (16, 0, True, True, False, True), (640, 2, True, True, True, False), (1100, 5, True, True, True, True), (6000, 1, True, True, True, True), (2500, 2, True, True, True, False)])
+@pytest.mark.parametrize("T", [5, 30, 170])
+def test_residual_norm(dtype, width, n_prev, two, gates, keep, norm, T):
+    """Few rows take a cluster of CTAs per row (from 1024 columns on), many one CTA each."""
     from triton_distributed_b200 import ops
-    T, P = 5, (width + 7) // 8 * 8
+    P = (width + 7) // 8 * 8
 
     def padded(*lead, dt=dtype, scale=1.0):
         t = torch.zeros(*lead, P, device="cuda", dtype=dt)

@@ -11,10 +11,11 @@
 //   warp 0     TMA producer: the Q tile once, then the tiles in slots of 128 keys x 128 columns (two 64-column swizzle atoms)
 //   warp 1     MMA issuer; a slot is given back as soon as its chunk of the output has been accumulated, so the next tile
 //              streams in while the rest of this one is still being multiplied
-//   warps 4-7  softmax, one thread per key of the tile: column maxima by warp-wide redux + shared memory, exponentials, P as
-//              16-bit into a swizzled tile. The reference maximum of a row only moves when it is exceeded by more than 2^8, so
-//              the output in tensor memory is rescaled a few times per sequence at most; sums and output use the same reference,
-//              which cancels in the end.
+//   warps 4-11 softmax, two threads per key of the tile (each has half of the query rows): exponentials against a reference
+//              maximum per row, P as 16-bit into a swizzled tile. The reference only moves when a score exceeds it by more than
+//              2^8: one vote per tile decides, and only then are the maxima reduced over the keys and the sums and the output in
+//              tensor memory rescaled. Sums and output share the reference, which cancels in the end.
+// The producer also asks L2 for the tile after next, so that a slot that becomes free is refilled at L2 latency.
 // Every barrier wait is bounded; on expiry the CTA unwinds through an abort flag and reports a status.
 #include "b200/host.h"
 #include "b200/primitives.cuh"
@@ -27,7 +28,7 @@ namespace b200 {
 constexpr int kLdKeys = 128;              // keys per tile
 constexpr int kLdAtom = kLdKeys * 128;    // 128 keys x 64 columns: 16 KB
 constexpr int kLdSlot = 2 * kLdAtom;      // 128 keys x 128 columns
-constexpr int kLdThreads = 256;
+constexpr int kLdThreads = 384;
 constexpr float kLdSlack = 8.f;           // how far (log2) a score may exceed the reference before it moves
 constexpr int kLdSmemMax = 226 * 1024;
 
@@ -66,16 +67,42 @@ __device__ __forceinline__ float ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-__device__ __forceinline__ void tmem_st_32x16(uint32_t taddr, const uint32_t (&r)[16]) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], "
-      "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};" ::"r"(taddr),
-      "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]),
-      "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
-      : "memory");
+__device__ __forceinline__ void tmem_st_32x8(uint32_t taddr, const uint32_t (&r)[8]) {
+  asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"r"(taddr), "r"(r[0]), "r"(r[1]),
+               "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7])
+               : "memory");
 }
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
-__device__ __forceinline__ void ld_softmax_bar() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+// barrier of the 256 softmax threads, and the same with a vote
+__device__ __forceinline__ void ld_softmax_bar() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
+__device__ __forceinline__ bool ld_softmax_any(bool v) {
+  uint32_t r;
+  asm volatile(
+      "{\n"
+      ".reg .pred P, Q;\n"
+      "setp.ne.u32 P, %1, 0;\n"
+      "barrier.cta.red.or.pred Q, 2, 256, P;\n"
+      "selp.u32 %0, 1, 0, Q;\n"
+      "}\n"
+      : "=r"(r)
+      : "r"(v ? 1u : 0u)
+      : "memory");
+  return r != 0;
+}
+// reads kCols (8, 16 or 32) consecutive columns of this thread's lane
+template <int kCols>
+__device__ __forceinline__ void tmem_ld_cols(uint32_t taddr, float (&v)[kCols]) {
+  uint32_t r[kCols];
+  if constexpr (kCols == 8) tmem_ld_32x8(taddr, r);
+  else if constexpr (kCols == 16) tmem_ld_32x16(taddr, r);
+  else tmem_ld_32x32(taddr, r);
+  tmem_ld_wait();
+#pragma unroll
+  for (int i = 0; i < kCols; ++i) v[i] = __uint_as_float(r[i]);
+}
+__device__ __forceinline__ void tma_prefetch_l2_2d(const CUtensorMap* map, int x, int y) {
+  asm volatile("cp.async.bulk.prefetch.tensor.2d.L2.global [%0, {%1, %2}];" ::"l"(map), "r"(x), "r"(y) : "memory");
+}
 
 // N: query rows per CTA (16, 32 or 64); RK: rank rounded up to a multiple of 128 (TMA fills the padding columns with zeros)
 template <int N, int RK>
@@ -99,7 +126,6 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
   uint64_t* o_full = bars + 35;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 36);
   volatile uint32_t* abort_flag = tmem_slot + 1;
-  volatile int* moved = reinterpret_cast<volatile int*>(tmem_slot + 2);  // last tile at which a reference maximum moved
   float* xmax = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(bars) + 512);  // [4 warps][N]
   float* mref = xmax + 4 * N;                                                      // [N]
   float* corr = mref + N;                                                          // [N]; at the end 1 / row sum
@@ -118,10 +144,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
     }
     mbar_init(q_full, 1);
     mbar_init(s_full, 1);
-    mbar_init(p_full, 4);
+    mbar_init(p_full, 8);
     mbar_init(o_full, 1);
     *abort_flag = 0;
-    *moved = -1;
     mbar_fence_init();
     tma_prefetch_desc(&tmC);
     tma_prefetch_desc(&tmQ);
@@ -151,16 +176,26 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
       mbar_expect_tx(q_full, (RK / 64) * kRowAtom);
       for (int a = 0; a < RK / 64; ++a) tma_load_2d(sQ + a * kRowAtom, &tmQ, q_full, a * 64, row_base);
       const int* table = p.block_table + static_cast<size_t>(b) * p.bt_stride;
+      // 64 keys lie in one page; a half beyond the last key repeats the first
+      auto slot_row = [&](int tile, int half) {
+        int key = tile * kLdKeys + 64 * half;
+        if (key >= n_keys) key = tile * kLdKeys;
+        return table[key / p.page] * p.page + key % p.page;
+      };
+      auto prefetch = [&](int tile) {
+        if (tile >= tile1) return;
+        for (int half = 0; half < 2; ++half) {
+          const int row = slot_row(tile, half);
+          for (int a = 0; a < RK / 64; ++a)
+            if (a * 64 < p.pitch) tma_prefetch_l2_2d(&tmC, a * 64, row);
+        }
+      };
       int it = 0;
       bool ok = true;
+      prefetch(tile0 + 1);
       for (int tile = tile0; tile < tile1 && ok; ++tile) {
-        int row[2];
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {  // 64 keys lie in one page; a half beyond the last key repeats the first
-          int key = tile * kLdKeys + 64 * half;
-          if (key >= n_keys) key = tile * kLdKeys;
-          row[half] = table[key / p.page] * p.page + key % p.page;
-        }
+        const int row[2] = {slot_row(tile, 0), slot_row(tile, 1)};
+        prefetch(tile + 2);
         for (int pr = 0; pr < kPairs && ok; ++pr, ++it) {
           const int slot = it % kSlots;
           ok = mbar_wait(empty + slot, ((it / kSlots) & 1) ^ 1, abort_flag, timeout_ns);
@@ -214,11 +249,14 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
     }
     __syncwarp();
   } else if (warp >= 4) {
-    const int w4 = warp & 3, t = threadIdx.x - 128;  // t: key of the tile = TMEM lane
-    const uint32_t lane_base = tmem_base + (static_cast<uint32_t>(w4 * 32) << 16);
-    float l[N];  // this key's share of every row sum
+    constexpr int kCols = N / 2;  // query rows of this thread
+    const int w4 = warp & 3, half = (warp - 4) >> 2;
+    const int t = w4 * 32 + lane;  // key of the tile = TMEM lane
+    const int n0 = half * kCols;
+    const uint32_t lane_base = tmem_base + (static_cast<uint32_t>(w4 * 32) << 16) + n0;
+    float l[kCols];  // this key's share of the row sums
 #pragma unroll
-    for (int n = 0; n < N; ++n) l[n] = 0.f;
+    for (int i = 0; i < kCols; ++i) l[i] = 0.f;
     const int all_below = r0 + N <= n_rows ? first_limit + r0 / p.H : -1;  // keys up to here are visible to all rows
     uint8_t* p_col = sP + (t >> 6) * kRowAtom + (t & 7) * 2;
     const int p_chunk = (t & 63) >> 3;
@@ -231,74 +269,69 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
       tc_fence_after_sync();
       const int key = tile * kLdKeys + t;
       const bool masked = tile * kLdKeys + kLdKeys - 1 > all_below;
+      float s[kCols];
+      bool exceeds = false;
       if (ok) {
+        tmem_ld_cols<kCols>(lane_base, s);
 #pragma unroll
-        for (int c = 0; c < N / 16; ++c) {
-          uint32_t r[16];
-          tmem_ld_32x16(lane_base + c * 16, r);
-          tmem_ld_wait();
-          float mine = 0.f;
+        for (int i = 0; i < kCols; ++i) {
+          s[i] *= p.scale_log2e;
+          if (masked) s[i] = key <= limit[n0 + i] ? s[i] : -INFINITY;
+          exceeds |= s[i] > mref[n0 + i] + kLdSlack;  // (always when the row has no reference yet and sees this key)
+        }
+      }
+      if (ld_softmax_any(exceeds)) {
+        if (ok) {
 #pragma unroll
-          for (int i = 0; i < 16; ++i) {
-            float v = __uint_as_float(r[i]);
-            if (masked) v = key <= limit[c * 16 + i] ? v : -INFINITY;
-            const float m = redux_max(v);
-            mine = lane == i ? m : mine;
+          for (int i = 0; i < kCols; ++i) {
+            const float m = redux_max(s[i]);
+            if (lane == 0) xmax[w4 * N + n0 + i] = m;
           }
-          if (lane < 16) xmax[w4 * N + c * 16 + lane] = mine;
         }
-      }
-      ld_softmax_bar();
-      if (t < N) {
-        const float mx = fmaxf(fmaxf(xmax[t], xmax[N + t]), fmaxf(xmax[2 * N + t], xmax[3 * N + t])) * p.scale_log2e;
-        const float old = mref[t];
-        if (mx > old + kLdSlack) {  // (always when the row has no reference yet and sees a key)
-          corr[t] = ex2(old - mx);
-          mref[t] = mx;
-          *moved = tile;
-        } else {
-          corr[t] = 1.f;
+        ld_softmax_bar();
+        if (half == 0 && t < N) {
+          const float mx = fmaxf(fmaxf(xmax[t], xmax[N + t]), fmaxf(xmax[2 * N + t], xmax[3 * N + t]));
+          const float old = mref[t];
+          const bool up = mx > old + kLdSlack;
+          corr[t] = up ? ex2(old - mx) : 1.f;
+          if (up) mref[t] = mx;
         }
-      }
-      ld_softmax_bar();
-      if (!ok) continue;
-      if (*moved == tile && tile != tile0) {
+        ld_softmax_bar();
+        if (ok && tile != tile0) {
 #pragma unroll
-        for (int n = 0; n < N; ++n) l[n] *= corr[n];
+          for (int i = 0; i < kCols; ++i) l[i] *= corr[n0 + i];
 #pragma unroll 1
-        for (int c = 0; c < kPairs * (N / 16); ++c) {
-          uint32_t r[16];
-          const uint32_t at = lane_base + N + c * 16;
-          tmem_ld_32x16(at, r);
-          tmem_ld_wait();
+          for (int pr = 0; pr < kPairs; ++pr) {
 #pragma unroll
-          for (int i = 0; i < 16; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * corr[(c % (N / 16)) * 16 + i]);
-          tmem_st_32x16(at, r);
+            for (int c = 0; c < kCols / 8; ++c) {
+              uint32_t r[8];
+              const uint32_t at = lane_base + N * (1 + pr) + c * 8;
+              tmem_ld_32x8(at, r);
+              tmem_ld_wait();
+#pragma unroll
+              for (int i = 0; i < 8; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * corr[n0 + c * 8 + i]);
+              tmem_st_32x8(at, r);
+            }
+          }
+          tmem_st_wait();
         }
-        tmem_st_wait();
       }
+      if (!ok) continue;
 #pragma unroll
-      for (int c = 0; c < N / 16; ++c) {
-        uint32_t r[16];
-        tmem_ld_32x16(lane_base + c * 16, r);
-        tmem_ld_wait();
-#pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          const int n = c * 16 + i;
-          float pr = ex2(fmaf(__uint_as_float(r[i]), p.scale_log2e, -mref[n]));
-          if (masked) pr = key <= limit[n] ? pr : 0.f;
-          l[n] += pr;
-          const uint16_t h = p.bf16 ? __bfloat16_as_ushort(__float2bfloat16(pr)) : __half_as_ushort(__float2half(pr));
-          *reinterpret_cast<uint16_t*>(p_col + n * 128 + ((p_chunk ^ (n & 7)) << 4)) = h;
-        }
+      for (int i = 0; i < kCols; ++i) {
+        const int n = n0 + i;
+        float pr = ex2(s[i] - mref[n]);
+        if (masked) pr = key <= limit[n] ? pr : 0.f;
+        l[i] += pr;
+        const uint16_t h = p.bf16 ? __bfloat16_as_ushort(__float2bfloat16(pr)) : __half_as_ushort(__float2half(pr));
+        *reinterpret_cast<uint16_t*>(p_col + n * 128 + ((p_chunk ^ (n & 7)) << 4)) = h;
       }
       if (key >= n_keys) {  // slots beyond the sequence may hold anything: their weight is zero, make the value zero too
-        for (int pr = 0; pr < kPairs; ++pr)
-          for (int a = 0; a < 2; ++a) {
-            uint4* dst = reinterpret_cast<uint4*>(ring + ((it + pr) % kSlots) * kLdSlot + a * kLdAtom + t * 128);
+        for (int pr = 0; pr < kPairs; ++pr) {
+          uint4* dst = reinterpret_cast<uint4*>(ring + ((it + pr) % kSlots) * kLdSlot + half * kLdAtom + t * 128);
 #pragma unroll
-            for (int i = 0; i < 8; ++i) dst[i] = make_uint4(0, 0, 0, 0);
-          }
+          for (int i = 0; i < 8; ++i) dst[i] = make_uint4(0, 0, 0, 0);
+        }
       }
       tc_fence_before_sync();     // this thread's TMEM accesses are done
       fence_view_async_shared();  // its shared-memory writes are visible to the tensor core
@@ -307,22 +340,17 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
     }
     // ---- row sums over the keys, then the normalised partial output and its log-sum-exp
 #pragma unroll
-    for (int c = 0; c < N / 16; ++c) {
-      float mine = 0.f;
-#pragma unroll
-      for (int i = 0; i < 16; ++i) {
-        const float s = warp_sum(l[c * 16 + i]);
-        mine = lane == i ? s : mine;
-      }
-      if (lane < 16) xsum[w4 * N + c * 16 + lane] = mine;
+    for (int i = 0; i < kCols; ++i) {
+      const float sum = warp_sum(l[i]);
+      if (lane == 0) xsum[w4 * N + n0 + i] = sum;
     }
     ld_softmax_bar();
-    if (t < N) {
-      const float s = (xsum[t] + xsum[N + t]) + (xsum[2 * N + t] + xsum[3 * N + t]);
-      corr[t] = s > 0.f ? 1.f / s : 0.f;
+    if (half == 0 && t < N) {
+      const float sum = (xsum[t] + xsum[N + t]) + (xsum[2 * N + t] + xsum[3 * N + t]);
+      corr[t] = sum > 0.f ? 1.f / sum : 0.f;
       if (r0 + t < n_rows)
         p.lse_part[static_cast<size_t>(row_base + t) * p.splits + split] =
-            s > 0.f ? (mref[t] + log2f(s)) * 0.6931471805599453f : -INFINITY;
+            sum > 0.f ? (mref[t] + log2f(sum)) * 0.6931471805599453f : -INFINITY;
     }
     ld_softmax_bar();
     if (tile0 < tile1) {
@@ -333,18 +361,12 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
 #pragma unroll 1
         for (int pr = 0; pr < kPairs; ++pr) {
           const int col = pr * 128 + t;
+          float o[kCols];
+          tmem_ld_cols<kCols>(lane_base + N * (1 + pr), o);
 #pragma unroll
-          for (int c = 0; c < N / 16; ++c) {
-            uint32_t r[16];
-            tmem_ld_32x16(lane_base + N * (1 + pr) + c * 16, r);
-            tmem_ld_wait();
-#pragma unroll
-            for (int i = 0; i < 16; ++i) {
-              const int n = c * 16 + i;
-              if (r0 + n < n_rows && col < p.pitch)
-                p.o_part[(static_cast<size_t>(row_base + n) * p.splits + split) * p.pitch + col] = __uint_as_float(r[i]) * corr[n];
-            }
-          }
+          for (int i = 0; i < kCols; ++i)
+            if (r0 + n0 + i < n_rows && col < p.pitch)
+              p.o_part[(static_cast<size_t>(row_base + n0 + i) * p.splits + split) * p.pitch + col] = o[i] * corr[n0 + i];
         }
       }
     }

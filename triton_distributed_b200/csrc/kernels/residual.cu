@@ -10,8 +10,13 @@
 // gain and an optional bias. The stream, the states and all arithmetic are fp32; a, b, the gates and h have the model's
 // storage type (bf16 / f16 / fp32). Rows are `pitch` wide: columns in [width, pitch) are padding, which carries zeros and
 // is left out of the statistics.
+//
+// Few tokens (decode) do not fill the machine with one CTA each, and a row with many earlier states is a long chain of loads:
+// then a cluster of CTAs shares a row, a slice of columns each, and exchanges (count, mean, squared deviations) of the slices
+// through distributed shared memory, which merge exactly.
 #include "b200/elem.cuh"
 #include "b200/host.h"
+#include "b200/tcgen05.cuh"
 
 #include <cstring>
 
@@ -61,78 +66,127 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return warp_sum((threadIdx.x & 31) < nw ? red[threadIdx.x & 31] : 0.f);
 }
 
-// U groups of four columns per thread: group u of a thread starts at column 4 * (threadIdx.x + u * blockDim.x)
-template <typename T, int U>
-__device__ __forceinline__ void norm_row(const NormParams& n, size_t row, const float4 (&v)[U], const float4 (&gain)[U],
-                                         const float4 (&bias)[U], float* red) {
-  if (n.gain == nullptr) return;
-  float mean = 0.f;
+// The slice of a row that a CTA owns: all of it, or one of kCl equal parts (in groups of four columns).
+template <int kCl>
+struct Slice {
+  int begin, end;
+  __device__ __forceinline__ explicit Slice(int pitch) {
+    const int span = ((pitch / 4 + kCl - 1) / kCl) * 4;
+    begin = kCl == 1 ? 0 : static_cast<int>(cluster_ctarank()) * span;
+    end = min(pitch, begin + span);
+  }
+  // group u of this thread: columns [col(u), col(u) + 4)
+  __device__ __forceinline__ int col(int u) const { return begin + 4 * (threadIdx.x + u * blockDim.x); }
+};
+
+struct RowStats {
+  float mean, m2;  // mean, sum of squared deviations from it
+};
+
+// statistics of the CTA's slice; RMS norm (center = 0) takes the deviations from zero
+template <int U, int kCl>
+__device__ __forceinline__ RowStats slice_stats(const NormParams& n, const Slice<kCl>& sl, const float4 (&v)[U], int count, float* red) {
+  RowStats st{0.f, 0.f};
   if (n.center) {
     float s = 0.f;
 #pragma unroll
-    for (int u = 0; u < U; ++u) s += (v[u].x + v[u].y) + (v[u].z + v[u].w);
-    mean = block_sum(s, red) / n.width;
+    for (int u = 0; u < U; ++u) s += (v[u].x + v[u].y) + (v[u].z + v[u].w);  // padding columns are zero
+    st.mean = count > 0 ? block_sum(s, red) / count : block_sum(s, red);
   }
   float ss = 0.f;
 #pragma unroll
   for (int u = 0; u < U; ++u) {
-    const int c = 4 * (threadIdx.x + u * blockDim.x);
-    const float d[4] = {v[u].x - mean, v[u].y - mean, v[u].z - mean, v[u].w - mean};
+    const int c = sl.col(u);
+    const float d[4] = {v[u].x - st.mean, v[u].y - st.mean, v[u].z - st.mean, v[u].w - st.mean};
 #pragma unroll
-    for (int e = 0; e < 4; ++e) ss += c + e < n.width ? d[e] * d[e] : 0.f;
+    for (int e = 0; e < 4; ++e) ss += c + e < min(sl.end, n.width) ? d[e] * d[e] : 0.f;
   }
-  const float inv = 1.f / sqrtf(block_sum(ss, red) / n.width + n.eps);
+  st.m2 = block_sum(ss, red);
+  return st;
+}
+
+template <typename T, int U, int kCl>
+__device__ __forceinline__ void norm_row(const NormParams& n, const Slice<kCl>& sl, size_t row, const float4 (&v)[U],
+                                         const float4 (&gain)[U], const float4 (&bias)[U], float* red, float4* shared_stats) {
+  if (n.gain == nullptr) return;  // the same for the whole cluster
+  const int count = max(0, min(sl.end, n.width) - sl.begin);
+  RowStats st = slice_stats<U, kCl>(n, sl, v, count, red);
+  if (kCl > 1) {
+    const uint32_t me = cluster_ctarank();
+    if (threadIdx.x < kCl) {
+      const uint32_t dst = mapa_u32(shared_stats + me, threadIdx.x);
+      asm volatile("st.shared::cluster.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(dst), "f"(static_cast<float>(count)), "f"(st.mean),
+                   "f"(st.m2), "f"(0.f)
+                   : "memory");
+    }
+    cluster_sync_all();
+    float total = 0.f;
+#pragma unroll
+    for (int i = 0; i < kCl; ++i) total += shared_stats[i].x * shared_stats[i].y;
+    const float mean = total / n.width;
+    float m2 = 0.f;
+#pragma unroll
+    for (int i = 0; i < kCl; ++i) {
+      const float d = shared_stats[i].y - mean;
+      m2 += shared_stats[i].z + shared_stats[i].x * d * d;
+    }
+    st = RowStats{mean, m2};
+  }
+  const float inv = 1.f / sqrtf(st.m2 / n.width + n.eps);
 #pragma unroll
   for (int u = 0; u < U; ++u) {
-    const int c = 4 * (threadIdx.x + u * blockDim.x);
-    if (c < n.pitch) {
+    const int c = sl.col(u);
+    if (c < sl.end) {
       float4 o;
-      o.x = (v[u].x - mean) * inv * gain[u].x + bias[u].x;
-      o.y = (v[u].y - mean) * inv * gain[u].y + bias[u].y;
-      o.z = (v[u].z - mean) * inv * gain[u].z + bias[u].z;
-      o.w = (v[u].w - mean) * inv * gain[u].w + bias[u].w;
+      o.x = (v[u].x - st.mean) * inv * gain[u].x + bias[u].x;
+      o.y = (v[u].y - st.mean) * inv * gain[u].y + bias[u].y;
+      o.z = (v[u].z - st.mean) * inv * gain[u].z + bias[u].z;
+      o.w = (v[u].w - st.mean) * inv * gain[u].w + bias[u].w;
       store4(static_cast<T*>(n.h) + row * n.pitch + c, o);
     }
   }
 }
 
 // the gain and bias are weights: read before the dependency wait
-template <typename T, int U>
-__device__ __forceinline__ void load_norm_weights(const NormParams& n, float4 (&gain)[U], float4 (&bias)[U]) {
+template <typename T, int U, int kCl>
+__device__ __forceinline__ void load_norm_weights(const NormParams& n, const Slice<kCl>& sl, float4 (&gain)[U], float4 (&bias)[U]) {
 #pragma unroll
   for (int u = 0; u < U; ++u) {
-    const int c = 4 * (threadIdx.x + u * blockDim.x);
+    const int c = sl.col(u);
     gain[u] = bias[u] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (n.gain != nullptr && c < n.pitch) {
+    if (n.gain != nullptr && c < sl.end) {
       gain[u] = load4(static_cast<const T*>(n.gain) + c);
       if (n.bias != nullptr) bias[u] = load4(static_cast<const T*>(n.bias) + c);
     }
   }
 }
 
-template <typename T, int U>
+template <typename T, int U, int kCl>
 __global__ void __launch_bounds__(kRnThreads) embed_norm_kernel(const EmbedParams p) {
   __shared__ float red[32];
-  const size_t t = blockIdx.x;
+  __shared__ float4 stats[kCl];
+  const size_t t = blockIdx.x / kCl;
   const int pitch = p.norm.pitch;
+  const Slice<kCl> sl(pitch);
   griddep_launch_dependents();
   float4 gain[U], bias[U], v[U];
-  load_norm_weights<T, U>(p.norm, gain, bias);
+  load_norm_weights<T, U, kCl>(p.norm, sl, gain, bias);
+  if (kCl > 1) cluster_sync_all();  // every CTA of the cluster runs before any writes to another's shared memory
   griddep_wait();
   const long long id = p.ids[t];
   const bool ok = id >= 0 && id < p.V;   // an id outside the table reads as a zero row
 #pragma unroll
   for (int u = 0; u < U; ++u) {
-    const int c = 4 * (threadIdx.x + u * blockDim.x);
+    const int c = sl.col(u);
     v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (c < pitch) {
+    if (c < sl.end) {
       if (ok) v[u] = load4(static_cast<const T*>(p.table) + static_cast<size_t>(id) * pitch + c);
       v[u].x *= p.scale; v[u].y *= p.scale; v[u].z *= p.scale; v[u].w *= p.scale;
       store4(p.x + t * pitch + c, v[u]);
       if (p.state0 != nullptr) store4(p.state0 + t * pitch + c, v[u]);
     }
   }
-  norm_row<T, U>(p.norm, t, v, gain, bias, red);
+  norm_row<T, U, kCl>(p.norm, sl, t, v, gain, bias, red, stats);
 }
 
 __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
@@ -151,24 +205,39 @@ __device__ __forceinline__ float4 gated(const void* val, const void* gate, const
   return a;
 }
 
-template <typename T, int U>
+template <typename T, int U, int kCl>
 __global__ void __launch_bounds__(kRnThreads) residual_norm_kernel(const ResidualParams p) {
   __shared__ float red[32];
-  const size_t t = blockIdx.x;
+  __shared__ float4 stats[kCl];
+  const size_t t = blockIdx.x / kCl;
   const int pitch = p.norm.pitch;
+  const Slice<kCl> sl(pitch);
   griddep_launch_dependents();
   float4 gain[U], bias[U], x[U];
-  load_norm_weights<T, U>(p.norm, gain, bias);
+  load_norm_weights<T, U, kCl>(p.norm, sl, gain, bias);
+  if (kCl > 1) cluster_sync_all();  // every CTA of the cluster runs before any writes to another's shared memory
   griddep_wait();
 #pragma unroll
   for (int u = 0; u < U; ++u) {
-    const int c = 4 * (threadIdx.x + u * blockDim.x);
+    const int c = sl.col(u);
     x[u] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (c >= pitch) continue;
+    if (c >= sl.end) continue;
     const size_t at = t * pitch + c;
+    // the average over the earlier states first: its loads do not depend on anything else of the row
+    float4 avg = make_float4(0.f, 0.f, 0.f, 0.f);
+    float wn = 1.f;
+    if (p.weights != nullptr) {
+      const float* st = p.states + at;
+      wn = __ldg(p.weights + p.n_prev);
+#pragma unroll 8
+      for (int j = 0; j < p.n_prev; ++j) {
+        const float w = __ldg(p.weights + j);
+        const float4 o = load4(st + j * p.state_stride);
+        avg.x = fmaf(w, o.x, avg.x); avg.y = fmaf(w, o.y, avg.y); avg.z = fmaf(w, o.z, avg.z); avg.w = fmaf(w, o.w, avg.w);
+      }
+    }
     float4 r = load4(p.x + at);
-    const float4 a = gated<T>(p.a, p.gate_a, p.bias_a, t, pitch, p.ldg, c);
-    float4 s = a;
+    float4 s = gated<T>(p.a, p.gate_a, p.bias_a, t, pitch, p.ldg, c);
     if (p.b != nullptr) {
       const float4 b = gated<T>(p.b, p.gate_b, p.bias_b, t, pitch, p.ldg, c);
       s.x += b.x; s.y += b.y; s.z += b.z; s.w += b.w;
@@ -176,20 +245,12 @@ __global__ void __launch_bounds__(kRnThreads) residual_norm_kernel(const Residua
     r.x = fmaf(p.mult, s.x, r.x); r.y = fmaf(p.mult, s.y, r.y); r.z = fmaf(p.mult, s.z, r.z); r.w = fmaf(p.mult, s.w, r.w);
     if (p.weights != nullptr) {
       if (p.keep) store4(p.states + p.n_prev * p.state_stride + at, r);
-      const float wn = __ldg(p.weights + p.n_prev);
-      r.x *= wn; r.y *= wn; r.z *= wn; r.w *= wn;
-      const float* st = p.states + at;
-#pragma unroll 8
-      for (int j = 0; j < p.n_prev; ++j) {
-        const float w = __ldg(p.weights + j);
-        const float4 o = load4(st + j * p.state_stride);
-        r.x = fmaf(w, o.x, r.x); r.y = fmaf(w, o.y, r.y); r.z = fmaf(w, o.z, r.z); r.w = fmaf(w, o.w, r.w);
-      }
+      r.x = fmaf(wn, r.x, avg.x); r.y = fmaf(wn, r.y, avg.y); r.z = fmaf(wn, r.z, avg.z); r.w = fmaf(wn, r.w, avg.w);
     }
     x[u] = r;
     store4(p.x + at, r);
   }
-  norm_row<T, U>(p.norm, t, x, gain, bias, red);
+  norm_row<T, U, kCl>(p.norm, sl, t, x, gain, bias, red, stats);
 }
 
 static int check_norm(const NormParams& n) {
@@ -209,14 +270,51 @@ static int row_threads(int pitch) {
   return ((pitch / 4 + g - 1) / g + 31) / 32 * 32;
 }
 
-template <typename T, typename P>
-static int launch_rows(void (*k1)(P), void (*k2)(P), void (*k3)(P), void (*k4)(P), void (*k8)(P), const P& p, int T_rows,
-                       cudaStream_t s) {
-  const int groups = row_groups(p.norm.pitch);
-  B200_CHECK_CUDA(launch_pdl(groups == 1 ? k1 : groups == 2 ? k2 : groups == 3 ? k3 : groups == 4 ? k4 : k8, dim3(T_rows),
-                             dim3(row_threads(p.norm.pitch)), 0, s, p));
+template <typename P>
+static int launch_cluster(void (*kernel)(P), const P& p, int rows, int cl, int threads, cudaStream_t s) {
+  cudaLaunchConfig_t cfg;
+  memset(&cfg, 0, sizeof(cfg));
+  cfg.gridDim = dim3(rows * cl);
+  cfg.blockDim = dim3(threads);
+  cfg.stream = s;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = cl;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = pdl_enabled() ? 2 : 1;
+  B200_CHECK_CUDA(cudaLaunchKernelEx(&cfg, kernel, p));
   return kOk;
 }
+
+// CTAs that share a row: several when the rows alone leave most of the machine idle
+static int row_cluster(int rows, int pitch) {
+  if (pitch < 1024) return 1;
+  if (rows * 8 <= sm_count() && pitch >= 2048) return 8;
+  return rows * 4 <= sm_count() ? 4 : 1;
+}
+
+template <typename P>
+using RowKernel = void (*)(P);
+
+// `k`: kernels for 1, 2, 3, 4 and 8 groups per thread; `k4`, `k8`: one group per thread in clusters of 4 and 8
+template <typename P>
+static int launch_rows(const RowKernel<P> (&k)[5], RowKernel<P> k4, RowKernel<P> k8, const P& p, int rows, cudaStream_t s) {
+  const int pitch = p.norm.pitch, cl = row_cluster(rows, pitch);
+  if (cl > 1) {
+    const int groups = (pitch / 4 + cl - 1) / cl;
+    if (groups <= kRnThreads) return launch_cluster(cl == 8 ? k8 : k4, p, rows, cl, (groups + 31) / 32 * 32, s);
+  }
+  const int g = row_groups(pitch);
+  B200_CHECK_CUDA(launch_pdl(k[g == 8 ? 4 : g - 1], dim3(rows), dim3(row_threads(pitch)), 0, s, p));
+  return kOk;
+}
+
+#define B200_ROW_KERNELS(K, P)                                                                                   \
+  const RowKernel<P> k[5] = {K<T, 1, 1>, K<T, 2, 1>, K<T, 3, 1>, K<T, 4, 1>, K<T, 8, 1>};                          \
+  return launch_rows<P>(k, K<T, 1, 4>, K<T, 1, 8>, p, rows, static_cast<cudaStream_t>(stream))
 
 }  // namespace b200
 
@@ -232,8 +330,7 @@ B200_API int b200_embed_norm(const long long* ids, const void* table, int rows, 
   p.norm = NormParams{width, pitch, center, eps, gain, bias, h};
   int rc = check_norm(p.norm);
   if (rc != kOk) return rc;
-  B200_DISPATCH_FLOAT(dtype, return launch_rows<T>(embed_norm_kernel<T, 1>, embed_norm_kernel<T, 2>, embed_norm_kernel<T, 3>, embed_norm_kernel<T, 4>,
-                                                   embed_norm_kernel<T, 8>, p, rows, static_cast<cudaStream_t>(stream)););
+  B200_DISPATCH_FLOAT(dtype, B200_ROW_KERNELS(embed_norm_kernel, EmbedParams););
 }
 
 // `states` holds n_prev earlier states of [rows, pitch] each, state_stride elements apart; with keep != 0 the new state
@@ -253,6 +350,5 @@ B200_API int b200_residual_norm(const void* a, const void* gate_a, const void* b
   p.norm = NormParams{width, pitch, center, eps, gain, bias, h};
   int rc = check_norm(p.norm);
   if (rc != kOk) return rc;
-  B200_DISPATCH_FLOAT(dtype, return launch_rows<T>(residual_norm_kernel<T, 1>, residual_norm_kernel<T, 2>, residual_norm_kernel<T, 3>, residual_norm_kernel<T, 4>,
-                                                   residual_norm_kernel<T, 8>, p, rows, static_cast<cudaStream_t>(stream)););
+  B200_DISPATCH_FLOAT(dtype, B200_ROW_KERNELS(residual_norm_kernel, ResidualParams););
 }
