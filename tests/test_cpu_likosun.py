@@ -143,3 +143,14 @@ def test_planted_mistakes_show_in_the_logits():
             assert moved(cfg, w) > 0.03, shift
     finally:
         ref.likosun.sink_softmax_ref = real
+
+
+def test_latent_split_choice():
+    from triton_distributed_b200.ops import choose_latent_splits
+    for batch in (1, 3, 8, 64, 300):
+        for rows in (1, 6, 16, 17, 33, 64, 200, 31 * 128):
+            for kv in (1, 64, 129, 2048, 16384, 131072):
+                splits, per_cta = choose_latent_splits(batch, rows, kv)
+                assert 1 <= splits <= 64 and splits <= (kv + 127) // 128 and per_cta in (16, 32, 64)
+                assert per_cta == 16 or rows > per_cta // 2
+    assert choose_latent_splits(8, 64, 16384) == (16, 64) and choose_latent_splits(1, 64, 2048)[1] == 16

@@ -559,11 +559,22 @@ def head_linear(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
 
 
 def choose_latent_splits(batch: int, rows: int, max_kv_len: int, sm_count: int = 148) -> tuple[int, int]:
-    """(splits, query rows per CTA) of the absorbed latent attention: one wave of CTAs (a CTA keeps most of an SM's shared
-    memory) over 128-key tiles."""
-    per_cta = 16 if rows <= 16 else 32 if rows <= 32 else 64
-    ctas = batch * ((rows + per_cta - 1) // per_cta)
-    return int(max(1, min(sm_count // max(ctas, 1), (max_kv_len + 255) // 256, 64))), per_cta
+    """(splits, query rows per CTA) of the absorbed latent attention, for `rows` query rows of each of `batch` sequences. One
+    wave of CTAs (each keeps most of an SM's shared memory); the estimate is microseconds per 128-key tile by rows per CTA, as
+    measured, plus what merging one more split costs."""
+    n_tiles = max(1, (max_kv_len + 127) // 128)
+    best = None
+    for per_cta, tile_us in ((16, 2.1), (32, 2.5), (64, 3.5)):
+        if per_cta > 16 and rows <= per_cta // 2:
+            continue
+        ctas = batch * ((rows + per_cta - 1) // per_cta)
+        tiles = -(-n_tiles // max(1, min(sm_count // ctas, n_tiles, 64)))
+        splits = -(-n_tiles // tiles)
+        waves = -(-ctas * splits // sm_count)
+        cost = waves * tiles * tile_us + 0.1 * splits
+        if best is None or cost < best[0]:
+            best = (cost, splits, per_cta)
+    return best[1], best[2]
 
 
 def latent_attention(q: torch.Tensor, cache: torch.Tensor, kv_lens: torch.Tensor, block_table: torch.Tensor, tokens: int,
