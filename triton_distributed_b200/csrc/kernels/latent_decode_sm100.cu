@@ -2,20 +2,20 @@
 //
 // The roles of the operands are swapped so that the few query rows (query token x head, N of them) are the narrow side of
 // every tcgen05.mma and no tensor-core row is padding:
-//   scores   S^T [128 keys, N]  = C [128 keys, rank] . Q [N, rank]^T        (C and Q K-major)
-//   values   O^T [rank, N]     += C^T [rank, 128 keys] . P [N, 128 keys]^T  (C^T is the same shared-memory tile read MN-major)
+//   scores   S^T [64 keys, N]   = C [64 keys, rank] . Q [N, rank]^T         (C and Q K-major)
+//   values   O^T [rank, N]     += C^T [rank, 64 keys] . P [N, 64 keys]^T   (C^T is the same shared-memory tile read MN-major)
 // so a latent row is loaded once and used twice, and the running output stays in tensor memory: lane = column of the latent
 // (in chunks of 128), column = query row.
 //
-// One CTA owns N query rows of a sequence and a range of 128-key tiles (split-KV; latent_combine merges, and adds the sink):
-//   warp 0     TMA producer: the Q tile once, then the tiles in slots of 128 keys x 128 columns (two 64-column swizzle atoms)
-//   warp 1     MMA issuer; a slot is given back as soon as its chunk of the output has been accumulated, so the next tile
-//              streams in while the rest of this one is still being multiplied
+// One CTA owns N query rows of a sequence and a range of 64-key tiles (split-KV; latent_combine merges, and adds the sink):
+//   warp 0     TMA producer: the Q tile once, then the tiles in slots of 64 keys x 128 columns (two 64-column swizzle atoms)
+//   warp 1     MMA issuer: the scores of tile j + 1 are computed while tile j is in the softmax (two score buffers, two P
+//              tiles); a slot is given back as soon as its chunk of the output has been accumulated
 //   warps 4-11 softmax, two threads per key of the tile (each has half of the query rows): exponentials against a reference
 //              maximum per row, P as 16-bit into a swizzled tile. The reference only moves when a score exceeds it by more than
 //              2^8: one vote per tile decides, and only then are the maxima reduced over the keys and the sums and the output in
 //              tensor memory rescaled. Sums and output share the reference, which cancels in the end.
-// The producer also asks L2 for the tile after next, so that a slot that becomes free is refilled at L2 latency.
+// The producer also asks L2 for tiles beyond the ring, so that a slot that becomes free is refilled at L2 latency.
 // Every barrier wait is bounded; on expiry the CTA unwinds through an abort flag and reports a status.
 #include "b200/host.h"
 #include "b200/primitives.cuh"
@@ -25,16 +25,16 @@
 
 namespace b200 {
 
-constexpr int kLdKeys = 128;              // keys per tile
-constexpr int kLdAtom = kLdKeys * 128;    // 128 keys x 64 columns: 16 KB
-constexpr int kLdSlot = 2 * kLdAtom;      // 128 keys x 128 columns
+constexpr int kLdKeys = 64;               // keys per tile
+constexpr int kLdAtom = kLdKeys * 128;    // 64 keys x 64 columns: 8 KB
+constexpr int kLdSlot = 2 * kLdAtom;      // 64 keys x 128 columns
 constexpr int kLdThreads = 384;
 constexpr float kLdSlack = 8.f;           // how far (log2) a score may exceed the reference before it moves
 constexpr int kLdSmemMax = 226 * 1024;
 
 constexpr int ld_fixed_bytes(int n, int rk) { return (rk / 64 + 2) * n * 128 + 1024 + 512 + n * 44; }
 constexpr int ld_slots(int n, int rk) {
-  const int fit = (kLdSmemMax - ld_fixed_bytes(n, rk)) / kLdSlot, want = 2 * (rk / 128) + 1;
+  const int fit = (kLdSmemMax - ld_fixed_bytes(n, rk)) / kLdSlot, want = 4 * (rk / 128) + 2 < 16 ? 4 * (rk / 128) + 2 : 16;
   return fit < want ? fit : want;
 }
 constexpr int ld_smem_bytes(int n, int rk) { return ld_fixed_bytes(n, rk) + ld_slots(n, rk) * kLdSlot; }
@@ -109,22 +109,22 @@ template <int N, int RK>
 __global__ void __launch_bounds__(kLdThreads, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant__ CUtensorMap tmQ, const LatentDecodeParams p) {
   constexpr int kPairs = RK / 128, kSlots = ld_slots(N, RK), kRowAtom = N * 128;
-  static_assert(kSlots >= kPairs && kSlots <= 16, "a tile must fit in the ring, the ring in the barrier layout");
-  constexpr uint32_t kTmemNeed = N * (1 + kPairs);
+  static_assert(kSlots >= 2 * kPairs && kSlots <= 16, "two tiles must fit in the ring, the ring in the barrier layout");
+  constexpr uint32_t kTmemNeed = N * (2 + kPairs);
   constexpr uint32_t kTmemCols = kTmemNeed <= 32 ? 32 : kTmemNeed <= 64 ? 64 : kTmemNeed <= 128 ? 128 : kTmemNeed <= 256 ? 256 : 512;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint8_t* ring = smem;                             // [kSlots][2 atoms][128 keys][128 B]
+  uint8_t* ring = smem;                             // [kSlots][2 atoms][64 keys][128 B]
   uint8_t* sQ = ring + kSlots * kLdSlot;            // [RK / 64 atoms][N rows][128 B]
-  uint8_t* sP = sQ + (RK / 64) * kRowAtom;          // [2 atoms][N rows][128 B], columns = keys
+  uint8_t* sP = sQ + (RK / 64) * kRowAtom;          // [2 tile parities][N rows][128 B], columns = keys
   uint64_t* bars = reinterpret_cast<uint64_t*>(sP + 2 * kRowAtom);
   uint64_t* full = bars;                // [kSlots]
   uint64_t* empty = bars + 16;          // [kSlots]
   uint64_t* q_full = bars + 32;
-  uint64_t* s_full = bars + 33;
-  uint64_t* p_full = bars + 34;
-  uint64_t* o_full = bars + 35;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 36);
+  uint64_t* s_full = bars + 33;         // [2] by tile parity
+  uint64_t* p_full = bars + 35;         // [2]
+  uint64_t* o_done = bars + 37;         // one phase per tile: its values have been accumulated
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 38);
   volatile uint32_t* abort_flag = tmem_slot + 1;
   float* xmax = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(bars) + 512);  // [4 warps][N]
   float* mref = xmax + 4 * N;                                                      // [N]
@@ -143,9 +143,11 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
       mbar_init(empty + i, 1);
     }
     mbar_init(q_full, 1);
-    mbar_init(s_full, 1);
-    mbar_init(p_full, 8);
-    mbar_init(o_full, 1);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(s_full + i, 1);
+      mbar_init(p_full + i, 8);
+    }
+    mbar_init(o_done, 1);
     *abort_flag = 0;
     mbar_fence_init();
     tma_prefetch_desc(&tmC);
@@ -168,7 +170,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
   tc_fence_before_sync();
   __syncthreads();
   tc_fence_after_sync();
-  const uint32_t tmem_base = *tmem_slot;  // columns [0, N) S^T, then kPairs x N columns of O^T
+  const uint32_t tmem_base = *tmem_slot;  // 2 x N columns of S^T, then kPairs x N columns of O^T
 
   if (warp == 0) {
     if (elect_one() && tile0 < tile1) {
@@ -176,26 +178,19 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
       mbar_expect_tx(q_full, (RK / 64) * kRowAtom);
       for (int a = 0; a < RK / 64; ++a) tma_load_2d(sQ + a * kRowAtom, &tmQ, q_full, a * 64, row_base);
       const int* table = p.block_table + static_cast<size_t>(b) * p.bt_stride;
-      // 64 keys lie in one page; a half beyond the last key repeats the first
-      auto slot_row = [&](int tile, int half) {
-        int key = tile * kLdKeys + 64 * half;
-        if (key >= n_keys) key = tile * kLdKeys;
-        return table[key / p.page] * p.page + key % p.page;
-      };
+      auto slot_row = [&](int tile) { return table[tile * kLdKeys / p.page] * p.page + tile * kLdKeys % p.page; };
       auto prefetch = [&](int tile) {
         if (tile >= tile1) return;
-        for (int half = 0; half < 2; ++half) {
-          const int row = slot_row(tile, half);
-          for (int a = 0; a < RK / 64; ++a)
-            if (a * 64 < p.pitch) tma_prefetch_l2_2d(&tmC, a * 64, row);
-        }
+        const int row = slot_row(tile);
+        for (int a = 0; a < RK / 64; ++a)
+          if (a * 64 < p.pitch) tma_prefetch_l2_2d(&tmC, a * 64, row);
       };
       int it = 0;
       bool ok = true;
-      prefetch(tile0 + 1);
+      prefetch(tile0 + 2);
       for (int tile = tile0; tile < tile1 && ok; ++tile) {
-        const int row[2] = {slot_row(tile, 0), slot_row(tile, 1)};
-        prefetch(tile + 2);
+        const int row = slot_row(tile);
+        prefetch(tile + 3);
         for (int pr = 0; pr < kPairs && ok; ++pr, ++it) {
           const int slot = it % kSlots;
           ok = mbar_wait(empty + slot, ((it / kSlots) & 1) ^ 1, abort_flag, timeout_ns);
@@ -203,79 +198,82 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
           mbar_expect_tx(full + slot, kLdSlot);
 #pragma unroll
           for (int a = 0; a < 2; ++a)
-#pragma unroll
-            for (int half = 0; half < 2; ++half)
-              tma_load_2d(ring + slot * kLdSlot + a * kLdAtom + half * (kLdAtom / 2), &tmC, full + slot, pr * 128 + a * 64, row[half]);
+            tma_load_2d(ring + slot * kLdSlot + a * kLdAtom, &tmC, full + slot, pr * 128 + a * 64, row);
         }
       }
     }
     __syncwarp();
   } else if (warp == 1) {
     if (elect_one() && tile0 < tile1) {
-      const uint32_t idesc_s = umma_idesc_f16(128, N, p.bf16 != 0);
-      const uint32_t idesc_o = idesc_s | (1u << 15);  // A is MN-major
+      const uint32_t idesc_s = umma_idesc_f16(kLdKeys, N, p.bf16 != 0);
+      const uint32_t idesc_o = umma_idesc_f16(128, N, p.bf16 != 0) | (1u << 15);  // A is MN-major
       bool ok = mbar_wait(q_full, 0, abort_flag, timeout_ns);
-      int it = 0;
-      for (int tile = tile0; tile < tile1 && ok; ++tile, it += kPairs) {
-        for (int pr = 0; pr < kPairs && ok; ++pr) {
-          const int slot = (it + pr) % kSlots;
-          ok = mbar_wait(full + slot, ((it + pr) / kSlots) & 1, abort_flag, timeout_ns);
-          if (!ok) break;
+      const int n = tile1 - tile0;
+      auto issue_scores = [&](int j) -> bool {  // tile j of this CTA
+        for (int pr = 0; pr < kPairs; ++pr) {
+          const int it = j * kPairs + pr, slot = it % kSlots;
+          if (!mbar_wait(full + slot, (it / kSlots) & 1, abort_flag, timeout_ns)) return false;
           tc_fence_after_sync();
 #pragma unroll
           for (int kk = 0; kk < 8; ++kk) {
             const uint64_t da = umma_desc_sw128_kmajor(smem_u32(ring + slot * kLdSlot + (kk >> 2) * kLdAtom)) + 2 * (kk & 3);
             const uint64_t db = umma_desc_sw128_kmajor(smem_u32(sQ + (2 * pr + (kk >> 2)) * kRowAtom)) + 2 * (kk & 3);
-            umma_f16(tmem_base, da, db, idesc_s, (pr | kk) != 0 ? 1u : 0u);
+            umma_f16(tmem_base + (j & 1) * N, da, db, idesc_s, (pr | kk) != 0 ? 1u : 0u);
           }
         }
+        umma_commit(s_full + (j & 1));  // also: the values of tile j - 2 have been accumulated
+        return true;
+      };
+      if (ok) ok = issue_scores(0);
+      for (int j = 0; j < n && ok; ++j) {
+        if (j + 1 < n) ok = issue_scores(j + 1);
         if (!ok) break;
-        umma_commit(s_full);  // also: every product of the tile before has been accumulated
-        ok = mbar_wait(p_full, (tile - tile0) & 1, abort_flag, timeout_ns);
+        ok = mbar_wait(p_full + (j & 1), (j >> 1) & 1, abort_flag, timeout_ns);
         if (!ok) break;
         tc_fence_after_sync();
         for (int pr = 0; pr < kPairs; ++pr) {
-          const int slot = (it + pr) % kSlots;
+          const int slot = (j * kPairs + pr) % kSlots;
 #pragma unroll
           for (int kk = 0; kk < kLdKeys / 16; ++kk) {
             const uint64_t da = umma_desc_sw128_mnmajor(smem_u32(ring + slot * kLdSlot + kk * 16 * 128), kLdAtom);
-            const uint64_t db = umma_desc_sw128_kmajor(smem_u32(sP + (kk >> 2) * kRowAtom)) + 2 * (kk & 3);
-            umma_f16(tmem_base + N * (1 + pr), da, db, idesc_o, (tile != tile0 || kk != 0) ? 1u : 0u);
+            const uint64_t db = umma_desc_sw128_kmajor(smem_u32(sP + (j & 1) * kRowAtom)) + 2 * kk;
+            umma_f16(tmem_base + N * (2 + pr), da, db, idesc_o, (j | kk) != 0 ? 1u : 0u);
           }
           umma_commit(empty + slot);
         }
+        umma_commit(o_done);
       }
-      if (ok) umma_commit(o_full);
     }
     __syncwarp();
   } else if (warp >= 4) {
     constexpr int kCols = N / 2;  // query rows of this thread
     const int w4 = warp & 3, half = (warp - 4) >> 2;
-    const int t = w4 * 32 + lane;  // key of the tile = TMEM lane
+    // a 64-row accumulator keeps rows 16 q ... 16 q + 15 in the first 16 lanes of quarter q: those threads own a key each
+    const bool live = lane < 16;
+    const int t = w4 * 16 + (lane & 15);  // key of the tile
     const int n0 = half * kCols;
     const uint32_t lane_base = tmem_base + (static_cast<uint32_t>(w4 * 32) << 16) + n0;
     float l[kCols];  // this key's share of the row sums
 #pragma unroll
     for (int i = 0; i < kCols; ++i) l[i] = 0.f;
     const int all_below = r0 + N <= n_rows ? first_limit + r0 / p.H : -1;  // keys up to here are visible to all rows
-    uint8_t* p_col = sP + (t >> 6) * kRowAtom + (t & 7) * 2;
-    const int p_chunk = (t & 63) >> 3;
+    uint8_t* p_col = sP + (t & 7) * 2;
+    const int p_chunk = t >> 3, n_mine = tile1 - tile0;
     bool ok = true;
-    int it = 0;
     // every thread meets the barriers of every tile, also after a pipeline wait has failed
-    for (int tile = tile0; tile < tile1; ++tile, it += kPairs) {
-      if (ok) ok = mbar_wait(s_full, (tile - tile0) & 1, abort_flag, timeout_ns);
+    for (int j = 0; j < n_mine; ++j) {
+      if (ok) ok = mbar_wait(s_full + (j & 1), (j >> 1) & 1, abort_flag, timeout_ns);
       ok = __all_sync(0xffffffffu, ok);
       tc_fence_after_sync();
-      const int key = tile * kLdKeys + t;
-      const bool masked = tile * kLdKeys + kLdKeys - 1 > all_below;
+      const int key0 = (tile0 + j) * kLdKeys, key = key0 + t;
+      const bool masked = key0 + kLdKeys - 1 > all_below;
       float s[kCols];
       bool exceeds = false;
       if (ok) {
-        tmem_ld_cols<kCols>(lane_base, s);
+        tmem_ld_cols<kCols>(lane_base + (j & 1) * N, s);
 #pragma unroll
         for (int i = 0; i < kCols; ++i) {
-          s[i] *= p.scale_log2e;
+          s[i] = live ? s[i] * p.scale_log2e : -INFINITY;
           if (masked) s[i] = key <= limit[n0 + i] ? s[i] : -INFINITY;
           exceeds |= s[i] > mref[n0 + i] + kLdSlack;  // (always when the row has no reference yet and sees this key)
         }
@@ -289,15 +287,19 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
           }
         }
         ld_softmax_bar();
-        if (half == 0 && t < N) {
-          const float mx = fmaxf(fmaxf(xmax[t], xmax[N + t]), fmaxf(xmax[2 * N + t], xmax[3 * N + t]));
-          const float old = mref[t];
+        const int r = threadIdx.x - 128;
+        if (r < N) {
+          const float mx = fmaxf(fmaxf(xmax[r], xmax[N + r]), fmaxf(xmax[2 * N + r], xmax[3 * N + r]));
+          const float old = mref[r];
           const bool up = mx > old + kLdSlack;
-          corr[t] = up ? ex2(old - mx) : 1.f;
-          if (up) mref[t] = mx;
+          corr[r] = up ? ex2(old - mx) : 1.f;
+          if (up) mref[r] = mx;
         }
         ld_softmax_bar();
-        if (ok && tile != tile0) {
+        if (ok && j > 0) ok = mbar_wait(o_done, (j - 1) & 1, abort_flag, timeout_ns);  // nothing is being added to the output
+        ok = __all_sync(0xffffffffu, ok);
+        tc_fence_after_sync();
+        if (ok && j > 0) {
 #pragma unroll
           for (int i = 0; i < kCols; ++i) l[i] *= corr[n0 + i];
 #pragma unroll 1
@@ -305,7 +307,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
 #pragma unroll
             for (int c = 0; c < kCols / 8; ++c) {
               uint32_t r[8];
-              const uint32_t at = lane_base + N * (1 + pr) + c * 8;
+              const uint32_t at = lane_base + N * (2 + pr) + c * 8;
               tmem_ld_32x8(at, r);
               tmem_ld_wait();
 #pragma unroll
@@ -321,14 +323,14 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
       for (int i = 0; i < kCols; ++i) {
         const int n = n0 + i;
         float pr = ex2(s[i] - mref[n]);
-        if (masked) pr = key <= limit[n] ? pr : 0.f;
+        if (masked) pr = live && key <= limit[n] ? pr : 0.f;
         l[i] += pr;
         const uint16_t h = p.bf16 ? __bfloat16_as_ushort(__float2bfloat16(pr)) : __half_as_ushort(__float2half(pr));
-        *reinterpret_cast<uint16_t*>(p_col + n * 128 + ((p_chunk ^ (n & 7)) << 4)) = h;
+        if (live) *reinterpret_cast<uint16_t*>(p_col + (j & 1) * kRowAtom + n * 128 + ((p_chunk ^ (n & 7)) << 4)) = h;
       }
-      if (key >= n_keys) {  // slots beyond the sequence may hold anything: their weight is zero, make the value zero too
+      if (live && key >= n_keys) {  // slots beyond the sequence may hold anything: their weight is zero, make the value zero too
         for (int pr = 0; pr < kPairs; ++pr) {
-          uint4* dst = reinterpret_cast<uint4*>(ring + ((it + pr) % kSlots) * kLdSlot + half * kLdAtom + t * 128);
+          uint4* dst = reinterpret_cast<uint4*>(ring + ((j * kPairs + pr) % kSlots) * kLdSlot + half * kLdAtom + t * 128);
 #pragma unroll
           for (int i = 0; i < 8; ++i) dst[i] = make_uint4(0, 0, 0, 0);
         }
@@ -336,7 +338,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
       tc_fence_before_sync();     // this thread's TMEM accesses are done
       fence_view_async_shared();  // its shared-memory writes are visible to the tensor core
       __syncwarp();
-      if (lane == 0) mbar_arrive(p_full);
+      if (lane == 0) mbar_arrive(p_full + (j & 1));
     }
     // ---- row sums over the keys, then the normalised partial output and its log-sum-exp
 #pragma unroll
@@ -345,24 +347,25 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
       if (lane == 0) xsum[w4 * N + n0 + i] = sum;
     }
     ld_softmax_bar();
-    if (half == 0 && t < N) {
-      const float sum = (xsum[t] + xsum[N + t]) + (xsum[2 * N + t] + xsum[3 * N + t]);
-      corr[t] = sum > 0.f ? 1.f / sum : 0.f;
-      if (r0 + t < n_rows)
-        p.lse_part[static_cast<size_t>(row_base + t) * p.splits + split] =
-            sum > 0.f ? (mref[t] + log2f(sum)) * 0.6931471805599453f : -INFINITY;
+    const int r = threadIdx.x - 128;
+    if (r < N) {
+      const float sum = (xsum[r] + xsum[N + r]) + (xsum[2 * N + r] + xsum[3 * N + r]);
+      corr[r] = sum > 0.f ? 1.f / sum : 0.f;
+      if (r0 + r < n_rows)
+        p.lse_part[static_cast<size_t>(row_base + r) * p.splits + split] =
+            sum > 0.f ? (mref[r] + log2f(sum)) * 0.6931471805599453f : -INFINITY;
     }
     ld_softmax_bar();
     if (tile0 < tile1) {
-      if (ok) ok = mbar_wait(o_full, 0, abort_flag, timeout_ns);
+      if (ok) ok = mbar_wait(o_done, (n_mine - 1) & 1, abort_flag, timeout_ns);
       ok = __all_sync(0xffffffffu, ok);
       tc_fence_after_sync();
       if (ok) {
 #pragma unroll 1
         for (int pr = 0; pr < kPairs; ++pr) {
-          const int col = pr * 128 + t;
+          const int col = pr * 128 + w4 * 32 + lane;
           float o[kCols];
-          tmem_ld_cols<kCols>(lane_base + N * (1 + pr), o);
+          tmem_ld_cols<kCols>(lane_base + N * (2 + pr), o);
 #pragma unroll
           for (int i = 0; i < kCols; ++i)
             if (r0 + n0 + i < n_rows && col < p.pitch)
