@@ -151,6 +151,6 @@ def test_latent_split_choice():
         for rows in (1, 6, 16, 17, 33, 64, 200, 31 * 128):
             for kv in (1, 64, 129, 2048, 16384, 131072):
                 splits, per_cta = choose_latent_splits(batch, rows, kv)
-                assert 1 <= splits <= 64 and splits <= (kv + 127) // 128 and per_cta in (16, 32, 64)
+                assert 1 <= splits <= 64 and splits <= (kv + 63) // 64 and per_cta in (16, 32, 64)
                 assert per_cta == 16 or rows > per_cta // 2
-    assert choose_latent_splits(8, 64, 16384) == (16, 64) and choose_latent_splits(1, 64, 2048)[1] == 16
+    assert choose_latent_splits(8, 64, 16384) == (18, 64) and choose_latent_splits(1, 16, 2048) == (32, 16)

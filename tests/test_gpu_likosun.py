@@ -161,8 +161,8 @@ def _absorbed_ref(q, c, sink, scale, first):
     return ref.latent_attention_ref(q, c, eye, eye, sink, scale, first)
 
 
-@pytest.mark.parametrize("dtype,variant", [(torch.bfloat16, "tc"), (torch.float16, "tc"), (torch.bfloat16, "mma"), (torch.float16, "mma"),
-                                           (torch.bfloat16, "plain"), (torch.float32, "plain")])
+@pytest.mark.parametrize("dtype,variant", [(torch.bfloat16, "tc"), (torch.float16, "tc"), (torch.bfloat16, "plain"),
+                                           (torch.float32, "plain")])
 @pytest.mark.parametrize("H,S,rank,lens,splits,page", [
     (1, 1, 8, [1, 2, 63, 64, 65], 1, 64), (6, 1, 72, [300, 17, 128, 129], 3, 64), (16, 1, 512, [700, 64, 1], 5, 128),
     (3, 2, 40, [2, 65, 66, 130], 2, 64), (5, 7, 136, [7, 8, 70, 134], 2, 192), (33, 3, 264, [200, 3], 4, 64), (4, 31, 384, [31, 95], 1, 64),
@@ -204,7 +204,7 @@ def test_latent_attention_with_scores_that_grow():
     c, q = c.bfloat16(), q.bfloat16()
     cache, table = _paged([c], rank, 64, torch.bfloat16)
     want = _absorbed_ref(q.double(), c.double(), torch.zeros(H, dtype=torch.float64), 1.0, n - 1)
-    for variant in ("tc", "mma", "plain"):
+    for variant in ("tc", "plain"):
         for splits in (1, 3):
             out = ops.latent_attention(q.cuda(), cache, torch.tensor([n], dtype=torch.int32, device="cuda"), table, 1, 1.0,
                                        torch.zeros(H, device="cuda"), splits, variant=variant)
@@ -212,7 +212,7 @@ def test_latent_attention_with_scores_that_grow():
     ops.check_pipeline_status()
 
 
-@pytest.mark.parametrize("variant", ["tc", "mma", "plain"])
+@pytest.mark.parametrize("variant", ["tc", "plain"])
 @pytest.mark.parametrize("kv_len,S", [(1, 1), (64, 1), (65, 1), (128, 5), (190, 3), (321, 1)])
 def test_latent_attention_sees_exactly_the_keys_up_to_its_own(variant, kv_len, S):
     """One key at a time gets a score that dwarfs the others: rows whose position is at or after it return its latent, rows

@@ -5,9 +5,7 @@
 //   latent_prep       RMS norm of the down-projected row, written to the cache slot of its token; squared-relu of the
 //                     feed-forward's up-projection, which sits in the same GEMM output
 //   head_linear       y[t, h, :] = W[h] x[t, h, :]  (per-head GEMM: Wk^T on the query, Wv on the attended latent)
-//   latent_attention  split-KV attention over the paged latents. One CTA owns 16 or 32 rows (query token x head) of a
-//                     sequence and a range of 64-token tiles; a tile is loaded into shared memory once and serves as keys
-//                     (scores) and as values. The M side is a handful of heads, so it uses warp-level m16n8k16 products.
+//   attention over the paged latents, which serve as keys and as values: latent_decode_sm100.cu (split-KV partial results)
 //   latent_combine    merges the splits; a per-head sink logit joins the softmax denominator here, once
 //   latent_attention_plain   one warp per row, any rank, any storage type (the 32-bit mode and shapes outside the above)
 // Many query tokens go through prefill_attn_sm100.cu on expanded keys and values instead.
@@ -182,214 +180,11 @@ struct LatentParams {
   const void* cache;       // [blocks, page, pitch]
   const int* block_table;  // [B, bt_stride]
   const int* kv_lens;      // [B] keys in the cache, the S new ones included
-  float* o_part;           // [B * S * H, splits, pitch]
-  float* lse_part;         // [B * S * H, splits] natural log
-  const float* sink;       // [H] or null (latent_attention_plain)
-  void* out;               // [B * S * H, pitch]  (latent_attention_plain)
-  int bt_stride, page, H, S, pitch, splits;
-  float scale, scale_log2e;
+  const float* sink;       // [H] or null
+  void* out;               // [B * S * H, pitch]
+  int bt_stride, page, H, S, pitch;
+  float scale;
 };
-
-constexpr int kLtKeys = 64;                 // keys per tile; the page size is a multiple of it
-constexpr int kLtScorePitch = kLtKeys + 4;  // floats
-constexpr int kLtProbPitch = kLtKeys + 8;   // 16-bit elements
-
-template <int RM, int RK>
-constexpr int latent_smem_bytes() {
-  return (16 * RM + 2 * kLtKeys) * (RK + 8) * 2 + 16 * RM * (kLtScorePitch * 4 + kLtProbPitch * 2 + 8);
-}
-
-// RM: 16-row tiles per CTA (1 or 2); RK: rank rounded up to a multiple of 128 (the padding columns are zero in shared
-// memory). 8 warps. Scores: a warp owns 16 keys x one row tile (RM = 2) or 8 keys (RM = 1). Values: a warp owns RK / 8
-// columns of all rows. A row stride of RK + 8 elements puts the eight rows of an ldmatrix into different banks.
-template <bool BF16, int RM, int RK>
-__global__ void __launch_bounds__(256, 1) latent_attention_kernel(const LatentParams p) {
-  constexpr int kRows = 16 * RM, kPitch = RK + 8, kNP = RK / 128;
-  extern __shared__ __align__(16) uint8_t smem[];
-  uint16_t* sq = reinterpret_cast<uint16_t*>(smem);
-  uint16_t* sc = sq + kRows * kPitch;                                  // [2][64][kPitch]
-  float* ss = reinterpret_cast<float*>(sc + 2 * kLtKeys * kPitch);     // [kRows][68]
-  uint16_t* sp = reinterpret_cast<uint16_t*>(ss + kRows * kLtScorePitch);  // [kRows][72]
-  float* corr = reinterpret_cast<float*>(sp + kRows * kLtProbPitch);   // [kRows]
-  float* inv_l = corr + kRows;                                         // [kRows]
-
-  const int split = blockIdx.x, b = blockIdx.z, r0 = blockIdx.y * kRows;
-  const int n_rows = p.S * p.H;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  griddep_launch_dependents();
-  griddep_wait();
-  const int kv_len = p.kv_lens[b];
-  const int first_key_limit = kv_len - p.S;  // last key of token 0; token i adds i
-  // keys any row of this block attends, cut into `splits` ranges of whole tiles
-  const int last_tok = (min(r0 + kRows, n_rows) - 1) / p.H;
-  const int n_keys = max(0, min(kv_len, first_key_limit + last_tok + 1));
-  const int n_tiles = (n_keys + kLtKeys - 1) / kLtKeys;
-  const int per = (n_tiles + p.splits - 1) / p.splits;
-  const int tile0 = min(n_tiles, split * per), tile1 = min(n_tiles, tile0 + per);
-  const size_t row_base = static_cast<size_t>(b) * n_rows;
-  if (tile0 >= tile1) {
-    for (int r = threadIdx.x; r < kRows; r += blockDim.x)
-      if (r0 + r < n_rows) p.lse_part[(row_base + r0 + r) * p.splits + split] = -INFINITY;
-    return;
-  }
-  const uint16_t* q = static_cast<const uint16_t*>(p.q);
-  const uint16_t* cache = static_cast<const uint16_t*>(p.cache);
-  const int* table = p.block_table + static_cast<size_t>(b) * p.bt_stride;
-
-  auto load_tile = [&](int tile, int stage) {
-    const int j0 = tile * kLtKeys;
-    const size_t base = static_cast<size_t>(table[j0 / p.page]) * p.page + j0 % p.page;
-    for (int i = threadIdx.x; i < kLtKeys * (RK / 8); i += 256) {
-      const int key = i / (RK / 8), c = (i - key * (RK / 8)) * 8;
-      const bool in = j0 + key < n_keys && c < p.pitch;
-      cp_async_16(static_cast<uint32_t>(__cvta_generic_to_shared(sc + (stage * kLtKeys + key) * kPitch + c)),
-                  in ? cache + (base + key) * p.pitch + c : cache, in ? 16 : 0);
-    }
-    cp_async_commit();
-  };
-  for (int i = threadIdx.x; i < kRows * (RK / 8); i += 256) {
-    const int r = i / (RK / 8), c = (i - r * (RK / 8)) * 8;
-    const bool in = r0 + r < n_rows && c < p.pitch;
-    cp_async_16(static_cast<uint32_t>(__cvta_generic_to_shared(sq + r * kPitch + c)), in ? q + (row_base + r0 + r) * p.pitch + c : q,
-                in ? 16 : 0);
-  }
-  load_tile(tile0, 0);  // one group with the query rows
-
-  constexpr int kRowsPerWarp = kRows / 8;
-  float m_run[kRowsPerWarp], l_run[kRowsPerWarp];
-#pragma unroll
-  for (int i = 0; i < kRowsPerWarp; ++i) m_run[i] = -INFINITY, l_run[i] = 0.f;
-  float acc[RM][2 * kNP][4] = {};
-  const int g = lane >> 2, tq = lane & 3;
-  const int col0 = warp * (RK / 8);
-
-  for (int tile = tile0; tile < tile1; ++tile) {
-    const int stage = (tile - tile0) & 1;
-    cp_async_wait<0>();
-    __syncthreads();  // this tile has landed for every thread, and the other stage is no longer being read
-    if (tile + 1 < tile1) load_tile(tile + 1, stage ^ 1);
-    const uint16_t* ct = sc + stage * kLtKeys * kPitch;
-    // ---- scores
-    {
-      const int mt = RM == 2 ? warp >> 2 : 0;
-      const uint32_t qa = static_cast<uint32_t>(__cvta_generic_to_shared(
-          sq + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kPitch + (lane >> 4) * 8));
-      if (RM == 2) {
-        const int kg = (warp & 3) * 16;
-        const uint32_t ka = static_cast<uint32_t>(__cvta_generic_to_shared(
-            ct + (kg + (lane & 7) + ((lane >> 4) & 1) * 8) * kPitch + ((lane >> 3) & 1) * 8));
-        float s[2][4] = {};
-#pragma unroll 8
-        for (int kk = 0; kk < RK / 16; ++kk) {
-          uint32_t a[4], b0, b1, b2, b3;
-          ldmatrix_x4(qa + kk * 32, a[0], a[1], a[2], a[3]);
-          ldmatrix_x4(ka + kk * 32, b0, b1, b2, b3);
-          mma16816<BF16>(s[0], a, b0, b1);
-          mma16816<BF16>(s[1], a, b2, b3);
-        }
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          float* dst = ss + (mt * 16 + g) * kLtScorePitch + kg + n * 8 + 2 * tq;
-          dst[0] = s[n][0]; dst[1] = s[n][1];
-          dst[8 * kLtScorePitch] = s[n][2]; dst[8 * kLtScorePitch + 1] = s[n][3];
-        }
-      } else {
-        const int kg = warp * 8;
-        const uint32_t ka = static_cast<uint32_t>(__cvta_generic_to_shared(ct + (kg + (lane & 7)) * kPitch + (lane >> 3) * 8));
-        float s[2][4] = {};
-#pragma unroll 4
-        for (int kk = 0; kk < RK / 32; ++kk) {
-          uint32_t a[4], b0, b1, b2, b3;
-          ldmatrix_x4(ka + kk * 64, b0, b1, b2, b3);
-          ldmatrix_x4(qa + kk * 64, a[0], a[1], a[2], a[3]);
-          mma16816<BF16>(s[0], a, b0, b1);
-          ldmatrix_x4(qa + kk * 64 + 32, a[0], a[1], a[2], a[3]);
-          mma16816<BF16>(s[1], a, b2, b3);
-        }
-        float* dst = ss + g * kLtScorePitch + kg + 2 * tq;
-        dst[0] = s[0][0] + s[1][0]; dst[1] = s[0][1] + s[1][1];
-        dst[8 * kLtScorePitch] = s[0][2] + s[1][2]; dst[8 * kLtScorePitch + 1] = s[0][3] + s[1][3];
-      }
-    }
-    __syncthreads();
-    // ---- online softmax, one row per warp at a time
-#pragma unroll
-    for (int i = 0; i < kRowsPerWarp; ++i) {
-      const int r = warp * kRowsPerWarp + i;
-      const int limit = r0 + r < n_rows ? first_key_limit + (r0 + r) / p.H - tile * kLtKeys : -1;  // last visible key of the tile
-      const float s0 = lane <= limit ? ss[r * kLtScorePitch + lane] * p.scale_log2e : -INFINITY;
-      const float s1 = lane + 32 <= limit ? ss[r * kLtScorePitch + lane + 32] * p.scale_log2e : -INFINITY;
-      const float m_new = fmaxf(m_run[i], warp_max(fmaxf(s0, s1)));
-      const float base = m_new == -INFINITY ? 0.f : m_new;
-      const float p0 = exp2f(s0 - base), p1 = exp2f(s1 - base), c = exp2f(m_run[i] - base);
-      l_run[i] = l_run[i] * c + warp_sum(p0 + p1);
-      m_run[i] = m_new;
-      const uint32_t packed = BF16 ? pack_bf16x2(p0, p1) : pack_f16x2(p0, p1);
-      sp[r * kLtProbPitch + lane] = static_cast<uint16_t>(packed & 0xffffu);
-      sp[r * kLtProbPitch + lane + 32] = static_cast<uint16_t>(packed >> 16);
-      if (lane == 0) corr[r] = c;
-    }
-    __syncthreads();
-    // ---- values
-#pragma unroll
-    for (int mt = 0; mt < RM; ++mt) {
-      const float c0 = corr[mt * 16 + g], c1 = corr[mt * 16 + g + 8];
-#pragma unroll
-      for (int n = 0; n < 2 * kNP; ++n) {
-        acc[mt][n][0] *= c0; acc[mt][n][1] *= c0;
-        acc[mt][n][2] *= c1; acc[mt][n][3] *= c1;
-      }
-    }
-#pragma unroll
-    for (int kk = 0; kk < kLtKeys / 16; ++kk) {
-      uint32_t a[RM][4];
-#pragma unroll
-      for (int mt = 0; mt < RM; ++mt)
-        ldmatrix_x4(static_cast<uint32_t>(__cvta_generic_to_shared(
-                        sp + (mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kLtProbPitch + kk * 16 + (lane >> 4) * 8)),
-                    a[mt][0], a[mt][1], a[mt][2], a[mt][3]);
-#pragma unroll
-      for (int n = 0; n < kNP; ++n) {
-        uint32_t b0, b1, b2, b3;
-        ldmatrix_x4_trans(static_cast<uint32_t>(__cvta_generic_to_shared(
-                              ct + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kPitch + col0 + n * 16 + (lane >> 4) * 8)),
-                          b0, b1, b2, b3);
-#pragma unroll
-        for (int mt = 0; mt < RM; ++mt) {
-          mma16816<BF16>(acc[mt][2 * n], a[mt], b0, b1);
-          mma16816<BF16>(acc[mt][2 * n + 1], a[mt], b2, b3);
-        }
-      }
-    }
-  }
-  // ---- normalised partial result and log-sum-exp of this split
-#pragma unroll
-  for (int i = 0; i < kRowsPerWarp; ++i) {
-    const int r = warp * kRowsPerWarp + i;
-    if (lane == 0) {
-      inv_l[r] = l_run[i] > 0.f ? 1.f / l_run[i] : 0.f;
-      if (r0 + r < n_rows)
-        p.lse_part[(row_base + r0 + r) * p.splits + split] =
-            l_run[i] > 0.f ? (m_run[i] + log2f(l_run[i])) * 0.6931471805599453f : -INFINITY;
-    }
-  }
-  __syncthreads();
-#pragma unroll
-  for (int mt = 0; mt < RM; ++mt)
-#pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int r = mt * 16 + g + 8 * half;
-      if (r0 + r >= n_rows) continue;
-      const float il = inv_l[r];
-      float* dst = p.o_part + ((row_base + r0 + r) * p.splits + split) * p.pitch;
-#pragma unroll
-      for (int n = 0; n < 2 * kNP; ++n) {
-        const int c = col0 + n * 8 + 2 * tq;
-        if (c < p.pitch)
-          *reinterpret_cast<float2*>(dst + c) = make_float2(acc[mt][n][2 * half] * il, acc[mt][n][2 * half + 1] * il);
-      }
-    }
-}
 
 // grid (ceil(pitch / 128), rows): merge of the splits. The sink is one more term exp(sink) of the denominator without a
 // value: the merged row is scaled by exp(lse) / (exp(lse) + exp(sink)).
@@ -464,29 +259,6 @@ __global__ void __launch_bounds__(128) latent_attention_plain_kernel(const Laten
   for (int i = lane; i < p.pitch; i += 32) static_cast<T*>(p.out)[row * p.pitch + i] = from_float<T>(o[i] * inv);
 }
 
-template <bool BF16, int RM, int RK>
-static int launch_latent(const LatentParams& p, int B, cudaStream_t s) {
-  constexpr int smem = latent_smem_bytes<RM, RK>();
-  static bool configured[64] = {false};
-  int dev = 0;
-  B200_CHECK_CUDA(cudaGetDevice(&dev));
-  if (!configured[dev & 63]) {
-    B200_CHECK_CUDA(cudaFuncSetAttribute(latent_attention_kernel<BF16, RM, RK>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-    configured[dev & 63] = true;
-  }
-  const dim3 grid(p.splits, (p.S * p.H + 16 * RM - 1) / (16 * RM), B);
-  B200_REQUIRE(grid.y <= 65535, "too many query rows (%d) for the absorbed attention", p.S * p.H);
-  B200_CHECK_CUDA(launch_pdl(latent_attention_kernel<BF16, RM, RK>, grid, dim3(256), smem, s, p));
-  return kOk;
-}
-template <bool BF16, int RM>
-static int launch_latent_rank(const LatentParams& p, int B, cudaStream_t s) {
-  if (p.pitch <= 128) return launch_latent<BF16, RM, 128>(p, B, s);
-  if (p.pitch <= 256) return launch_latent<BF16, RM, 256>(p, B, s);
-  if (p.pitch <= 384) return launch_latent<BF16, RM, 384>(p, B, s);
-  return launch_latent<BF16, RM, 512>(p, B, s);
-}
-
 }  // namespace b200
 
 using namespace b200;
@@ -536,27 +308,11 @@ static int fill_latent(LatentParams& p, const void* q, const void* cache, const 
   B200_REQUIRE(pitch % 8 == 0, "the latent row (%d elements) must be a multiple of 8", pitch);
   memset(&p, 0, sizeof(p));
   p.q = q; p.cache = cache; p.block_table = block_table; p.kv_lens = kv_lens; p.bt_stride = bt_stride; p.page = page;
-  p.H = H; p.S = S; p.pitch = pitch; p.scale = scale; p.scale_log2e = scale * 1.4426950408889634f;
+  p.H = H; p.S = S; p.pitch = pitch; p.scale = scale;
   return kOk;
 }
 
-// Split partials: o_part fp32 [B * S * H, splits, pitch], lse_part fp32 [B * S * H, splits]; merge with b200_latent_combine.
-B200_API int b200_latent_attention(const void* q, const void* cache, const int* block_table, int bt_stride, const int* kv_lens, int B,
-                                   int S, int H, int pitch, int page, float scale, int splits, float* o_part, float* lse_part,
-                                   int dtype, void* stream) {
-  LatentParams p;
-  int rc = fill_latent(p, q, cache, block_table, bt_stride, kv_lens, B, S, H, pitch, page, scale);
-  if (rc != kOk) return rc;
-  B200_REQUIRE(dtype == kBF16 || dtype == kF16, "latent attention supports bf16 / f16 (b200_latent_attention_plain takes fp32)");
-  B200_REQUIRE(pitch <= 512, "latent attention handles ranks up to 512, got %d", pitch);
-  B200_REQUIRE(page % kLtKeys == 0, "the page size (%d) must be a multiple of %d", page, kLtKeys);
-  B200_REQUIRE(splits >= 1 && o_part && lse_part, "latent attention needs its partial buffers");
-  p.splits = splits; p.o_part = o_part; p.lse_part = lse_part;
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dtype == kBF16) return S * H > 16 ? launch_latent_rank<true, 2>(p, B, s) : launch_latent_rank<true, 1>(p, B, s);
-  return S * H > 16 ? launch_latent_rank<false, 2>(p, B, s) : launch_latent_rank<false, 1>(p, B, s);
-}
-
+// Merges partial results o_part fp32 [rows, splits, pitch] with log-sum-exps lse_part fp32 [rows, splits]; row % H is the head.
 B200_API int b200_latent_combine(const float* o_part, const float* lse_part, const float* sink, int rows, int H, int splits, int pitch,
                                  void* out, int dtype, void* stream) {
   if (rows <= 0) return kOk;

@@ -11,8 +11,9 @@
 //   warp 0     TMA producer: the Q tile once, then the tiles in slots of 64 keys x 128 columns (two 64-column swizzle atoms)
 //   warp 1     MMA issuer: the scores of tile j + 1 are computed while tile j is in the softmax (two score buffers, two P
 //              tiles); a slot is given back as soon as its chunk of the output has been accumulated
-//   warps 4-11 softmax, two threads per key of the tile (each has half of the query rows): exponentials against a reference
-//              maximum per row, P as 16-bit into a swizzled tile. The reference only moves when a score exceeds it by more than
+//   warps 4-11 softmax, half of the query rows each: exponentials against a reference maximum per row, P as 16-bit into a
+//              swizzled tile. The scores are read in the 16-lane x 256-bit shape (a 64-row accumulator occupies 16 lanes of every
+//              quarter), whose fragments stmatrix writes transposed, eight keys of a row at a time. The reference only moves when a score exceeds it by more than
 //              2^8: one vote per tile decides, and only then are the maxima reduced over the keys and the sums and the output in
 //              tensor memory rescaled. Sums and output share the reference, which cancels in the end.
 // The producer also asks L2 for tiles beyond the ring, so that a slot that becomes free is refilled at L2 latency.
@@ -57,11 +58,6 @@ __device__ __forceinline__ uint64_t umma_desc_sw128_mnmajor(uint32_t smem_addr, 
   d |= static_cast<uint64_t>(mn_stride >> 4) << 16;
   return d;
 }
-__device__ __forceinline__ float redux_max(float v) {
-  float r;
-  asm volatile("redux.sync.max.f32 %0, %1, 0xffffffff;" : "=f"(r) : "f"(v));
-  return r;
-}
 __device__ __forceinline__ float ex2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
@@ -99,6 +95,35 @@ __device__ __forceinline__ void tmem_ld_cols(uint32_t taddr, float (&v)[kCols]) 
   tmem_ld_wait();
 #pragma unroll
   for (int i = 0; i < kCols; ++i) v[i] = __uint_as_float(r[i]);
+}
+// 16 lanes x 8 columns per group of four registers, as an m16n8 fragment: registers 0, 1 hold lane (thread / 4), columns
+// 2 (thread % 4) and the next; registers 2, 3 the same columns of lane (thread / 4) + 8
+template <int kGroups>
+__device__ __forceinline__ void tmem_ld_frag(uint32_t taddr, float (&v)[4 * kGroups]) {
+  uint32_t r[4 * kGroups];
+  if constexpr (kGroups == 1)
+    asm volatile("tcgen05.ld.sync.aligned.16x256b.x1.b32 {%0, %1, %2, %3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(taddr) : "memory");
+  else if constexpr (kGroups == 2)
+    asm volatile("tcgen05.ld.sync.aligned.16x256b.x2.b32 {%0, %1, %2, %3, %4, %5, %6, %7}, [%8];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7])
+                 : "r"(taddr) : "memory");
+  else
+    asm volatile("tcgen05.ld.sync.aligned.16x256b.x4.b32 {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
+                   "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+                 : "r"(taddr) : "memory");
+  tmem_ld_wait();
+#pragma unroll
+  for (int i = 0; i < 4 * kGroups; ++i) v[i] = __uint_as_float(r[i]);
+}
+// 8 x 8 fragments stored transposed; lanes 8 m ... 8 m + 7 address the rows of matrix m
+__device__ __forceinline__ void stmatrix_x2_trans(uint32_t addr, uint32_t r0, uint32_t r1) {
+  asm volatile("stmatrix.sync.aligned.m8n8.x2.trans.shared.b16 [%0], {%1, %2};" ::"r"(addr), "r"(r0), "r"(r1) : "memory");
+}
+__device__ __forceinline__ void stmatrix_x4_trans(uint32_t addr, uint32_t r0, uint32_t r1, uint32_t r2, uint32_t r3) {
+  asm volatile("stmatrix.sync.aligned.m8n8.x4.trans.shared.b16 [%0], {%1, %2, %3, %4};" ::"r"(addr), "r"(r0), "r"(r1), "r"(r2), "r"(r3)
+               : "memory");
 }
 __device__ __forceinline__ void tma_prefetch_l2_2d(const CUtensorMap* map, int x, int y) {
   asm volatile("cp.async.bulk.prefetch.tensor.2d.L2.global [%0, {%1, %2}];" ::"l"(map), "r"(x), "r"(y) : "memory");
@@ -246,44 +271,59 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
     }
     __syncwarp();
   } else if (warp >= 4) {
-    constexpr int kCols = N / 2;  // query rows of this thread
+    constexpr int kCols = N / 2, kGroups = kCols / 8;  // query rows of this warp, in groups of eight
     const int w4 = warp & 3, half = (warp - 4) >> 2;
-    // a 64-row accumulator keeps rows 16 q ... 16 q + 15 in the first 16 lanes of quarter q: those threads own a key each
-    const bool live = lane < 16;
-    const int t = w4 * 16 + (lane & 15);  // key of the tile
-    const int n0 = half * kCols;
+    // a 64-row accumulator keeps keys 16 q ... 16 q + 15 in the first 16 lanes of quarter q: this thread has keys kt and kt + 8
+    // of the tile and query rows n0 + 8 g + 2 (lane % 4) + {0, 1} for every group g
+    const int kt = w4 * 16 + (lane >> 2);
+    const int n0 = half * kCols, nq = n0 + 2 * (lane & 3);
     const uint32_t lane_base = tmem_base + (static_cast<uint32_t>(w4 * 32) << 16) + n0;
-    float l[kCols];  // this key's share of the row sums
+    float l[2 * kGroups];  // share of these keys in the row sums
 #pragma unroll
-    for (int i = 0; i < kCols; ++i) l[i] = 0.f;
+    for (int i = 0; i < 2 * kGroups; ++i) l[i] = 0.f;
     const int all_below = r0 + N <= n_rows ? first_limit + r0 / p.H : -1;  // keys up to here are visible to all rows
-    uint8_t* p_col = sP + (t & 7) * 2;
-    const int p_chunk = t >> 3, n_mine = tile1 - tile0;
+    // row of this lane's matrix for stmatrix: matrices alternate between the key blocks (8 keys) and go on to the next group
+    const int p_chunk = w4 * 2 + ((lane >> 3) & 1), p_row = n0 + 8 * (lane >> 4) + (lane & 7);
+    const uint32_t p_addr = smem_u32(sP + p_row * 128 + ((p_chunk ^ (lane & 7)) << 4));
+    const int n_mine = tile1 - tile0;
     bool ok = true;
     // every thread meets the barriers of every tile, also after a pipeline wait has failed
     for (int j = 0; j < n_mine; ++j) {
       if (ok) ok = mbar_wait(s_full + (j & 1), (j >> 1) & 1, abort_flag, timeout_ns);
       ok = __all_sync(0xffffffffu, ok);
       tc_fence_after_sync();
-      const int key0 = (tile0 + j) * kLdKeys, key = key0 + t;
+      const int key0 = (tile0 + j) * kLdKeys;
       const bool masked = key0 + kLdKeys - 1 > all_below;
-      float s[kCols];
+      float s[4 * kGroups];  // [group][key block][row of the pair]
       bool exceeds = false;
       if (ok) {
-        tmem_ld_cols<kCols>(lane_base + (j & 1) * N, s);
+        tmem_ld_frag<kGroups>(lane_base + (j & 1) * N, s);
 #pragma unroll
-        for (int i = 0; i < kCols; ++i) {
-          s[i] = live ? s[i] * p.scale_log2e : -INFINITY;
-          if (masked) s[i] = key <= limit[n0 + i] ? s[i] : -INFINITY;
-          exceeds |= s[i] > mref[n0 + i] + kLdSlack;  // (always when the row has no reference yet and sees this key)
+        for (int g = 0; g < kGroups; ++g) {
+          const float2 m = *reinterpret_cast<const float2*>(mref + nq + 8 * g);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[4 * g + e] *= p.scale_log2e;
+          if (masked) {
+            const int2 lim = *reinterpret_cast<const int2*>(limit + nq + 8 * g);
+            const int key = key0 + kt;
+            s[4 * g] = key <= lim.x ? s[4 * g] : -INFINITY;
+            s[4 * g + 1] = key <= lim.y ? s[4 * g + 1] : -INFINITY;
+            s[4 * g + 2] = key + 8 <= lim.x ? s[4 * g + 2] : -INFINITY;
+            s[4 * g + 3] = key + 8 <= lim.y ? s[4 * g + 3] : -INFINITY;
+          }
+          // (always when a row has no reference yet and sees a key)
+          exceeds |= fmaxf(s[4 * g], s[4 * g + 2]) > m.x + kLdSlack || fmaxf(s[4 * g + 1], s[4 * g + 3]) > m.y + kLdSlack;
         }
       }
       if (ld_softmax_any(exceeds)) {
         if (ok) {
 #pragma unroll
-          for (int i = 0; i < kCols; ++i) {
-            const float m = redux_max(s[i]);
-            if (lane == 0) xmax[w4 * N + n0 + i] = m;
+          for (int i = 0; i < 2 * kGroups; ++i) {
+            const int g = i >> 1, e = i & 1;
+            float m = fmaxf(s[4 * g + e], s[4 * g + 2 + e]);
+#pragma unroll
+            for (int o = 4; o < 32; o <<= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+            if (lane < 4) xmax[w4 * N + nq + 8 * g + e] = m;
           }
         }
         ld_softmax_bar();
@@ -301,7 +341,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
         tc_fence_after_sync();
         if (ok && j > 0) {
 #pragma unroll
-          for (int i = 0; i < kCols; ++i) l[i] *= corr[n0 + i];
+          for (int i = 0; i < 2 * kGroups; ++i) l[i] *= corr[nq + 8 * (i >> 1) + (i & 1)];
 #pragma unroll 1
           for (int pr = 0; pr < kPairs; ++pr) {
 #pragma unroll
@@ -319,22 +359,36 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
         }
       }
       if (!ok) continue;
+      uint32_t pk[2 * kGroups];  // [group][key block]
 #pragma unroll
-      for (int i = 0; i < kCols; ++i) {
-        const int n = n0 + i;
-        float pr = ex2(s[i] - mref[n]);
-        if (masked) pr = live && key <= limit[n] ? pr : 0.f;
-        l[i] += pr;
-        const uint16_t h = p.bf16 ? __bfloat16_as_ushort(__float2bfloat16(pr)) : __half_as_ushort(__float2half(pr));
-        if (live) *reinterpret_cast<uint16_t*>(p_col + (j & 1) * kRowAtom + n * 128 + ((p_chunk ^ (n & 7)) << 4)) = h;
+      for (int g = 0; g < kGroups; ++g) {
+        const float2 m = *reinterpret_cast<const float2*>(mref + nq + 8 * g);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float x = ex2(s[4 * g + e] - ((e & 1) ? m.y : m.x));
+          s[4 * g + e] = masked && !(s[4 * g + e] > -INFINITY) ? 0.f : x;  // a masked score is -inf, also without a reference
+        }
+        l[2 * g] += s[4 * g] + s[4 * g + 2];
+        l[2 * g + 1] += s[4 * g + 1] + s[4 * g + 3];
+#pragma unroll
+        for (int kb = 0; kb < 2; ++kb)
+          pk[2 * g + kb] = p.bf16 ? pack_bf16x2(s[4 * g + 2 * kb], s[4 * g + 2 * kb + 1]) : pack_f16x2(s[4 * g + 2 * kb], s[4 * g + 2 * kb + 1]);
       }
-      if (live && key >= n_keys) {  // slots beyond the sequence may hold anything: their weight is zero, make the value zero too
-        for (int pr = 0; pr < kPairs; ++pr) {
-          uint4* dst = reinterpret_cast<uint4*>(ring + ((j * kPairs + pr) % kSlots) * kLdSlot + half * kLdAtom + t * 128);
+      const uint32_t dst = p_addr + (j & 1) * kRowAtom;
+      if constexpr (kGroups == 1) {
+        stmatrix_x2_trans(dst, pk[0], pk[1]);
+      } else {
 #pragma unroll
-          for (int i = 0; i < 8; ++i) dst[i] = make_uint4(0, 0, 0, 0);
+        for (int g = 0; g < kGroups; g += 2) stmatrix_x4_trans(dst + g * 8 * 128, pk[2 * g], pk[2 * g + 1], pk[2 * g + 2], pk[2 * g + 3]);
+      }
+      if (lane < 16 && key0 + w4 * 16 + lane >= n_keys) {  // slots beyond the sequence may hold anything: zero weight, zero value
+        for (int pr = 0; pr < kPairs; ++pr) {
+          uint4* row = reinterpret_cast<uint4*>(ring + ((j * kPairs + pr) % kSlots) * kLdSlot + half * kLdAtom + (w4 * 16 + lane) * 128);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) row[i] = make_uint4(0, 0, 0, 0);
         }
       }
+      __syncwarp();
       tc_fence_before_sync();     // this thread's TMEM accesses are done
       fence_view_async_shared();  // its shared-memory writes are visible to the tensor core
       __syncwarp();
@@ -342,9 +396,11 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
     }
     // ---- row sums over the keys, then the normalised partial output and its log-sum-exp
 #pragma unroll
-    for (int i = 0; i < kCols; ++i) {
-      const float sum = warp_sum(l[i]);
-      if (lane == 0) xsum[w4 * N + n0 + i] = sum;
+    for (int i = 0; i < 2 * kGroups; ++i) {
+      float sum = l[i];
+#pragma unroll
+      for (int o = 4; o < 32; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+      if (lane < 4) xsum[w4 * N + nq + 8 * (i >> 1) + (i & 1)] = sum;
     }
     ld_softmax_bar();
     const int r = threadIdx.x - 128;

@@ -11,6 +11,7 @@ Replaces in the reference: cuBLAS ``F.linear``, ``flashinfer.norm.rmsnorm``,
 from __future__ import annotations
 
 import ctypes
+import functools
 import os
 
 import torch
@@ -558,22 +559,22 @@ def head_linear(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return y
 
 
+@functools.lru_cache(maxsize=None)
 def choose_latent_splits(batch: int, rows: int, max_kv_len: int, sm_count: int = 148) -> tuple[int, int]:
-    """(splits, query rows per CTA) of the absorbed latent attention, for `rows` query rows of each of `batch` sequences. One
-    wave of CTAs (each keeps most of an SM's shared memory); the estimate is microseconds per 128-key tile by rows per CTA, as
-    measured, plus what merging one more split costs."""
-    n_tiles = max(1, (max_kv_len + 127) // 128)
-    best = None
-    for per_cta, tile_us in ((16, 2.1), (32, 2.5), (64, 3.5)):
+    """(splits, query rows per CTA) of the absorbed latent attention, for `rows` query rows of each of `batch` sequences: the
+    least estimated time, from what a 64-key tile takes by rows per CTA (measured; a CTA has an SM to itself) and what writing
+    and merging the partial results of one more split costs."""
+    n_tiles = max(1, (max_kv_len + 63) // 64)
+    best = (float("inf"), 1, 16)
+    for per_cta, tile_us in ((16, 1.2), (32, 1.25), (64, 1.4)):
         if per_cta > 16 and rows <= per_cta // 2:
             continue
         ctas = batch * ((rows + per_cta - 1) // per_cta)
-        tiles = -(-n_tiles // max(1, min(sm_count // ctas, n_tiles, 64)))
-        splits = -(-n_tiles // tiles)
-        waves = -(-ctas * splits // sm_count)
-        cost = waves * tiles * tile_us + 0.1 * splits
-        if best is None or cost < best[0]:
-            best = (cost, splits, per_cta)
+        for splits in range(1, min(64, n_tiles) + 1):
+            tiles = -(-n_tiles // splits)
+            cost = -(-ctas * splits // sm_count) * tiles * tile_us + 7e-4 * batch * rows * splits
+            if cost < best[0]:
+                best = (cost, -(-n_tiles // tiles), per_cta)
     return best[1], best[2]
 
 
@@ -584,8 +585,8 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, kv_lens: torch.Tensor
     [blocks, page, P]; kv_lens int32 [B] (the new tokens included); block_table int32 [B, *]; query token i of a sequence attends
     keys j <= kv_len - tokens + i. ``sink`` fp32 [H]. Returns [B * tokens, H, P].
 
-    ``variant``: "tc" (tcgen05 tiles, 16-bit, ranks up to 512), "mma" (warp-level products, same limits) or "plain" (one warp per
-    row, any type and rank); None picks the first that handles the operands."""
+    ``variant``: "tc" (tcgen05 tiles; 16-bit, ranks up to 512) or "plain" (one warp per row, any type and rank); None picks the
+    first that handles the operands."""
     _lib.require_cuda()
     T, H, P = q.shape
     B = kv_lens.numel()
@@ -604,13 +605,9 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, kv_lens: torch.Tensor
         return out
     o_part = torch.empty((T * H, num_splits, P), dtype=torch.float32, device=q.device)
     lse_part = torch.empty((T * H, num_splits), dtype=torch.float32, device=q.device)
-    if variant == "tc":
-        per_cta = rows_per_cta or (16 if tokens * H <= 16 else 32 if tokens * H <= 32 else 64)
-        _lib.call("b200_latent_decode", ptr(q), ptr(cache), ctypes.c_longlong(cache.shape[0] * page), *shape, num_splits, per_cta,
-                  ptr(o_part), ptr(lse_part), dtype_code(q.dtype), ptr(_pipeline_status(q.device)), stream_ptr())
-    else:
-        _lib.call("b200_latent_attention", ptr(q), ptr(cache), *shape, num_splits, ptr(o_part), ptr(lse_part), dtype_code(q.dtype),
-                  stream_ptr())
+    per_cta = rows_per_cta or (16 if tokens * H <= 16 else 32 if tokens * H <= 32 else 64)
+    _lib.call("b200_latent_decode", ptr(q), ptr(cache), ctypes.c_longlong(cache.shape[0] * page), *shape, num_splits, per_cta,
+              ptr(o_part), ptr(lse_part), dtype_code(q.dtype), ptr(_pipeline_status(q.device)), stream_ptr())
     _lib.call("b200_latent_combine", ptr(o_part), ptr(lse_part), ptr(sink), T * H, H, num_splits, P, ptr(out), dtype_code(q.dtype),
               stream_ptr())
     _count(2)
