@@ -23,7 +23,8 @@ from .. import ops, utils
 from ..utils import perf_func_cold
 
 OPS = ["decode_step", "prefill_attn", "gemm_skinny_fused", "ag_gemm", "gemm_rs", "grouped_gemm", "grouped_gemm_fp8", "ag_group_gemm", "moe_reduce_rs", "allreduce_rmsnorm", "ep_dispatch_combine",
-       "decode_attn", "sp_decode", "moe_sort", "sampling", "rmsnorm", "qk_norm_rope"]
+       "decode_attn", "sp_decode", "moe_sort", "sampling", "rmsnorm", "qk_norm_rope",
+       "latent_decode", "residual_norm"]
 
 
 def main() -> None:
@@ -164,6 +165,23 @@ def main() -> None:
         g = torch.ones(8192, device=dev, dtype=dt)
         fn = lambda: ops.rmsnorm(x, g, 1e-6)
         info = {"bytes": 2.0 * x.numel() * 2}
+    elif args.op == "latent_decode":  # batch 8, 32 heads, latent rank 512
+        B, H, r = 8, 32, 512
+        cache = torch.randn(B * args.kv_len // 64, 64, r, device=dev, dtype=dt)
+        table = torch.arange(cache.shape[0], dtype=torch.int32, device=dev).view(B, -1)
+        lens, q = torch.full((B,), args.kv_len, dtype=torch.int32, device=dev), torch.randn(B, H, r, device=dev, dtype=dt)
+        splits, rows = ops.choose_latent_splits(B, H, args.kv_len)
+        sink = torch.zeros(H, device=dev)
+        fn = lambda: ops.latent_attention(q, cache, lens, table, 1, 0.05, sink, args.splits or splits, rows)
+        info = {"bytes": 2.0 * cache.numel(), "splits": args.splits or splits}
+    elif args.op == "residual_norm":  # 4096 tokens, 16 earlier states
+        T, W, n = 4096, 4096, 16
+        x, states = torch.randn(T, W, device=dev), torch.randn(n + 1, T, W, device=dev)
+        a, b = torch.randn(2, T, W, device=dev, dtype=dt)
+        gates, w = torch.randn(T, 2 * W, device=dev, dtype=dt), torch.ones(n + 1, device=dev)
+        g = torch.ones(W, device=dev, dtype=dt)
+        fn = lambda: ops.residual_norm(x, W, 0.5, a, gates[:, :W], g, b, gates[:, W:], g, states=states, weights=w, keep=True, gain=g, bias=g)
+        info = {"bytes": T * W * (8 + 8 + 4 + 4.0 * n + 4 + 2)}
     else:  # qk_norm_rope
         T, Hq, Hkv, D = 16384, 64, 8, 128
         qkv = torch.randn(T, (Hq + 2 * Hkv) * D, device=dev, dtype=dt)
