@@ -20,7 +20,7 @@ import torch
 _PKG = Path(__file__).resolve().parent
 _DEBUG = os.environ.get("B200DIST_DEBUG_LIB", "0") == "1"   # the checking build (python -m ...build --debug)
 LIB_PATH = _PKG / "lib" / ("libb200dist_debug.so" if _DEBUG else "libb200dist.so")
-_serving = False   # see use_serving_library
+_subset: str | None = None   # see use_subset
 
 _lock = threading.Lock()
 _lib: ctypes.CDLL | None = None
@@ -34,11 +34,11 @@ class NativeError(RuntimeError):
         self.code = code
 
 
-def use_serving_library() -> None:
+def use_subset(name: str | None) -> None:
     """For single-GPU programs, before the first kernel: unless the full library has been built already, build and load the
-    subset that serving one GPU needs (``build.SERVING_SOURCES``)."""
-    global _serving
-    _serving = True
+    kernels of one model family only (``build.SUBSETS``; None = the full library)."""
+    global _subset
+    _subset = name
 
 
 def lib_available() -> bool:
@@ -57,11 +57,11 @@ def load(build_if_missing: bool = True) -> ctypes.CDLL:
                 raise RuntimeError(
                     f"native library {LIB_PATH} is missing; run `python -m triton_distributed_b200.build`")
             from . import build as _build
-            path = _build.build(debug=_DEBUG, serving=_serving and not _DEBUG)
+            path = _build.build(debug=_DEBUG, subset=None if _DEBUG else _subset)
         lib = ctypes.CDLL(str(path))
         lib.b200_last_error.restype = ctypes.c_char_p
         for name in ("b200_heap_base", "b200_heap_mc_base", "b200_heap_bytes", "b200_heap_live_bytes"):
-            if hasattr(lib, name):  # not in the serving subset
+            if hasattr(lib, name):  # not in the subsets
                 getattr(lib, name).restype = ctypes.c_uint64
         _lib = lib
         return lib

@@ -7,10 +7,10 @@ Compilation is incremental (source / header mtimes) and parallel.
 Role in the reference: CMake + setup.py building ``libtriton_distributed.so`` and the Triton
 backend (``CMakeLists.txt:15-26``, ``csrc/lib/CMakeLists.txt:47``, ``python/setup.py``).
 
-Usage: ``python -m triton_distributed_b200.build [--force] [--verbose] [--debug | --serving]``
+Usage: ``python -m triton_distributed_b200.build [--force] [--verbose] [--debug | --subset NAME]``
 
-``--serving`` builds only what single-GPU serving needs into ``lib/libb200dist_serving.so``; programs that ask for it
-(``_lib.use_serving_library``) get it when the full library has not been built.
+``--subset NAME`` builds only the kernels that one model family needs on one GPU into ``lib/libb200dist_NAME.so``; programs that
+ask for it (``_lib.use_subset``) get it when the full library has not been built.
 
 ``--debug`` builds a second library, ``lib/libb200dist_debug.so``, with ``-DB200_DEBUG_CHECKS``: bounds-checked symmetric
 address translation and pseudo-random delays in front of every notify / wait / barrier (see ``b200/primitives.cuh``).
@@ -33,12 +33,13 @@ BUILD = PKG.parent / "build" / "b200dist"
 LIB_DIR = PKG / "lib"
 LIB_PATH = LIB_DIR / "libb200dist.so"
 DEBUG_LIB_PATH = LIB_DIR / "libb200dist_debug.so"
-SERVING_LIB_PATH = LIB_DIR / "libb200dist_serving.so"
 
-# sources of the single-GPU serving subset: no heap, no collectives, no expert kernels
-SERVING_SOURCES = ("runtime/host.cc", "kernels/decode_attn.cu", "kernels/elementwise.cu", "kernels/gemm_f32.cu",
-                   "kernels/gemm_skinny_sm100.cu", "kernels/gemm_sm100.cu", "kernels/latent_attn.cu", "kernels/latent_decode_sm100.cu",
-                   "kernels/prefill_attn_sm100.cu", "kernels/residual.cu", "kernels/sampling.cu")
+# what a model family launches on one GPU: no heap, no collectives
+_GEMMS = ("runtime/host.cc", "kernels/gemm_sm100.cu", "kernels/gemm_skinny_sm100.cu", "kernels/prefill_attn_sm100.cu")
+SUBSETS = {
+    "likosun": _GEMMS + ("kernels/gemm_f32.cu", "kernels/latent_attn.cu", "kernels/latent_decode_sm100.cu", "kernels/residual.cu"),
+    "qwen3": _GEMMS + ("kernels/decode_attn.cu", "kernels/elementwise.cu"),
+}
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -59,9 +60,9 @@ def _nvcc() -> str:
     return exe
 
 
-def sources(serving: bool = False) -> list[Path]:
-    if serving:
-        return [CSRC / name for name in SERVING_SOURCES]
+def sources(subset: str | None = None) -> list[Path]:
+    if subset is not None:
+        return [CSRC / name for name in SUBSETS[subset]]
     out = sorted(list(CSRC.glob("runtime/*.cc")) + list(CSRC.glob("runtime/*.cu")) + list(CSRC.glob("kernels/*.cu")))
     return out
 
@@ -81,21 +82,21 @@ def _compile(src: Path, obj: Path, verbose: bool, ptxas_v: bool, debug: bool = F
 
 
 def build(force: bool = False, verbose: bool = False, ptxas_v: bool = False, jobs: int | None = None,
-          debug: bool = False, serving: bool = False) -> Path:
-    """Compile what is out of date and link the shared library (the checking build with ``debug``, the single-GPU subset with
-    ``serving``). Returns its path. Processes that build at the same time take turns."""
+          debug: bool = False, subset: str | None = None) -> Path:
+    """Compile what is out of date and link the shared library (the checking build with ``debug``, a family's kernels with
+    ``subset``). Returns its path. Processes that build at the same time take turns."""
     BUILD.mkdir(parents=True, exist_ok=True)
     LIB_DIR.mkdir(parents=True, exist_ok=True)
     with open(BUILD / ".lock", "w") as lock:
         fcntl.flock(lock, fcntl.LOCK_EX)
-        return _build_locked(force, verbose, ptxas_v, jobs, debug, serving)
+        return _build_locked(force, verbose, ptxas_v, jobs, debug, subset)
 
 
-def _build_locked(force: bool, verbose: bool, ptxas_v: bool, jobs: int | None, debug: bool, serving: bool) -> Path:
+def _build_locked(force: bool, verbose: bool, ptxas_v: bool, jobs: int | None, debug: bool, subset: str | None) -> Path:
     hdr_time = max(_headers_mtime(), Path(__file__).stat().st_mtime)
-    lib_path = DEBUG_LIB_PATH if debug else SERVING_LIB_PATH if serving else LIB_PATH
+    lib_path = DEBUG_LIB_PATH if debug else LIB_DIR / f"libb200dist_{subset}.so" if subset else LIB_PATH
     todo, objs = [], []
-    for src in sources(serving):
+    for src in sources(subset):
         obj = BUILD / (src.parent.name + "_" + src.stem + (".dbg.o" if debug else ".o"))
         objs.append(obj)
         if force or not obj.exists() or obj.stat().st_mtime < max(src.stat().st_mtime, hdr_time):
@@ -142,9 +143,9 @@ def main() -> None:
     ap.add_argument("--verbose", action="store_true")
     ap.add_argument("--ptxas-v", action="store_true", help="print registers / spills / shared memory per kernel")
     ap.add_argument("--debug", action="store_true", help="build lib/libb200dist_debug.so with B200_DEBUG_CHECKS")
-    ap.add_argument("--serving", action="store_true", help="build only lib/libb200dist_serving.so (single-GPU serving)")
+    ap.add_argument("--subset", choices=sorted(SUBSETS), help="build only the kernels of one model family (one GPU)")
     args = ap.parse_args()
-    print(build(force=args.force, verbose=args.verbose, ptxas_v=args.ptxas_v, debug=args.debug, serving=args.serving))
+    print(build(force=args.force, verbose=args.verbose, ptxas_v=args.ptxas_v, debug=args.debug, subset=args.subset))
 
 
 if __name__ == "__main__":

@@ -78,6 +78,7 @@ class LikosunLayer:
 class Likosun:
 
     dtypes = (torch.bfloat16, torch.float16, torch.float32)
+    library_subset = "likosun"   # the native kernels that one GPU needs (``build.SUBSETS``)
 
     def __init__(self, model_config: ModelConfig, group=None, source: WeightSource | None = None):
         self.model_config, self.group = model_config, group

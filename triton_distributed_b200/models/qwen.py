@@ -91,6 +91,7 @@ class Qwen3Layer:
 class Qwen3:
 
     dtypes = (torch.bfloat16, torch.float16)
+    library_subset = "qwen3"   # the native kernels that one GPU needs (``build.SUBSETS``); None = all
 
     def __init__(self, model_config: ModelConfig, group=None, source: WeightSource | None = None):
         self.model_config = model_config

@@ -36,6 +36,8 @@ def build_moe_block(src: WeightSource, prefix: str, arch: ArchConfig, rank: int,
 class Qwen3MoE(Qwen3):
     """``Qwen3`` restricted to architectures with experts; ``AutoLLM`` picks it for them."""
 
+    library_subset = None
+
     def __init__(self, model_config: ModelConfig, group=None, source: WeightSource | None = None):
         if not model_config.arch().num_experts:
             raise ValueError(f"{model_config.model_name} has no experts; use Qwen3")

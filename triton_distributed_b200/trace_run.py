@@ -3,9 +3,9 @@
     bin/trace_run --model DIR --dtype bfloat16|float32 --out DIR --max-tokens N < steps
 
 Each line of standard input is one step:
-``{"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}``. ``entries`` names requests and their next
-tokens, ``want`` the places among them whose logits are asked for, ``end`` the requests that are finished. A step with wanted
-logits writes ``OUT/<step>.f32`` (little-endian fp32 [wanted, vocab]); every step prints ``done <step>``. Tokens run through
+``{"step": 7, "entries": [{"id": "r1", "tokens": [40, 8, 21, 8], "want": [3]}], "end": ["r1"]}``. ``entries`` holds the requests of the
+step with the tokens that come next, ``want`` indexes into those tokens, ``end`` lists requests that give their cache back. A step
+that wants logits writes ``OUT/<step>.f32`` (little-endian fp32 [wanted, vocab]); every step prints ``done <step>``. Tokens run through
 ``Engine.extend`` from the cache that earlier steps left; nothing is sampled. One request is alive at a time.
 Exit code 3: the model class has no kernels for the asked storage type.
 """
@@ -26,14 +26,14 @@ def main(argv: list[str] | None = None) -> int:
     ap.add_argument("--model", required=True, help="directory with config.json and safetensors")
     ap.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16")
     ap.add_argument("--out", required=True, help="directory for the logits")
-    ap.add_argument("--max-tokens", type=int, required=True, help="most tokens that live requests hold at any time")
+    ap.add_argument("--max-tokens", type=int, required=True, help="size of the cache in tokens")
     args = ap.parse_args(argv)
 
     from .models import Engine, ModelConfig
-    from .models.auto import UnsupportedDtype
-    _lib.use_serving_library()
+    from .models.auto import AutoLLM, UnsupportedDtype
     cfg = ModelConfig(model_name=args.model, checkpoint_dir=args.model, max_length=max(1, args.max_tokens),
                       dtype=getattr(torch, args.dtype), rank=0, world_size=1)
+    _lib.use_subset(AutoLLM.model_class(cfg).library_subset)
     try:
         engine = Engine(cfg, temperature=0.0)
     except UnsupportedDtype as e:
