@@ -38,6 +38,8 @@ DEBUG_LIB_PATH = LIB_DIR / "libb200dist_debug.so"
 _GEMMS = ("runtime/host.cc", "kernels/gemm_sm100.cu", "kernels/gemm_skinny_sm100.cu", "kernels/prefill_attn_sm100.cu")
 SUBSETS = {
     "likosun": _GEMMS + ("kernels/gemm_f32.cu", "kernels/latent_attn.cu", "kernels/latent_decode_sm100.cu", "kernels/residual.cu"),
+    "sizilorn": _GEMMS + ("kernels/gemm_f32.cu", "kernels/latent_attn.cu", "kernels/residual.cu", "kernels/elementwise.cu",
+                          "kernels/recurrent.cu", "kernels/gqa_attn.cu", "kernels/decode_attn.cu", "kernels/token_side.cu"),
     "qwen3": _GEMMS + ("kernels/decode_attn.cu", "kernels/elementwise.cu"),
 }
 

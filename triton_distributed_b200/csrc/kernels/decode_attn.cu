@@ -555,6 +555,7 @@ __global__ void __launch_bounds__(kAttnThreads) decode_split_ring_kernel(const D
   if (FUSE && !p.direct) combine_by_last_cta<BF16>(p, b, head0, nrows);
 }
 
+// With `gate` ([B, Hq], row pitch ldg) every head's merged output is multiplied by sigmoid(gate).
 // out[bh, :] = sum_s w_s o[bh, s, :] / sum_s w_s with w_s = exp(lse_s - max lse); partials with
 // lse = -inf are skipped. Strides are in elements so the same kernel merges split partials
 // ([B*Hq, S, D]) and the all-gathered per-rank partials of sequence-parallel decode ([R, B*Hq, D(+1)]).
@@ -562,12 +563,17 @@ template <bool BF16>
 __global__ void __launch_bounds__(kD) decode_combine_kernel(const float* o_part, const float* lse_part, long long o_stride_bh,
                                                             long long o_stride_s, long long lse_stride_bh,
                                                             long long lse_stride_s, int S, void* out, float* out_f32,
-                                                            float* out_lse) {
+                                                            float* out_lse, const void* gate, int ldg, int Hq) {
   const int bh = blockIdx.x, c = threadIdx.x;
   griddep_launch_dependents();
   griddep_wait();
   float o, lse;
   merge_splits(lse_part + bh * lse_stride_bh, lse_stride_s, o_part + bh * o_stride_bh + c, o_stride_s, S, o, lse);
+  if (gate) {
+    const size_t at = static_cast<size_t>(bh / Hq) * ldg + bh % Hq;
+    const float z = BF16 ? __bfloat162float(static_cast<const __nv_bfloat16*>(gate)[at]) : __half2float(static_cast<const __half*>(gate)[at]);
+    o /= 1.f + expf(-z);
+  }
   if (out) {
     if (BF16) static_cast<__nv_bfloat16*>(out)[static_cast<size_t>(bh) * kD + c] = __float2bfloat16(o);
     else static_cast<__half*>(out)[static_cast<size_t>(bh) * kD + c] = __float2half(o);
@@ -688,16 +694,29 @@ B200_API int b200_decode_attn_fused(const void* q, const void* k_cache, const vo
                           num_splits, o_part, lse_part, tickets, out, out_lse, dtype, -1, stream);
 }
 
+static int combine_impl(const float* o_part, const float* lse_part, long long o_stride_bh, long long o_stride_s,
+                        long long lse_stride_bh, long long lse_stride_s, int BH, int S, void* out, float* out_f32, float* out_lse,
+                        const void* gate, int ldg, int Hq, int dtype, void* stream) {
+  if (BH == 0) return kOk;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  auto kernel = dtype == kBF16 ? decode_combine_kernel<true> : decode_combine_kernel<false>;
+  B200_CHECK_CUDA(launch_pdl(kernel, BH, kD, 0, s, o_part, lse_part, o_stride_bh, o_stride_s, lse_stride_bh, lse_stride_s, S, out,
+                             out_f32, out_lse, gate, ldg, Hq));
+  return kOk;
+}
+
 B200_API int b200_decode_combine(const float* o_part, const float* lse_part, long long o_stride_bh, long long o_stride_s,
                                  long long lse_stride_bh, long long lse_stride_s, int BH, int S, void* out, float* out_f32,
                                  float* out_lse, int dtype, void* stream) {
-  if (BH == 0) return kOk;
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dtype == kBF16)
-    B200_CHECK_CUDA(launch_pdl(decode_combine_kernel<true>, BH, kD, 0, s, o_part, lse_part, o_stride_bh, o_stride_s,
-                               lse_stride_bh, lse_stride_s, S, out, out_f32, out_lse));
-  else
-    B200_CHECK_CUDA(launch_pdl(decode_combine_kernel<false>, BH, kD, 0, s, o_part, lse_part, o_stride_bh, o_stride_s,
-                               lse_stride_bh, lse_stride_s, S, out, out_f32, out_lse));
-  return kOk;
+  return combine_impl(o_part, lse_part, o_stride_bh, o_stride_s, lse_stride_bh, lse_stride_s, BH, S, out, out_f32, out_lse, nullptr, 0, 1,
+                      dtype, stream);
+}
+
+// Merge of the split partials o_part [B, Hq, S, 128], lse_part [B, Hq, S] with a gate logit per (sequence, head):
+// out [B, Hq, 128] = sigmoid(gate[b * ldg + h]) * merged row.
+B200_API int b200_decode_combine_gated(const float* o_part, const float* lse_part, int B, int Hq, int S, const void* gate, int ldg,
+                                       void* out, int dtype, void* stream) {
+  B200_REQUIRE(dtype == kBF16 || dtype == kF16, "decode attention supports bf16/f16");
+  return combine_impl(o_part, lse_part, static_cast<long long>(S) * kD, kD, S, 1, B * Hq, S, out, nullptr, nullptr, gate, ldg, Hq, dtype,
+                      stream);
 }

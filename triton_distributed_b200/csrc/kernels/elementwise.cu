@@ -196,6 +196,18 @@ __global__ void __launch_bounds__(256) silu_mul_kernel(const uint4* __restrict__
   }
 }
 
+// the same for fp32 storage, any row pitch
+__global__ void __launch_bounds__(256) silu_mul_f32_kernel(const float* __restrict__ x, float* __restrict__ out, int T, int inter, int ldx) {
+  griddep_launch_dependents();
+  griddep_wait();
+  const size_t total = static_cast<size_t>(T) * inter;
+  for (size_t idx = blockIdx.x * (size_t)blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = idx / inter, i = idx - t * inter;
+    const float g = x[t * ldx + i];
+    out[idx] = g / (1.f + expf(-g)) * x[t * ldx + inter + i];
+  }
+}
+
 // SwiGLU gate fused with the block quantisation of its result: out8[t, i] = e4m3(silu(x[t, i]) * x[t, inter + i] / s) with
 // one fp32 scale s = amax / 448 per 128 channels (the activation format of the block-scaled fp8 grouped GEMM), so the
 // down-projection of an fp8 expert reads a quarter of the bytes a bf16 intermediate would cost. One half-warp owns a
@@ -422,7 +434,14 @@ B200_API int b200_qk_norm_rope(const void* qkv, const int* positions, const int6
 }
 
 B200_API int b200_silu_mul(const void* x, void* out, int T, int inter, int ldx, int dtype, void* stream) {
-  B200_REQUIRE(dtype == kBF16 || dtype == kF16, "silu_mul supports bf16/f16");
+  if (dtype == kF32) {
+    if (T == 0) return kOk;
+    const long long blocks = (static_cast<long long>(T) * inter + 255) / 256;
+    B200_CHECK_CUDA(launch_pdl(silu_mul_f32_kernel, static_cast<unsigned>(blocks < 16LL * sm_count() ? blocks : 16LL * sm_count()), 256, 0,
+                               static_cast<cudaStream_t>(stream), static_cast<const float*>(x), static_cast<float*>(out), T, inter, ldx));
+    return kOk;
+  }
+  B200_REQUIRE(dtype == kBF16 || dtype == kF16, "silu_mul supports bf16/f16/f32");
   B200_REQUIRE(inter % 8 == 0 && ldx % 8 == 0, "inter (%d) and ldx (%d) must be multiples of 8", inter, ldx);
   if (T == 0) return kOk;
   const long long total = static_cast<long long>(T) * (inter / 8);

@@ -41,6 +41,8 @@ constexpr int kSkWBytes = kSkBN * kSkBK * 2;
 constexpr int kSkMaxStages = 12;
 constexpr int kSkSmemBudget = 216 * 1024;  // ring; the kernel's static shared memory (8.7 KB) comes on top
 
+constexpr int kSkMaxGroups = 8;
+
 enum SkinnyEpilogueKind : int { kEpNone = 0, kEpQkvHeads = 1, kEpResidual = 2 };
 
 struct SkinnyEpilogue {
@@ -82,6 +84,9 @@ struct SkinnyParams {
   float* scratch;     // [tiles][dual ? 2 : 1][MB][128] fp32, zero on entry and on exit
   uint32_t* tickets;  // [tiles], zero on entry and on exit
   SkinnyEpilogue ep;
+  // several inputs side by side in X ([M, groups * group_cols]): the tiles before group_tile_end[g] read input g
+  int groups, group_cols;
+  int group_tile_end[kSkMaxGroups];
   unsigned long long* trace;  // optional [gridDim.x][8] %globaltimer checkpoints of every CTA (tuning aid), else null
 };
 
@@ -100,6 +105,13 @@ __device__ __forceinline__ bool next_segment(const SkinnyParams& p, int& u, int 
   s.kb1 = min(p.num_kb, s.kb0 + (u1 - u));
   u += s.kb1 - s.kb0;
   return true;
+}
+
+// first column of X that a tile multiplies by
+__device__ __forceinline__ int tile_x_col(const SkinnyParams& p, int tile) {
+  int g = 0;
+  for (int i = 0; i + 1 < p.groups; ++i) g += tile >= p.group_tile_end[i] ? 1 : 0;
+  return g * p.group_cols;
 }
 
 __device__ __forceinline__ float ld_elem(const void* p, size_t i, bool bf16) {
@@ -308,6 +320,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
       Segment sg;
       bool ok = true;
       while (ok && next_segment(p, u, u_end, sg)) {
+        const int x_col = tile_x_col(p, sg.tile);
         for (int kb = sg.kb0; kb < sg.kb1 && ok; ++kb) {
           uint64_t t0 = 0;
           uint32_t spins = 0;
@@ -322,7 +335,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
             }
           }
           if (!ok) break;
-          tma_load_2d(smem + stage * p.stage_bytes + kW * kSkWBytes, &tmX, full_bar + stage, kb * kSkBK, 0);
+          tma_load_2d(smem + stage * p.stage_bytes + kW * kSkWBytes, &tmX, full_bar + stage, x_col + kb * kSkBK, 0);
           ++done;
           if (++stage == static_cast<uint32_t>(p.stages)) stage = 0;
         }
@@ -533,7 +546,8 @@ B200_API long long b200_gemm_skinny_scratch_floats(int M, int N, int dual) {
 static unsigned long long* g_skinny_trace = nullptr;
 
 static int skinny_impl(const void* X, const void* W, void* C, int M, int N, int K, int ldx, int ldw, int ldc, int dual,
-                       int dtype, float* scratch, uint32_t* tickets, int splits, const SkinnyEpilogue* ep, void* stream) {
+                       int dtype, float* scratch, uint32_t* tickets, int splits, const SkinnyEpilogue* ep, void* stream,
+                       int groups = 1, const int* group_tiles = nullptr) {
   B200_REQUIRE(dtype == kBF16 || dtype == kF16, "gemm_skinny supports bf16/f16");
   B200_REQUIRE(M >= 1 && M <= 256, "gemm_skinny handles 1..256 tokens, got %d", M);
   B200_REQUIRE(K % 8 == 0, "K (%d) must be a multiple of 8", K);
@@ -552,6 +566,9 @@ static int skinny_impl(const void* X, const void* W, void* C, int M, int N, int 
   p.bf16 = dtype == kBF16;
   p.C = C; p.ldc = ldc; p.scratch = scratch; p.tickets = tickets;
   p.trace = g_skinny_trace;
+  p.groups = groups;
+  p.group_cols = K;
+  for (int i = 0; i < groups && group_tiles != nullptr; ++i) p.group_tile_end[i] = group_tiles[i] + (i > 0 ? p.group_tile_end[i - 1] : 0);
   if (ep != nullptr) {
     p.ep = *ep;
     const bool fused = ep->kind != kEpNone || ep->sumsq_in != nullptr;
@@ -582,7 +599,7 @@ static int skinny_impl(const void* X, const void* W, void* C, int M, int N, int 
   CUtensorMap tw, tx;
   int rc = make_tma_2d(&tw, W, dtype, static_cast<uint64_t>(kw) * N, K, ldw, kSkBN, kSkBK, true);
   if (rc != kOk) return rc;
-  rc = make_tma_2d(&tx, X, dtype, M, K, ldx, p.MB, kSkBK, true);
+  rc = make_tma_2d(&tx, X, dtype, M, static_cast<uint64_t>(groups) * K, ldx, p.MB, kSkBK, true);
   if (rc != kOk) return rc;
   const int smem = p.stages * p.stage_bytes + 1024;
   dim3 grid(ctas);
@@ -593,6 +610,21 @@ static int skinny_impl(const void* X, const void* W, void* C, int M, int N, int 
 B200_API int b200_gemm_skinny(const void* X, const void* W, void* C, int M, int N, int K, int ldx, int ldw, int ldc,
                               int dual, int dtype, float* scratch, uint32_t* tickets, int splits, void* stream) {
   return skinny_impl(X, W, C, M, N, K, ldx, ldw, ldc, dual, dtype, scratch, tickets, splits, nullptr, stream);
+}
+
+// Products of several inputs in one pass: X is [M, groups * K] (input g in columns [g * K, (g + 1) * K)), W [128 * sum(group_tiles),
+// K], and the tiles of 128 rows of W that belong to group g multiply input g. K must be a multiple of 8; when it is not one of
+// 64, the last k-block also reads the first columns of the next input, times zero: all inputs must be finite.
+B200_API int b200_gemm_skinny_groups(const void* X, const void* W, void* C, int M, int K, int groups, const int* group_tiles, int ldx,
+                                     int ldw, int ldc, int dtype, float* scratch, uint32_t* tickets, void* stream) {
+  B200_REQUIRE(groups >= 1 && groups <= kSkMaxGroups && group_tiles != nullptr, "gemm_skinny_groups handles 1..%d inputs, got %d",
+               kSkMaxGroups, groups);
+  int tiles = 0;
+  for (int i = 0; i < groups; ++i) {
+    B200_REQUIRE(group_tiles[i] >= 1, "an input without rows");
+    tiles += group_tiles[i];
+  }
+  return skinny_impl(X, W, C, M, tiles * kSkBN, K, ldx, ldw, ldc, 0, dtype, scratch, tickets, 0, nullptr, stream, groups, group_tiles);
 }
 
 // As b200_gemm_skinny with a fused epilogue (M <= 16). `epilogue` points to a SkinnyEpilogue (see the top of this file;

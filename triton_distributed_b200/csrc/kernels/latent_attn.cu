@@ -4,7 +4,8 @@
 // side ("absorbed"), which turns the op into multi-query attention of H heads over one shared key = value row:
 //   latent_prep       RMS norm of the down-projected row, written to the cache slot of its token; squared-relu of the
 //                     feed-forward's up-projection, which sits in the same GEMM output
-//   head_linear       y[t, h, :] = W[h] x[t, h, :]  (per-head GEMM: Wk^T on the query, Wv on the attended latent)
+//   head_linear       y[t, h, :] = W[h] x[t, h, :]  (per-head GEMM: Wk^T on the query, Wv on the attended latent); optionally
+//                     of tanh(x), the second half of a low-rank map with a tanh in the middle
 //   attention over the paged latents, which serve as keys and as values: latent_decode_sm100.cu (split-KV partial results)
 //   latent_combine    merges the splits; a per-head sink logit joins the softmax denominator here, once
 //   latent_attention_plain   one warp per row, any rank, any storage type (the 32-bit mode and shapes outside the above)
@@ -79,13 +80,20 @@ struct HeadLinearParams {
   long long ldx, xh, ldy, yh;
 };
 
+enum HeadLinearAct : int { kActNone = 0, kActTanh = 1 };   // applied to x on its way into the product
+template <bool BF16>
+__device__ __forceinline__ uint32_t tanh_pair(uint32_t v) {
+  const float2 f = BF16 ? unpack_bf16x2(v) : unpack_f16x2(v);
+  return BF16 ? pack_bf16x2(tanhf(f.x), tanhf(f.y)) : pack_f16x2(tanhf(f.x), tanhf(f.y));
+}
+
 constexpr int kHlTok = 4;  // token tiles of 8 per CTA
 
 // 16-bit: CTA = one head, 128 / KS output rows, 8 * kHlTok tokens. A warp multiplies 16 rows of W by the tokens over its K
 // slice; KS warps share the rows and add their partial sums through shared memory. Both fragments are read straight from
 // global memory: a lane takes 8 consecutive k per 32-wide step (one 16-byte load per row), which permutes k inside the
 // step the same way for both operands and leaves the sum over k unchanged.
-template <bool BF16, int KS>
+template <bool BF16, int KS, int kAct>
 __global__ void __launch_bounds__(256) head_linear_kernel(const HeadLinearParams p) {
   constexpr int kRows = 128 / KS;
   __shared__ float part[KS > 1 ? KS - 1 : 1][kRows / 16][32][kHlTok * 4];
@@ -121,6 +129,8 @@ __global__ void __launch_bounds__(256) head_linear_kernel(const HeadLinearParams
       for (int i = 0; i < 4; ++i) {
         const int k = kc + 32 * i + 8 * tq;
         xv[i] = (k < k_end && t < p.T) ? *reinterpret_cast<const uint4*>(x + t * p.ldx + k) : zero;
+        if (kAct == kActTanh)
+          xv[i] = make_uint4(tanh_pair<BF16>(xv[i].x), tanh_pair<BF16>(xv[i].y), tanh_pair<BF16>(xv[i].z), tanh_pair<BF16>(xv[i].w));
       }
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
@@ -158,13 +168,14 @@ __global__ void __launch_bounds__(256) head_linear_kernel(const HeadLinearParams
 }
 
 // fp32: one output per thread, the input row in shared memory
+template <int kAct>
 __global__ void __launch_bounds__(128) head_linear_f32_kernel(const HeadLinearParams p) {
   extern __shared__ float xs[];
   const int t = blockIdx.x, h = blockIdx.y;
   griddep_launch_dependents();
   griddep_wait();
   const float* x = static_cast<const float*>(p.x) + t * p.ldx + h * p.xh;
-  for (int k = threadIdx.x; k < p.K; k += blockDim.x) xs[k] = x[k];
+  for (int k = threadIdx.x; k < p.K; k += blockDim.x) xs[k] = kAct == kActTanh ? tanhf(x[k]) : x[k];
   __syncthreads();
   const float* w = static_cast<const float*>(p.w) + static_cast<size_t>(h) * p.N * p.K;
   for (int n = threadIdx.x; n < p.N; n += blockDim.x) {
@@ -275,31 +286,38 @@ B200_API int b200_latent_prep(const void* latent_in, const void* gain, void* cac
                       return kOk;);
 }
 
-// y[t * ldy + h * yh + n] = sum_k W[h, n, k] x[t * ldx + h * xh + k]. 16-bit: K, strides in multiples of 8 elements.
-B200_API int b200_head_linear(const void* x, const void* w, void* y, int T, int H, int N, int K, long long ldx, long long xh,
-                              long long ldy, long long yh, int dtype, void* stream) {
-  if (T <= 0) return kOk;
-  B200_REQUIRE(H >= 1 && N >= 1 && K >= 1 && H <= 65535, "bad head_linear shape");
-  HeadLinearParams p{x, w, y, T, H, N, K, ldx, xh, ldy, yh};
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
+template <int kAct>
+static int launch_head_linear(const HeadLinearParams& p, int dtype, cudaStream_t s) {
   if (dtype == kF32) {
-    B200_REQUIRE(K <= 8192, "head_linear: K (%d) is limited to 8192 in fp32", K);
-    B200_CHECK_CUDA(launch_pdl(head_linear_f32_kernel, dim3(T, H), dim3(128), static_cast<size_t>(K) * 4, s, p));
+    B200_REQUIRE(p.K <= 8192, "head_linear: K (%d) is limited to 8192 in fp32", p.K);
+    B200_CHECK_CUDA(launch_pdl(head_linear_f32_kernel<kAct>, dim3(p.T, p.H), dim3(128), static_cast<size_t>(p.K) * 4, s, p));
     return kOk;
   }
   B200_REQUIRE(dtype == kBF16 || dtype == kF16, "head_linear supports bf16 / f16 / f32");
-  B200_REQUIRE(K % 8 == 0 && ldx % 8 == 0 && xh % 8 == 0, "head_linear: K (%d) and the input strides must be multiples of 8", K);
-  const int tz = (T + 8 * kHlTok - 1) / (8 * kHlTok);
-  B200_REQUIRE(tz <= 65535, "head_linear: too many tokens (%d)", T);
-  const int ks = K > 256 ? 4 : K > 128 ? 2 : 1;
-  const dim3 grid((N + 128 / ks - 1) / (128 / ks), H, tz);
-#define B200_HL(BF)                                                                                       \
-  if (ks == 4) B200_CHECK_CUDA(launch_pdl(head_linear_kernel<BF, 4>, grid, dim3(256), 0, s, p));           \
-  else if (ks == 2) B200_CHECK_CUDA(launch_pdl(head_linear_kernel<BF, 2>, grid, dim3(256), 0, s, p));      \
-  else B200_CHECK_CUDA(launch_pdl(head_linear_kernel<BF, 1>, grid, dim3(256), 0, s, p))
+  B200_REQUIRE(p.K % 8 == 0 && p.ldx % 8 == 0 && p.xh % 8 == 0, "head_linear: K (%d) and the input strides must be multiples of 8", p.K);
+  const int tz = (p.T + 8 * kHlTok - 1) / (8 * kHlTok);
+  B200_REQUIRE(tz <= 65535, "head_linear: too many tokens (%d)", p.T);
+  const int ks = p.K > 256 ? 4 : p.K > 128 ? 2 : 1;
+  const dim3 grid((p.N + 128 / ks - 1) / (128 / ks), p.H, tz);
+#define B200_HL(BF)                                                                                             \
+  if (ks == 4) B200_CHECK_CUDA(launch_pdl(head_linear_kernel<BF, 4, kAct>, grid, dim3(256), 0, s, p));           \
+  else if (ks == 2) B200_CHECK_CUDA(launch_pdl(head_linear_kernel<BF, 2, kAct>, grid, dim3(256), 0, s, p));      \
+  else B200_CHECK_CUDA(launch_pdl(head_linear_kernel<BF, 1, kAct>, grid, dim3(256), 0, s, p))
   if (dtype == kBF16) { B200_HL(true); } else { B200_HL(false); }
 #undef B200_HL
   return kOk;
+}
+
+// y[t * ldy + h * yh + n] = sum_k W[h, n, k] act(x[t * ldx + h * xh + k]), act 0 = none, 1 = tanh. 16-bit: K, strides in
+// multiples of 8 elements.
+B200_API int b200_head_linear(const void* x, const void* w, void* y, int T, int H, int N, int K, long long ldx, long long xh,
+                              long long ldy, long long yh, int act, int dtype, void* stream) {
+  if (T <= 0) return kOk;
+  B200_REQUIRE(H >= 1 && N >= 1 && K >= 1 && H <= 65535, "bad head_linear shape");
+  B200_REQUIRE(act == kActNone || act == kActTanh, "head_linear: unknown activation %d", act);
+  const HeadLinearParams p{x, w, y, T, H, N, K, ldx, xh, ldy, yh};
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return act == kActTanh ? launch_head_linear<kActTanh>(p, dtype, s) : launch_head_linear<kActNone>(p, dtype, s);
 }
 
 static int fill_latent(LatentParams& p, const void* q, const void* cache, const int* block_table, int bt_stride, const int* kv_lens,

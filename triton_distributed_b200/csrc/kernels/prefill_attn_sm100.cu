@@ -28,7 +28,7 @@
 
 namespace b200 {
 
-constexpr int kPD = 128;                    // head dim of the row-major-V entry point; value columns per CTA
+constexpr int kPD = 128;                    // value columns per CTA
 constexpr int kPM = 128, kPN = 128;         // query rows per CTA, keys per step
 constexpr int kPAtom = 128 * 64 * 2;        // one 128-row x 64-column 16-bit swizzle atom: 16 KB
 constexpr int kPTile = 2 * kPAtom;          // a 128 x 128 tile: 32 KB
@@ -46,6 +46,8 @@ struct PrefillParams {
   int v_chunks;         // ceil(dv / 128): CTAs per (query block, head)
   int v_packed;         // V^T is [Hkv, dv, total_k], a sequence's keys at columns cu_k[b] ...; else [B * Hkv, dv, s_pad]
   const float* sink;    // nullable [Hq]
+  const void* gate;     // nullable [total_q, Hq] (row pitch ldg): every head's output is multiplied by sigmoid(gate)
+  int ldg;
   const int* cu_q;      // [B + 1] first packed query row of every sequence
   const int* cu_k;      // [B + 1] first key row of every sequence (only [0, B) is read when k_lens is given)
   const int* k_lens;    // nullable [B]: keys of every sequence; null = cu_k[b + 1] - cu_k[b] (packed sequences)
@@ -64,10 +66,10 @@ __device__ __forceinline__ float fast_exp2(float x) {
 // barrier of the 256 softmax threads (warps 4-11) only
 __device__ __forceinline__ void softmax_bar() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
-// V [total_k, Hkv, 128] -> Vt [B * Hkv, 128, s_pad] (keys contiguous, zero beyond each sequence's length)
+// V [total_k, Hkv, dv] -> Vt [B * Hkv, dv, s_pad] (keys contiguous, zero beyond each sequence's length)
 __global__ void __launch_bounds__(256) transpose_v_kernel(const uint16_t* __restrict__ v, uint16_t* __restrict__ vt,
                                                           const int* __restrict__ cu_k, const int* __restrict__ k_lens,
-                                                          int Hkv, int s_pad) {
+                                                          int Hkv, int dv, int s_pad) {
   __shared__ uint16_t tile[32][33];
   const int bh = blockIdx.z, b = bh / Hkv, kvh = bh - b * Hkv;
   const int k_start = cu_k[b], k_len = k_lens ? k_lens[b] : cu_k[b + 1] - k_start;
@@ -75,12 +77,12 @@ __global__ void __launch_bounds__(256) transpose_v_kernel(const uint16_t* __rest
   const int tx = threadIdx.x & 31, ty = threadIdx.x >> 5;  // 32 x 8
   for (int i = ty; i < 32; i += 8) {
     const int s = s0 + i;
-    tile[i][tx] = s < k_len ? v[(static_cast<size_t>(k_start + s) * Hkv + kvh) * kPD + d0 + tx] : uint16_t(0);
+    tile[i][tx] = s < k_len && d0 + tx < dv ? v[(static_cast<size_t>(k_start + s) * Hkv + kvh) * dv + d0 + tx] : uint16_t(0);
   }
   __syncthreads();
   for (int i = ty; i < 32; i += 8) {
     const int s = s0 + tx;
-    if (s < s_pad) vt[(static_cast<size_t>(bh) * kPD + d0 + i) * s_pad + s] = tile[tx][i];
+    if (s < s_pad && d0 + i < dv) vt[(static_cast<size_t>(bh) * dv + d0 + i) * s_pad + s] = tile[tx][i];
   }
 }
 
@@ -333,7 +335,12 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     l_run += xsum[(half ^ 1) * kPM + row];
     if (p.sink != nullptr) l_run += exp2f(p.sink[h] * 1.4426950408889634f - m_run);  // the sink counts once, unscaled
     if (ok && q_pos < q_len) {
-      const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      if (p.gate != nullptr) {
+        const size_t at = static_cast<size_t>(q_start + q_pos) * p.ldg + h;
+        const float z = p.bf16 ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.gate)[at]) : __half2float(static_cast<const __half*>(p.gate)[at]);
+        inv /= 1.f + expf(-z);
+      }
       uint8_t* dst = static_cast<uint8_t*>(p.out) + ((static_cast<size_t>(q_start + q_pos) * p.Hq + h) * p.dv + v_col0 + col0) * 2;
 #pragma unroll
       for (int c = 0; c < 8; ++c) {
@@ -373,7 +380,7 @@ static int launch_prefill_atoms(const CUtensorMap& tq, const CUtensorMap& tk, co
 
 static int prefill_launch(const void* q, int64_t ldq, const void* k, const void* vt, int s_pad, int v_packed, const int* cu_q,
                           const int* cu_k, const int* k_lens, int B, int total_q, int total_k, int max_q, int Hq, int Hkv, int dk, int dv, float scale,
-                          int causal, const float* sink, void* out, int dtype, uint32_t* status, cudaStream_t s) {
+                          int causal, const float* sink, const void* gate, int ldg, void* out, int dtype, uint32_t* status, cudaStream_t s) {
   CUtensorMap tq, tk, tv;
   int rc = make_tma_3d(&tq, q, dtype, dk, Hq, total_q, dk, static_cast<uint64_t>(ldq), 64, 1, kPM, true);
   if (rc != kOk) return rc;
@@ -385,7 +392,7 @@ static int prefill_launch(const void* q, int64_t ldq, const void* k, const void*
   PrefillParams p;
   memset(&p, 0, sizeof(p));
   p.Hq = Hq; p.Hkv = Hkv; p.causal = causal; p.bf16 = dtype == kBF16;
-  p.dk = dk; p.dv = dv; p.v_chunks = (dv + kPD - 1) / kPD; p.v_packed = v_packed; p.sink = sink;
+  p.dk = dk; p.dv = dv; p.v_chunks = (dv + kPD - 1) / kPD; p.v_packed = v_packed; p.sink = sink; p.gate = gate; p.ldg = ldg;
   p.cu_q = cu_q; p.cu_k = cu_k; p.k_lens = k_lens;
   p.scale_log2e = scale * 1.4426950408889634f;
   p.out = out; p.status = status;
@@ -403,39 +410,42 @@ static int prefill_launch(const void* q, int64_t ldq, const void* k, const void*
 
 using namespace b200;
 
-// Bytes of the transposed-V scratch that b200_prefill_attention needs: B * Hkv * 128 * s_pad elements of 2 bytes, where
+// Bytes of the transposed-V scratch that b200_prefill_attention needs: B * Hkv * dv * s_pad elements of 2 bytes, where
 // s_pad = max_k rounded up to 128.
-B200_API long long b200_prefill_attention_scratch_bytes(int B, int Hkv, int max_k) {
+B200_API long long b200_prefill_attention_scratch_bytes(int B, int Hkv, int dv, int max_k) {
   const long long s_pad = (static_cast<long long>(max_k) + 127) / 128 * 128;
-  return static_cast<long long>(B) * Hkv * kPD * s_pad * 2;
+  return static_cast<long long>(B) * Hkv * dv * s_pad * 2;
 }
 
-// q [total_q, Hq, 128], k / v [total_k, Hkv, 128] (contiguous rows), cu_q / cu_k int32 [B + 1] on the device, out
-// [total_q, Hq, 128]. Sequence b's keys are rows [cu_k[b], cu_k[b] + len) with len = k_lens[b], or cu_k[b + 1] - cu_k[b]
+// q [total_q, Hq, dk], k [total_k, Hkv, dk], v [total_k, Hkv, dv] (contiguous rows), cu_q / cu_k int32 [B + 1] on the device, out
+// [total_q, Hq, dv]. Sequence b's keys are rows [cu_k[b], cu_k[b] + len) with len = k_lens[b], or cu_k[b + 1] - cu_k[b]
 // when k_lens is null (packed sequences); with k_lens the key rows may sit anywhere in k / v, e.g. in the pages of a
 // KV cache whose sequences own contiguous runs of slots. With causal != 0 query i of a sequence attends keys
-// <= i + (k_len - q_len). vt_scratch: b200_prefill_attention_scratch_bytes(...) bytes, 16-byte aligned.
+// <= i + (k_len - q_len). gate: nullable [total_q, Hq] with row pitch ldg, every head's output times sigmoid(gate).
+// vt_scratch: b200_prefill_attention_scratch_bytes(...) bytes, 16-byte aligned. dk, dv: multiples of 8, dk <= 256.
 // dtype 0 = bf16, 1 = f16.
 B200_API int b200_prefill_attention(const void* q, const void* k, const void* v, const int* cu_q, const int* cu_k,
                                     const int* k_lens, int B,
-                                    int total_q, int total_k, int max_q, int max_k, int Hq, int Hkv, int head_dim,
-                                    float scale, int causal, void* vt_scratch, void* out, int dtype, uint32_t* status,
-                                    void* stream) {
+                                    int total_q, int total_k, int max_q, int max_k, int Hq, int Hkv, int dk, int dv,
+                                    float scale, int causal, const void* gate, int ldg, void* vt_scratch, void* out, int dtype,
+                                    uint32_t* status, void* stream) {
   B200_REQUIRE(dtype == kBF16 || dtype == kF16, "prefill attention supports bf16/f16");
-  B200_REQUIRE(head_dim == kPD, "prefill attention is specialised for head_dim 128, got %d", head_dim);
+  B200_REQUIRE(dk >= 8 && dk % 8 == 0 && dk <= 256 && dv >= 8 && dv % 8 == 0,
+               "prefill attention needs head sizes in multiples of 8, keys up to 256; got %d and %d", dk, dv);
   B200_REQUIRE(Hkv > 0 && Hq % Hkv == 0, "Hq (%d) must be a multiple of Hkv (%d)", Hq, Hkv);
   B200_REQUIRE(B >= 1 && max_q >= 1 && max_k >= 1 && total_q >= 1 && total_k >= 1, "empty problem");
   B200_REQUIRE(vt_scratch != nullptr, "the transposed-V scratch is required");
+  B200_REQUIRE(scale > 0.f, "the score scale must be positive");
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int s_pad = (max_k + 127) / 128 * 128;
-  transpose_v_kernel<<<dim3(s_pad / 32, kPD / 32, B * Hkv), 256, 0, s>>>(static_cast<const uint16_t*>(v),
-                                                                          static_cast<uint16_t*>(vt_scratch), cu_k, k_lens, Hkv, s_pad);
+  transpose_v_kernel<<<dim3(s_pad / 32, (dv + 31) / 32, B * Hkv), 256, 0, s>>>(
+      static_cast<const uint16_t*>(v), static_cast<uint16_t*>(vt_scratch), cu_k, k_lens, Hkv, dv, s_pad);
   B200_CHECK_CUDA(cudaGetLastError());
-  return prefill_launch(q, static_cast<int64_t>(Hq) * kPD, k, vt_scratch, s_pad, 0, cu_q, cu_k, k_lens, B, total_q, total_k, max_q, Hq,
-                        Hkv, kPD, kPD, scale, causal, nullptr, out, dtype, status, s);
+  return prefill_launch(q, static_cast<int64_t>(Hq) * dk, k, vt_scratch, s_pad, 0, cu_q, cu_k, k_lens, B, total_q, total_k, max_q, Hq,
+                        Hkv, dk, dv, scale, causal, nullptr, gate, ldg, out, dtype, status, s);
 }
 
-// As b200_prefill_attention for head sizes other than 128 and values that are already transposed:
+// As b200_prefill_attention for values that are already transposed:
 //   q [total_q, Hq, dk] with ldq elements between two tokens; k [total_k, Hkv, dk] contiguous; vt [Hkv, dv, total_k], the keys of
 //   a sequence at columns cu_k[b] ... (multiples of 8). Whole tiles of 128 keys are read: what follows a sequence must be finite;
 //   sink: nullable fp32 [Hq] on the device, a logit that joins every row's softmax denominator unscaled and has no value;
@@ -451,5 +461,5 @@ B200_API int b200_prefill_attention_vt(const void* q, long long ldq, const void*
                "prefill attention needs dk (%d) <= 256, and dk, dv (%d), ldq, total_k (%d) in multiples of 8", dk, dv, total_k);
   B200_REQUIRE(scale > 0.f, "the score scale must be positive");
   return prefill_launch(q, ldq, k, vt, total_k, 1, cu_q, cu_k, k_lens, B, total_q, total_k, max_q, Hq, Hkv, dk, dv, scale, causal, sink,
-                        out, dtype, status, static_cast<cudaStream_t>(stream));
+                        nullptr, 0, out, dtype, status, static_cast<cudaStream_t>(stream));
 }

@@ -6,8 +6,10 @@
 //   residual_norm    s = x + mult * (sigmoid(ga + ba) * a + sigmoid(gb + bb) * b)     (gates and b optional)
 //                    state_n = s;  x = w_0 state_0 + ... + w_{n-1} state_{n-1} + w_n s (with weights; else x = s)
 //                    h = norm(x)
-// norm is layer norm (center = 1: mean removed, variance = mean of squared deviations) or RMS norm (center = 0), with a
-// gain and an optional bias. The stream, the states and all arithmetic are fp32; a, b, the gates and h have the model's
+//   residual_post    x = x + mult * (rms(a) * gain_a + rms(b) * gain_b);  h = norm(x)  (b optional): sublayers whose results are
+//                    RMS-normed on their way into the stream
+// norm is layer norm (mean removed, variance = mean of squared deviations), RMS norm or tanh(alpha x), with a gain and an
+// optional bias; or a plain copy of x in the storage type. The stream, the states and all arithmetic are fp32; a, b, the gates and h have the model's
 // storage type (bf16 / f16 / fp32). Rows are `pitch` wide: columns in [width, pitch) are padding, which carries zeros and
 // is left out of the statistics.
 //
@@ -24,12 +26,14 @@ namespace b200 {
 
 constexpr int kRnThreads = 512;
 
+enum NormKind : int { kNormRms = 0, kNormLayer = 1, kNormTanh = 2, kNormCopy = 3 };
+
 struct NormParams {
-  int width, pitch, center;
-  float eps;
-  const void* gain;   // [pitch]; null: no norm, h is not written
+  int width, pitch, kind;
+  float eps;          // of the statistics (rms, layer); the factor alpha of kNormTanh
+  const void* gain;   // [pitch] (not read by kNormCopy)
   const void* bias;   // [pitch] or null
-  void* h;            // [T, pitch]
+  void* h;            // [T, pitch]; null: no norm
 };
 
 struct ResidualParams {
@@ -44,6 +48,14 @@ struct ResidualParams {
   const float* weights;           // [n_prev + 1] or null
   int n_prev;
   int keep;                       // store the new state at index n_prev
+  NormParams norm;
+};
+
+struct PostParams {
+  const void *a, *b;              // sublayer results [T, pitch]; b nullable
+  const void *gain_a, *gain_b;    // [pitch] gains of their RMS norms
+  float eps, mult;
+  float* x;                       // [T, pitch] in / out
   NormParams norm;
 };
 
@@ -83,11 +95,11 @@ struct RowStats {
   float mean, m2;  // mean, sum of squared deviations from it
 };
 
-// statistics of the CTA's slice; RMS norm (center = 0) takes the deviations from zero
+// statistics of the CTA's slice; RMS norm takes the deviations from zero
 template <int U, int kCl>
 __device__ __forceinline__ RowStats slice_stats(const NormParams& n, const Slice<kCl>& sl, const float4 (&v)[U], int count, float* red) {
   RowStats st{0.f, 0.f};
-  if (n.center) {
+  if (n.kind == kNormLayer) {
     float s = 0.f;
 #pragma unroll
     for (int u = 0; u < U; ++u) s += (v[u].x + v[u].y) + (v[u].z + v[u].w);  // padding columns are zero
@@ -108,7 +120,23 @@ __device__ __forceinline__ RowStats slice_stats(const NormParams& n, const Slice
 template <typename T, int U, int kCl>
 __device__ __forceinline__ void norm_row(const NormParams& n, const Slice<kCl>& sl, size_t row, const float4 (&v)[U],
                                          const float4 (&gain)[U], const float4 (&bias)[U], float* red, float4* shared_stats) {
-  if (n.gain == nullptr) return;  // the same for the whole cluster
+  if (n.h == nullptr) return;  // the same for the whole cluster
+  if (n.kind >= kNormTanh) {   // no statistics
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int c = sl.col(u);
+      if (c >= sl.end) continue;
+      float4 o = v[u];
+      if (n.kind == kNormTanh) {
+        o.x = tanhf(n.eps * o.x) * gain[u].x + bias[u].x;
+        o.y = tanhf(n.eps * o.y) * gain[u].y + bias[u].y;
+        o.z = tanhf(n.eps * o.z) * gain[u].z + bias[u].z;
+        o.w = tanhf(n.eps * o.w) * gain[u].w + bias[u].w;
+      }
+      store4(static_cast<T*>(n.h) + row * n.pitch + c, o);
+    }
+    return;
+  }
   const int count = max(0, min(sl.end, n.width) - sl.begin);
   RowStats st = slice_stats<U, kCl>(n, sl, v, count, red);
   if (kCl > 1) {
@@ -253,11 +281,84 @@ __global__ void __launch_bounds__(kRnThreads) residual_norm_kernel(const Residua
   norm_row<T, U, kCl>(p.norm, sl, t, x, gain, bias, red, stats);
 }
 
+// sum over the row of the squares of `v` and `w`, for the whole cluster
+template <int U, int kCl>
+__device__ __forceinline__ float2 row_squares(const float4 (&v)[U], const float4 (&w)[U], float* red, float2* shared_sums) {
+  float sv = 0.f, sw = 0.f;
+#pragma unroll
+  for (int u = 0; u < U; ++u) {  // padding columns are zero
+    sv += (v[u].x * v[u].x + v[u].y * v[u].y) + (v[u].z * v[u].z + v[u].w * v[u].w);
+    sw += (w[u].x * w[u].x + w[u].y * w[u].y) + (w[u].z * w[u].z + w[u].w * w[u].w);
+  }
+  float2 s = make_float2(block_sum(sv, red), block_sum(sw, red));
+  if (kCl > 1) {
+    const uint32_t me = cluster_ctarank();
+    if (threadIdx.x < kCl) {
+      const uint32_t dst = mapa_u32(shared_sums + me, threadIdx.x);
+      asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(dst), "f"(s.x), "f"(s.y) : "memory");
+    }
+    cluster_sync_all();
+    s = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < kCl; ++i) {
+      s.x += shared_sums[i].x;
+      s.y += shared_sums[i].y;
+    }
+  }
+  return s;
+}
+
+template <typename T, int U, int kCl>
+__global__ void __launch_bounds__(kRnThreads) residual_post_kernel(const PostParams p) {
+  __shared__ float red[32];
+  __shared__ float4 stats[kCl];
+  __shared__ float2 sums[kCl];
+  const size_t t = blockIdx.x / kCl;
+  const int pitch = p.norm.pitch;
+  const Slice<kCl> sl(pitch);
+  griddep_launch_dependents();
+  float4 gain[U], bias[U], a[U], b[U];
+  load_norm_weights<T, U, kCl>(p.norm, sl, gain, bias);
+  if (kCl > 1) cluster_sync_all();  // every CTA of the cluster runs before any writes to another's shared memory
+  griddep_wait();
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    const int c = sl.col(u);
+    a[u] = b[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c >= sl.end) continue;
+    a[u] = load4(static_cast<const T*>(p.a) + t * pitch + c);
+    if (p.b != nullptr) b[u] = load4(static_cast<const T*>(p.b) + t * pitch + c);
+  }
+  const float2 ss = row_squares<U, kCl>(a, b, red, sums);
+  const float ia = p.mult / sqrtf(ss.x / p.norm.width + p.eps), ib = p.mult / sqrtf(ss.y / p.norm.width + p.eps);
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    const int c = sl.col(u);
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < sl.end) {
+      x = load4(p.x + t * pitch + c);
+      const float4 ga = load4(static_cast<const T*>(p.gain_a) + c);
+      x.x = fmaf(a[u].x * ia, ga.x, x.x); x.y = fmaf(a[u].y * ia, ga.y, x.y);
+      x.z = fmaf(a[u].z * ia, ga.z, x.z); x.w = fmaf(a[u].w * ia, ga.w, x.w);
+      if (p.b != nullptr) {
+        const float4 gb = load4(static_cast<const T*>(p.gain_b) + c);
+        x.x = fmaf(b[u].x * ib, gb.x, x.x); x.y = fmaf(b[u].y * ib, gb.y, x.y);
+        x.z = fmaf(b[u].z * ib, gb.z, x.z); x.w = fmaf(b[u].w * ib, gb.w, x.w);
+      }
+      store4(p.x + t * pitch + c, x);
+    }
+    a[u] = x;
+  }
+  norm_row<T, U, kCl>(p.norm, sl, t, a, gain, bias, red, stats);
+}
+
 static int check_norm(const NormParams& n) {
   B200_REQUIRE(n.width > 0 && n.pitch % 4 == 0 && n.pitch >= n.width, "row pitch (%d) must be a multiple of 4 and >= width (%d)",
                n.pitch, n.width);
   B200_REQUIRE(n.pitch <= 4 * 8 * kRnThreads, "width (%d) is limited to %d", n.width, 4 * 8 * kRnThreads);
-  B200_REQUIRE(n.gain == nullptr || n.h != nullptr, "the norm needs an output");
+  B200_REQUIRE(n.kind >= kNormRms && n.kind <= kNormCopy, "unknown norm kind %d", n.kind);
+  B200_REQUIRE((n.gain == nullptr || n.h != nullptr) && (n.h == nullptr || n.kind == kNormCopy || n.gain != nullptr),
+               "the norm needs a gain and an output");
   return kOk;
 }
 // groups of four columns per thread, from the kernels' instantiations, and the threads that then cover a row
@@ -321,13 +422,13 @@ static int launch_rows(const RowKernel<P> (&k)[5], RowKernel<P> k4, RowKernel<P>
 using namespace b200;
 
 B200_API int b200_embed_norm(const long long* ids, const void* table, int rows, long long V, int width, int pitch, float scale,
-                             float* x, float* state0, const void* gain, const void* bias, float eps, int center, void* h,
+                             float* x, float* state0, const void* gain, const void* bias, float eps, int kind, void* h,
                              int dtype, void* stream) {
   if (rows <= 0) return kOk;
   EmbedParams p;
   memset(&p, 0, sizeof(p));
   p.ids = ids; p.table = table; p.V = V; p.scale = scale; p.x = x; p.state0 = state0;
-  p.norm = NormParams{width, pitch, center, eps, gain, bias, h};
+  p.norm = NormParams{width, pitch, kind, eps, gain, bias, h};
   int rc = check_norm(p.norm);
   if (rc != kOk) return rc;
   B200_DISPATCH_FLOAT(dtype, B200_ROW_KERNELS(embed_norm_kernel, EmbedParams););
@@ -338,7 +439,7 @@ B200_API int b200_embed_norm(const long long* ids, const void* table, int rows, 
 B200_API int b200_residual_norm(const void* a, const void* gate_a, const void* bias_a, const void* b, const void* gate_b,
                                 const void* bias_b, int ldg, float mult, float* x, float* states, long long state_stride,
                                 const float* weights, int n_prev, int keep, int rows, int width, int pitch, const void* gain,
-                                const void* bias, float eps, int center, void* h, int dtype, void* stream) {
+                                const void* bias, float eps, int kind, void* h, int dtype, void* stream) {
   if (rows <= 0) return kOk;
   B200_REQUIRE(a != nullptr && x != nullptr, "residual_norm needs a sublayer result and the stream");
   B200_REQUIRE(weights == nullptr || (states != nullptr && n_prev >= 1), "the depth average needs the earlier states");
@@ -347,8 +448,24 @@ B200_API int b200_residual_norm(const void* a, const void* gate_a, const void* b
   memset(&p, 0, sizeof(p));
   p.a = a; p.b = b; p.gate_a = gate_a; p.gate_b = gate_b; p.bias_a = bias_a; p.bias_b = bias_b; p.ldg = ldg; p.mult = mult;
   p.x = x; p.states = states; p.state_stride = state_stride; p.weights = weights; p.n_prev = n_prev; p.keep = keep;
-  p.norm = NormParams{width, pitch, center, eps, gain, bias, h};
+  p.norm = NormParams{width, pitch, kind, eps, gain, bias, h};
   int rc = check_norm(p.norm);
   if (rc != kOk) return rc;
   B200_DISPATCH_FLOAT(dtype, B200_ROW_KERNELS(residual_norm_kernel, ResidualParams););
+}
+
+// x += mult * (rms(a) * gain_a + rms(b) * gain_b) over rows of `width` (b, gain_b nullable), then the norm as above.
+B200_API int b200_residual_post(const void* a, const void* gain_a, const void* b, const void* gain_b, float post_eps, float mult,
+                                float* x, int rows, int width, int pitch, const void* gain, const void* bias, float eps, int kind,
+                                void* h, int dtype, void* stream) {
+  if (rows <= 0) return kOk;
+  B200_REQUIRE(a != nullptr && gain_a != nullptr && x != nullptr && (b == nullptr) == (gain_b == nullptr),
+               "residual_post needs sublayer results with their gains, and the stream");
+  PostParams p;
+  memset(&p, 0, sizeof(p));
+  p.a = a; p.b = b; p.gain_a = gain_a; p.gain_b = gain_b; p.eps = post_eps; p.mult = mult; p.x = x;
+  p.norm = NormParams{width, pitch, kind, eps, gain, bias, h};
+  int rc = check_norm(p.norm);
+  if (rc != kOk) return rc;
+  B200_DISPATCH_FLOAT(dtype, B200_ROW_KERNELS(residual_post_kernel, PostParams););
 }

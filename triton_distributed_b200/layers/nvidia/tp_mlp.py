@@ -87,6 +87,8 @@ class TP_MLP:
     def partial_fwd(self, x: torch.Tensor) -> torch.Tensor:
         """Native GEMMs, no reduction: returns this rank's partial sum of the down projection. x: [T, H]."""
         T = x.shape[0]
+        if x.dtype == torch.float32:
+            return ops.linear(ops.silu_mul(ops.linear(x, self.gate_up_proj)), self.down_proj)
         if T <= 128:
             act = ops.gemm_skinny(x, self.gate_up_proj, swiglu=True)
             return ops.gemm_skinny(act, self.down_proj)

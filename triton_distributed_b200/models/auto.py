@@ -11,9 +11,13 @@ class AutoLLM:
     @staticmethod
     def model_class(config: ModelConfig):
         arch = config.arch()
-        if getattr(arch, "architecture", None) == "Likosun":
+        design = getattr(arch, "architecture", None)
+        if design == "Likosun":
             from .likosun import Likosun
             return Likosun
+        if design == "Sizilorn":
+            from .sizilorn import Sizilorn
+            return Sizilorn
         if arch.num_experts:
             from .qwen_moe import Qwen3MoE
             return Qwen3MoE

@@ -63,12 +63,14 @@ class Engine:
         self.graph = None
         if self.no_graph:
             return
+        state = self.kv_cache.save_state()  # the warm-up steps are not part of the sequences
         s = torch.cuda.Stream()
         s.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(s):
             for _ in range(3):
                 self._decode_step()
         torch.cuda.current_stream().wait_stream(s)
+        self.kv_cache.restore_state(state)
         torch.cuda.synchronize()
         if dist.is_initialized() and self.model_config.world_size > 1:
             dist.barrier(group=self.group)

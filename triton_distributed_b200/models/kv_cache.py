@@ -1,4 +1,5 @@
-"""Paged caches: keys and values head-sharded over the tensor-parallel ranks, or one latent row per token and layer.
+"""Paged caches: keys and values head-sharded over the tensor-parallel ranks, one latent row per token and layer, or pages and
+recurrent states side by side.
 
 Same interface as the reference's dense cache (``python/triton_dist/models/kv_cache.py:29-66``:
 ``update_kv_cache``, ``rand_fill_kv_cache``, ``inc_offset``, ``clear``, ``get_kv_len``) but stored as pages
@@ -8,6 +9,8 @@ and a decode step can be captured in a CUDA graph. ``PagedCache`` owns the pages
 offsets), the subclasses own what a page holds.
 """
 from __future__ import annotations
+
+import dataclasses
 
 import torch
 
@@ -33,6 +36,14 @@ class PagedCache:
 
     def clear(self) -> None:
         self.kv_offset.zero_()
+
+    def save_state(self):
+        """What a decode step changes beyond the slots it writes (running a step again would change it again); None here: pages
+        are written at their slot, whatever was there."""
+        return None
+
+    def restore_state(self, saved) -> None:
+        """Back to ``save_state``'s result, in place."""
 
     def get_kv_len(self) -> torch.Tensor:
         return self.kv_offset
@@ -92,3 +103,45 @@ class LatentCache(PagedCache):
         """Zero the unused rows [start, stop) of every sequence."""
         if stop > start:
             self.c_cache[layer_idx].view(self.batch_size, self.blocks_per_seq * self.page_size, -1)[:, start:stop].zero_()
+
+
+class HybridCache(PagedCache):
+    """Layers of different kinds: some keep rows per token in pages, some a state of fixed size per sequence, some both.
+
+    ``layers[i]`` maps names to shapes: ``pages`` name -> the shape of a token's row, stored ``[num_blocks, page, *row]`` in the
+    cache's type; ``states`` name -> (shape, type), stored ``[batch, *shape]``. States start at zero: ``clear`` zeroes them (pages need
+    not be), in place, so that a captured decode step keeps its addresses."""
+
+    @dataclasses.dataclass
+    class Layer:
+        pages: dict[str, tuple[int, ...]] = dataclasses.field(default_factory=dict)
+        states: dict[str, tuple[tuple[int, ...], torch.dtype]] = dataclasses.field(default_factory=dict)
+
+    def __init__(self, layers: list["HybridCache.Layer"], batch_size: int, max_length: int, dtype=torch.bfloat16, page_size: int = 64,
+                 device="cuda") -> None:
+        super().__init__(len(layers), batch_size, max_length, dtype, page_size, device)
+        self._pages = [{n: torch.zeros((self.num_blocks, page_size, *row), device=device, dtype=dtype) for n, row in layer.pages.items()}
+                       for layer in layers]
+        self._states = [{n: torch.zeros((batch_size, *shape), device=device, dtype=dt) for n, (shape, dt) in layer.states.items()}
+                        for layer in layers]
+
+    def pages(self, layer_idx: int, name: str) -> torch.Tensor:
+        return self._pages[layer_idx][name]
+
+    def state(self, layer_idx: int, name: str) -> torch.Tensor:
+        return self._states[layer_idx][name]
+
+    def _all_states(self) -> list[torch.Tensor]:
+        return [t for layer in self._states for t in layer.values()]
+
+    def clear(self) -> None:
+        super().clear()
+        for t in self._all_states():
+            t.zero_()
+
+    def save_state(self):
+        return [t.clone() for t in self._all_states()]
+
+    def restore_state(self, saved) -> None:
+        for t, old in zip(self._all_states(), saved):
+            t.copy_(old)

@@ -13,7 +13,7 @@ import os
 
 import torch
 
-from .config import ArchConfig, LikosunConfig
+from .config import DESIGNS, Arch, ArchConfig, LikosunConfig, ParallelSpec, SizilornConfig
 
 
 def likosun_param_shapes(arch: LikosunConfig) -> dict[str, tuple[int, ...]]:
@@ -34,7 +34,50 @@ def likosun_param_shapes(arch: LikosunConfig) -> dict[str, tuple[int, ...]]:
     return out
 
 
-def param_shapes(arch: ArchConfig | LikosunConfig) -> dict[str, tuple[int, ...]]:
+def _wkv_shapes(m, W: int) -> dict[str, tuple[int, ...]]:
+    N = m.heads * m.dim
+    return {**{f"mu.{s}": (W,) for s in "rkvgw"}, **{s: (N, W) for s in "rkvg"}, "w1": (m.decay_rank, W), "w2": (N, m.decay_rank),
+            "w0": (N,), "u": (m.heads, m.dim), "norm": (N,), "o": (W, N)}
+
+
+def _gated_attention_shapes(m, W: int) -> dict[str, tuple[int, ...]]:
+    return {"q": (m.heads * m.dim, W), "k": (m.kv_heads * m.dim, W), "v": (m.kv_heads * m.vdim, W), "q.norm": (m.dim,), "k.norm": (m.dim,),
+            "g": (m.heads, W), "o": (W, m.heads * m.vdim)}
+
+
+def _gated_delta_shapes(m, W: int) -> dict[str, tuple[int, ...]]:
+    qk, v = m.kv_heads * m.dim, m.heads * m.vdim
+    return {"q": (qk, W), "k": (qk, W), "v": (v, W), "q.conv": (qk, m.conv), "k.conv": (qk, m.conv), "v.conv": (v, m.conv), "b": (m.heads, W),
+            "a": (m.heads, W), "A_log": (m.heads,), "dt_bias": (m.heads,), "norm": (m.vdim,), "g": (v, W), "o": (W, v)}
+
+
+def sizilorn_param_shapes(arch: SizilornConfig) -> dict[str, tuple[int, ...]]:
+    """Names and shapes of a Sizilorn checkpoint (linear weights [out, in])."""
+    W, side = arch.hidden_size, arch.side_dim
+
+    def norm(name):
+        return {name: (W,), name + ".b": (W,), name + ".alpha": ()}
+
+    out = {"embed": (arch.vocab_size, W), "side.embed": (arch.vocab_size, arch.num_hidden_layers * side)}
+    for i, layer in enumerate(arch.layers):
+        p, m = f"l{i}.", layer.mixer
+        out.update(norm(p + "norm1"))
+        if isinstance(m, ParallelSpec):
+            for name, part in (("left", _gated_attention_shapes(m.left, W)), ("right", _gated_delta_shapes(m.right, W))):
+                out.update({f"{p}mix.{name}.{k}": v for k, v in {**part, "out": (W,)}.items()})
+        else:
+            out.update({f"{p}mix.{k}": v for k, v in _wkv_shapes(m, W).items()})
+        if layer.mlp is not None:
+            out.update(norm(p + "norm2"))
+            out.update({p + "mlp.gate": (layer.mlp.ff, W), p + "mlp.up": (layer.mlp.ff, W), p + "mlp.down": (W, layer.mlp.ff)})
+        out.update({p + "side.gate": (side, W), p + "side.proj": (W, side), p + "side.norm": (W,)})
+    out.update({**norm("final.norm"), "head": (arch.vocab_size, W)})
+    return out
+
+
+def param_shapes(arch: Arch) -> dict[str, tuple[int, ...]]:
+    if isinstance(arch, SizilornConfig):
+        return sizilorn_param_shapes(arch)
     return likosun_param_shapes(arch) if isinstance(arch, LikosunConfig) else hf_param_shapes(arch)
 
 
@@ -69,10 +112,14 @@ def hf_param_shapes(arch: ArchConfig) -> dict[str, tuple[int, ...]]:
 
 
 def _constant_init(name: str, shape: tuple[int, ...], dtype: torch.dtype, device) -> torch.Tensor | None:
-    if name.endswith(("norm.weight", "layernorm.weight", ".norm", ".norm1")):
+    if name.endswith(("norm.weight", "layernorm.weight", ".norm", ".norm1", ".norm2", ".out", ".alpha")):
         return torch.ones(shape, dtype=dtype, device=device)
-    if name.endswith((".b", ".sink")):
+    if name.endswith((".b", ".sink", ".A_log", ".dt_bias")) and len(shape) == 1:
         return torch.zeros(shape, dtype=dtype, device=device)
+    if ".mu." in name:
+        return torch.full(shape, 0.5, dtype=dtype, device=device)
+    if name.endswith(".w0"):   # decays from slow to fast over the channels
+        return torch.linspace(-6.0, 0.0, shape[0], device=device).to(dtype)
     if name.endswith(".dwa"):
         t = torch.zeros(shape, dtype=dtype, device=device)
         t[-1] = 1
@@ -81,8 +128,8 @@ def _constant_init(name: str, shape: tuple[int, ...], dtype: torch.dtype, device
 
 
 def _init_tensor(name: str, shape: tuple[int, ...], dtype: torch.dtype, seed: int, device="cpu") -> torch.Tensor:
-    """N(0, 0.02) for matrices, ones for norm gains, zeros for biases and sinks, the newest state alone for depth-average
-    weights; the stream depends only on (seed, name)."""
+    """N(0, 0.02) for matrices, constants where the name says so (ones for norm gains, zeros for biases and sinks, the newest state
+    alone for depth-average weights, a range of decays); the stream depends only on (seed, name)."""
     const = _constant_init(name, shape, dtype, device)
     if const is not None:
         return const
@@ -91,9 +138,9 @@ def _init_tensor(name: str, shape: tuple[int, ...], dtype: torch.dtype, seed: in
     return (torch.randn(shape, generator=g, dtype=torch.float32, device=device) * 0.02).to(dtype)
 
 
-def _config_dict(arch: ArchConfig | LikosunConfig, dtype: torch.dtype) -> dict:
+def _config_dict(arch: Arch, dtype: torch.dtype) -> dict:
     """Contents of config.json."""
-    if isinstance(arch, LikosunConfig):
+    if not isinstance(arch, ArchConfig):
         return arch.to_dict()
     return {
         "architectures": ["Qwen3MoeForCausalLM" if arch.num_experts else "Qwen3ForCausalLM"],
@@ -107,7 +154,7 @@ def _config_dict(arch: ArchConfig | LikosunConfig, dtype: torch.dtype) -> dict:
     }
 
 
-def write_random_checkpoint(path: str, arch: ArchConfig | LikosunConfig, dtype: torch.dtype = torch.bfloat16, seed: int = 0,
+def write_random_checkpoint(path: str, arch: Arch, dtype: torch.dtype = torch.bfloat16, seed: int = 0,
                             max_shard_bytes: int = 2 << 30) -> None:
     """Write ``config.json``, ``model.safetensors.index.json`` and ``model-XXXXX-of-YYYYY.safetensors``."""
     from safetensors.torch import save_file
@@ -134,11 +181,11 @@ def write_random_checkpoint(path: str, arch: ArchConfig | LikosunConfig, dtype: 
         json.dump(_config_dict(arch, dtype), f, indent=1)
 
 
-def read_arch_from_checkpoint(path: str) -> ArchConfig | LikosunConfig:
+def read_arch_from_checkpoint(path: str) -> Arch:
     with open(os.path.join(path, "config.json")) as f:
         c = json.load(f)
-    if c.get("architecture") == LikosunConfig.architecture:
-        return LikosunConfig.from_dict(c)
+    if c.get("architecture") in DESIGNS:
+        return DESIGNS[c["architecture"]].from_dict(c)
     if "hidden_size" not in c:
         raise ValueError(f"unknown architecture in {path}/config.json: {c.get('architecture', c.get('architectures'))!r}")
     return ArchConfig(
@@ -190,13 +237,13 @@ class SafetensorsSource(WeightSource):
         return name in self.weight_map
 
     def get(self, name, rows=None, cols=None):
-        sl = self._file(self.weight_map[name]).get_slice(name)
+        file = self._file(self.weight_map[name])
         if rows is None and cols is None:
-            t = sl[:]
+            t = file.get_tensor(name)
         elif cols is None:
-            t = sl[rows]
+            t = file.get_slice(name)[rows]
         else:
-            t = sl[rows if rows is not None else slice(None), cols]
+            t = file.get_slice(name)[rows if rows is not None else slice(None), cols]
         t = t.to(self.device)
         return t.to(self.dtype) if self.dtype is not None else t
 
@@ -210,7 +257,7 @@ class RandomSource(WeightSource):
     seconds; the result is a valid random-init model, just not the same one for different world sizes.
     """
 
-    def __init__(self, arch: ArchConfig | LikosunConfig, dtype: torch.dtype, seed: int = 0, device="cuda", consistent: bool = True):
+    def __init__(self, arch: Arch, dtype: torch.dtype, seed: int = 0, device="cuda", consistent: bool = True):
         self.shapes = param_shapes(arch)
         self.dtype, self.seed, self.device, self.consistent = dtype, seed, device, consistent
 
@@ -226,6 +273,8 @@ class RandomSource(WeightSource):
             if cols is not None:
                 t = t[:, cols]
             return t.contiguous().to(self.device)
+        if not shape:
+            return _init_tensor(name, shape, self.dtype, self.seed, device=self.device)
         r = range(shape[0])[rows] if rows is not None else range(shape[0])
         if len(shape) == 1:
             return _init_tensor(name, (len(r),), self.dtype, self.seed, device=self.device)

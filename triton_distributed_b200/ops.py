@@ -11,6 +11,7 @@ Replaces in the reference: cuBLAS ``F.linear``, ``flashinfer.norm.rmsnorm``,
 from __future__ import annotations
 
 import ctypes
+import dataclasses
 import functools
 import os
 
@@ -191,6 +192,33 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None) ->
     return y.reshape(*lead, w.shape[0])
 
 
+_GROUP_TILE = 128  # rows of a decode-GEMM tile
+
+
+def linear_groups(x: torch.Tensor, w: torch.Tensor, rows: list[int]) -> torch.Tensor:
+    """Several inputs, each with its own rows of one weight matrix: x [T, G, K], w [sum(rows), K] with ``rows[g]`` rows (multiples
+    of 128) for input g; returns ``[x_0 @ w_0.T | x_1 @ w_1.T | ...]`` [T, sum(rows)]. Up to 256 tokens are one launch."""
+    _lib.require_cuda()
+    T, G, K = x.shape
+    if not x.is_contiguous() or w.shape != (sum(rows), K) or w.stride(1) != 1 or len(rows) != G or any(r % _GROUP_TILE for r in rows):
+        raise ValueError("linear_groups: shape/layout mismatch")
+    out = torch.empty((T, w.shape[0]), dtype=x.dtype, device=x.device)
+    if T <= 256 and x.dtype != torch.float32:
+        lib = _lib.load()
+        lib.b200_gemm_skinny_scratch_floats.restype = ctypes.c_longlong
+        scratch, tickets = _skinny_scratch.get(x.device, lib.b200_gemm_skinny_scratch_floats(T, w.shape[0], 0), w.shape[0] // _GROUP_TILE)
+        tiles = (ctypes.c_int * G)(*[r // _GROUP_TILE for r in rows])
+        _lib.call("b200_gemm_skinny_groups", ptr(x), ptr(w), ptr(out), T, K, G, tiles, G * K, w.stride(0), out.stride(0),
+                  dtype_code(x.dtype), ptr(scratch), ptr(tickets), stream_ptr())
+        _count()
+        return out
+    at = 0
+    for g, r in enumerate(rows):
+        (gemm_f32 if x.dtype == torch.float32 else gemm)(x[:, g], w[at:at + r], out[:, at:at + r])
+        at += r
+    return out
+
+
 def gemm_f32(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
     """``a[M,K] @ b[N,K].T`` in true fp32 (no TF32), for the models' 32-bit mode."""
     _lib.require_cuda()
@@ -355,13 +383,14 @@ _FUSED_COMBINE_DEFAULT = os.environ.get("B200DIST_ATTN_FUSED_COMBINE", "0") == "
 def decode_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, kv_lens: torch.Tensor,
                      block_table: torch.Tensor, scale: float, soft_cap: float = 0.0, num_splits: int = 1,
                      out: torch.Tensor | None = None, return_lse: bool = False, workspace: dict | None = None,
-                     fused_combine: bool | None = None, ring: int = -1):
+                     fused_combine: bool | None = None, ring: int = -1, gate: torch.Tensor | None = None):
     """Paged GQA decode attention. q [B,Hq,128]; caches [num_blocks, page, Hkv, 128]; kv_lens int32 [B];
     block_table int32 [B, max_blocks]. Returns out [B,Hq,128] (and natural-log LSE fp32 [B,Hq]).
 
     With ``num_splits > 1`` the last CTA of every (batch, head group) merges the split partials inside the same
     launch (``fused_combine=False`` runs the separate combine kernel instead). ``ring`` selects the K/V pipeline:
-    0 = two-stage CTA-wide, 3 / 6 = per-warp rings of that depth, -1 = the library default."""
+    0 = two-stage CTA-wide, 3 / 6 = per-warp rings of that depth, -1 = the library default. ``gate`` [B, Hq] (unit inner
+    stride): every head's output is multiplied by its sigmoid, in the combine launch."""
     _lib.require_cuda()
     B, Hq, D = q.shape
     page, Hkv = k_cache.shape[1], k_cache.shape[2]
@@ -369,11 +398,14 @@ def decode_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
         raise ValueError("decode_attention needs contiguous q / caches and a row-major block table")
     if out is None:
         out = torch.empty_like(q)
+    if gate is not None and (gate.shape != (B, Hq) or gate.stride(1) != 1 or gate.dtype != q.dtype or return_lse):
+        raise ValueError("decode_attention: the gate is [B, Hq] in the type of q, without a log-sum-exp")
     if fused_combine is None:
         fused_combine = _FUSED_COMBINE_DEFAULT
+    fused_combine = fused_combine and gate is None
     lse = torch.empty((B, Hq), dtype=torch.float32, device=q.device) if return_lse else None
     tickets = None
-    if num_splits > 1:
+    if num_splits > 1 or gate is not None:
         if workspace is not None and "o_part" in workspace and workspace["o_part"].numel() >= B * Hq * num_splits * D:
             o_part, lse_part = workspace["o_part"], workspace["lse_part"]
         else:
@@ -392,9 +424,13 @@ def decode_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
         o_part = lse_part = None
     _lib.call("b200_decode_attn", ptr(q), ptr(k_cache), ptr(v_cache), ptr(block_table), block_table.stride(0),
               ptr(kv_lens), B, Hq, Hkv, D, page, c_float(scale), c_float(soft_cap), num_splits, ptr(o_part),
-              ptr(lse_part), ptr(tickets), ptr(out), ptr(lse), dtype_code(q.dtype), ring, stream_ptr())
+              ptr(lse_part), ptr(tickets), ptr(None if gate is not None else out), ptr(lse), dtype_code(q.dtype), ring, stream_ptr())
     _count()
-    if num_splits > 1 and tickets is None:
+    if gate is not None:
+        _lib.call("b200_decode_combine_gated", ptr(o_part), ptr(lse_part), B, Hq, num_splits, ptr(gate), gate.stride(0), ptr(out),
+                  dtype_code(q.dtype), stream_ptr())
+        _count()
+    elif num_splits > 1 and tickets is None:
         _lib.call("b200_decode_combine", ptr(o_part), ptr(lse_part), ctypes.c_longlong(num_splits * D),
                   ctypes.c_longlong(D), ctypes.c_longlong(num_splits), ctypes.c_longlong(1), B * Hq, num_splits,
                   ptr(out), None, ptr(lse), dtype_code(q.dtype), stream_ptr())
@@ -430,18 +466,22 @@ def check_pipeline_status(device=None) -> None:
 def prefill_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_seqlens_q: torch.Tensor,
                       cu_seqlens_k: torch.Tensor, max_seqlen_q: int, max_seqlen_k: int, scale: float,
                       causal: bool = True, out: torch.Tensor | None = None,
-                      seqlens_k: torch.Tensor | None = None) -> torch.Tensor:
-    """Variable-length attention on the tcgen05 prefill kernel. q [total_q, Hq, 128]; k, v [total_k, Hkv, 128];
-    cu_seqlens_* int32 [B + 1] on the device. With ``causal`` query i of a sequence attends keys <= i + (k_len - q_len).
+                      seqlens_k: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> torch.Tensor:
+    """Variable-length attention on the tcgen05 prefill kernel. q [total_q, Hq, dk]; k [total_k, Hkv, dk], v [total_k, Hkv, dv]
+    (sizes in multiples of 8, dk <= 256); cu_seqlens_* int32 [B + 1] on the device. ``gate`` [total_q, Hq] (unit inner stride):
+    every head's output is multiplied by its sigmoid. With ``causal`` query i of a sequence attends keys <= i + (k_len - q_len).
 
     Packed sequences: leave ``seqlens_k`` None (lengths are differences of ``cu_seqlens_k``). Keys in place: give
     ``seqlens_k`` int32 [B]; sequence b then reads rows ``cu_seqlens_k[b] ... + seqlens_k[b]`` of k / v, which may be the
-    slot view of a paged KV cache whose sequences own contiguous runs of slots. Returns [total_q, Hq, 128]."""
+    slot view of a paged KV cache whose sequences own contiguous runs of slots. Returns [total_q, Hq, dv]."""
     _lib.require_cuda()
     total_q, Hq, D = q.shape
     total_k, Hkv, _ = k.shape
-    if not (q.is_contiguous() and k.is_contiguous() and v.is_contiguous()) or k.shape != v.shape or D != 128:
-        raise ValueError("prefill_attention needs contiguous q / k / v with head dim 128")
+    dv = v.shape[2]
+    if not (q.is_contiguous() and k.is_contiguous() and v.is_contiguous()) or k.shape[:2] != v.shape[:2] or k.shape[2] != D:
+        raise ValueError("prefill_attention needs contiguous q / k / v of matching shapes")
+    if gate is not None and (gate.shape != (total_q, Hq) or gate.stride(1) != 1 or gate.dtype != q.dtype):
+        raise ValueError("prefill_attention: the gate is [total_q, Hq] in the type of q")
     if q.dtype not in (torch.bfloat16, torch.float16) or k.dtype != q.dtype or v.dtype != q.dtype:
         raise TypeError("prefill_attention handles bf16 / f16")
     B = cu_seqlens_q.numel() - 1
@@ -450,12 +490,13 @@ def prefill_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_seql
     k_lens = seqlens_k.to(device=q.device, dtype=torch.int32).contiguous() if seqlens_k is not None else None
     lib = _lib.load()
     lib.b200_prefill_attention_scratch_bytes.restype = ctypes.c_longlong
-    nbytes = int(lib.b200_prefill_attention_scratch_bytes(B, Hkv, int(max_seqlen_k)))
+    nbytes = int(lib.b200_prefill_attention_scratch_bytes(B, Hkv, dv, int(max_seqlen_k)))
     scratch = torch.empty(nbytes, dtype=torch.uint8, device=q.device)
     if out is None:
-        out = torch.empty_like(q)
+        out = torch.empty((total_q, Hq, dv), dtype=q.dtype, device=q.device)
     _lib.call("b200_prefill_attention", ptr(q), ptr(k), ptr(v), ptr(cu_q), ptr(cu_k), ptr(k_lens), B, total_q, total_k,
-              int(max_seqlen_q), int(max_seqlen_k), Hq, Hkv, D, c_float(scale), 1 if causal else 0, ptr(scratch), ptr(out),
+              int(max_seqlen_q), int(max_seqlen_k), Hq, Hkv, D, dv, c_float(scale), 1 if causal else 0, ptr(gate),
+              gate.stride(0) if gate is not None else 0, ptr(scratch), ptr(out),
               dtype_code(q.dtype), ptr(_pipeline_status(q.device)), stream_ptr())
     _count(2)
     return out
@@ -474,14 +515,28 @@ def combine_partials(o_part: torch.Tensor, lse_part: torch.Tensor, out_dtype: to
 
 
 # ---- fp32 residual stream (csrc/kernels/residual.cu) ------------------------------------------
+@dataclasses.dataclass(frozen=True)
+class TanhNorm:
+    """``tanh(alpha x) * gain + bias`` in place of a norm with statistics (``center`` argument of the ops below)."""
+    alpha: float
+
+
+COPY = "copy"  # as ``center``: no norm, the stream in the storage type
+
+
 def _norm_args(width, gain, bias, eps, center, h):
-    return ptr(gain), ptr(bias), c_float(eps), 1 if center else 0, ptr(h)
+    """`center`: True = layer norm, False = RMS norm, a ``TanhNorm``, or ``COPY``."""
+    if isinstance(center, TanhNorm):
+        kind, factor = 2, center.alpha
+    else:
+        kind, factor = (3, 0.0) if center == COPY else (1 if center else 0, eps)
+    return ptr(gain), ptr(bias), c_float(factor), kind, ptr(h)
 
 
 def embed_norm(ids: torch.Tensor, table: torch.Tensor, scale: float, width: int, gain: torch.Tensor, bias: torch.Tensor | None,
-               eps: float, center: bool, state0: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
+               eps: float, center: bool | TanhNorm, state0: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
     """``x = table[ids] * scale`` in fp32 and ``h = norm(x)`` in the table's type, one kernel. ids int64 [T]; table [V, P]
-    with P >= width columns (padding columns zero). ``center``: layer norm, else RMS norm. ``state0`` fp32 [T, P]
+    with P >= width columns (padding columns zero). ``center``: layer norm, else RMS norm, or a ``TanhNorm``. ``state0`` fp32 [T, P]
     receives a copy of x. Returns (x fp32 [T, P], h [T, P])."""
     _lib.require_cuda()
     flat = ids.reshape(-1).to(torch.int64).contiguous()
@@ -498,11 +553,12 @@ def residual_norm(x: torch.Tensor, width: int, mult: float, a: torch.Tensor, gat
                   bias_a: torch.Tensor | None = None, b: torch.Tensor | None = None, gate_b: torch.Tensor | None = None,
                   bias_b: torch.Tensor | None = None, states: torch.Tensor | None = None, weights: torch.Tensor | None = None,
                   keep: bool = False, gain: torch.Tensor | None = None, bias: torch.Tensor | None = None, eps: float = 0.0,
-                  center: bool = True) -> torch.Tensor | None:
+                  center: bool | TanhNorm | str = True) -> torch.Tensor | None:
     """One pass over the fp32 residual stream ``x`` [T, P] (updated in place):
     ``s = x + mult * (sigmoid(gate_a + bias_a) * a + sigmoid(gate_b + bias_b) * b)``; with ``weights`` (fp32 [n + 1])
     ``x = sum_j weights[j] * states[j] + weights[n] * s`` over the n earlier states (``states`` fp32 [>= n, T, P]; s is stored
-    as state n with ``keep``), else ``x = s``; returns ``norm(x)`` when ``gain`` is given. a, b [T, P]; the gate logits may be
+    as state n with ``keep``), else ``x = s``; returns ``norm(x)`` when ``gain`` is given (see ``_norm_args`` for ``center``; ``COPY``
+    returns x in the type of a and takes no gain). a, b [T, P]; the gate logits may be
     column slices of a wider GEMM output (same row pitch)."""
     _lib.require_cuda()
     T, P = x.shape
@@ -517,12 +573,162 @@ def residual_norm(x: torch.Tensor, width: int, mult: float, a: torch.Tensor, gat
     if weights is not None and (weights.dtype != torch.float32 or states is None or states.shape[0] < n + (1 if keep else 0)
                                 or states.shape[1:] != x.shape or not states.is_contiguous()):
         raise ValueError("residual_norm: weights fp32 [n + 1] need contiguous fp32 states [>= n, T, P]")
-    h = torch.empty((T, P), dtype=a.dtype, device=a.device) if gain is not None else None
+    h = torch.empty((T, P), dtype=a.dtype, device=a.device) if gain is not None or center == COPY else None
     _lib.call("b200_residual_norm", ptr(a), ptr(gate_a), ptr(bias_a), ptr(b), ptr(gate_b), ptr(bias_b), ldg, c_float(mult), ptr(x),
               ptr(states), ctypes.c_longlong(T * P), ptr(weights), n, 1 if keep else 0, T, width, P,
               *_norm_args(width, gain, bias, eps, center, h), dtype_code(a.dtype), stream_ptr())
     _count()
     return h
+
+
+def residual_post(x: torch.Tensor, width: int, mult: float, a: torch.Tensor, gain_a: torch.Tensor, b: torch.Tensor | None = None,
+                  gain_b: torch.Tensor | None = None, post_eps: float = 0.0, gain: torch.Tensor | None = None,
+                  bias: torch.Tensor | None = None, eps: float = 0.0, center: bool | TanhNorm | str = True) -> torch.Tensor | None:
+    """``x += mult * (rms(a) * gain_a + rms(b) * gain_b)`` on the fp32 stream x [T, P] (in place; b optional): sublayer results [T, P]
+    that are RMS-normed over the width on their way in. Returns ``norm(x)`` as ``residual_norm`` does."""
+    _lib.require_cuda()
+    T, P = x.shape
+    if x.dtype != torch.float32 or a.shape != x.shape or not a.is_contiguous() or (b is not None and (b.shape != x.shape or not b.is_contiguous())):
+        raise ValueError("residual_post: x must be fp32 [T, P] and the sublayer results contiguous [T, P]")
+    h = torch.empty((T, P), dtype=a.dtype, device=a.device) if gain is not None or center == COPY else None
+    _lib.call("b200_residual_post", ptr(a), ptr(gain_a), ptr(b), ptr(gain_b), c_float(post_eps), c_float(mult), ptr(x), T, width, P,
+              *_norm_args(width, gain, bias, eps, center, h), dtype_code(a.dtype), stream_ptr())
+    _count()
+    return h
+
+
+def token_side(g: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, offset: int, dim: int) -> torch.Tensor:
+    """``gelu(g) * table[ids, offset : offset + dim]`` (tanh form of gelu). g [T, P] contiguous, P >= dim; ids int64 [T]; returns [T, P],
+    zeros behind `dim`."""
+    _lib.require_cuda()
+    if not g.is_contiguous() or not table.is_contiguous() or table.dtype != g.dtype or ids.dtype != torch.int64 or ids.numel() != g.shape[0]:
+        raise ValueError("token_side: shape/layout mismatch")
+    act = torch.empty_like(g)
+    _lib.call("b200_token_side", ptr(g), ptr(ids), ptr(table), ptr(act), g.shape[0], ctypes.c_longlong(table.shape[0]), dim, g.shape[1],
+              table.shape[1], offset, dtype_code(g.dtype), stream_ptr())
+    _count()
+    return act
+
+
+# ---- recurrent mixers (csrc/kernels/recurrent.cu) ---------------------------------------------
+def token_mix(h: torch.Tensor, mu: torch.Tensor, last: torch.Tensor) -> torch.Tensor:
+    """``h_t + (h_{t-1} - h_t) * mu_g`` for every row of mu [G, P]: h [B * S, P] -> [B * S, G, P]. ``last`` [B, P] is the token before
+    the call and is replaced by the call's last one."""
+    _lib.require_cuda()
+    T, P = h.shape
+    B, G = last.shape[0], mu.shape[0]
+    if not (h.is_contiguous() and mu.is_contiguous() and last.is_contiguous()) or T % B or mu.shape[1] != P or last.shape[1] != P:
+        raise ValueError("token_mix: shape/layout mismatch")
+    out = torch.empty((T, G, P), dtype=h.dtype, device=h.device)
+    _lib.call("b200_token_mix", ptr(h), ptr(mu), ptr(last), ptr(out), B, T // B, G, P, dtype_code(h.dtype), stream_ptr())
+    _count()
+    return out
+
+
+def short_conv(x: torch.Tensor, taps: torch.Tensor, last: torch.Tensor) -> torch.Tensor:
+    """Causal convolution per channel, then silu: x [B * S, C] (rows may be strided), taps fp32 [n, C] (the last weighs the current
+    token), ``last`` [B, n - 1, C] the inputs before the call, replaced by the last ones of the call. Returns [B * S, C]."""
+    _lib.require_cuda()
+    T, C = x.shape
+    n, B = taps.shape[0], last.shape[0]
+    if x.stride(1) != 1 or taps.dtype != torch.float32 or not (taps.is_contiguous() and last.is_contiguous()) or taps.shape[1] != C \
+            or last.shape[1:] != (n - 1, C) or last.dtype != x.dtype or T % B:
+        raise ValueError("short_conv: shape/layout mismatch")
+    out = torch.empty((T, C), dtype=x.dtype, device=x.device)
+    _lib.call("b200_short_conv", ptr(x), ptr(taps), ptr(last), ptr(out), B, T // B, C, n, x.stride(0), dtype_code(x.dtype), stream_ptr())
+    _count()
+    return out
+
+
+def _check_recurrent(state, rows, fp32, name):
+    if state.dtype != torch.float32 or not state.is_contiguous() or any(t.dtype != torch.float32 or not t.is_contiguous() for t in fp32):
+        raise ValueError(f"{name}: the state and the per-channel constants must be contiguous fp32")
+    if any(t.stride(1) != 1 or t.dtype != rows[0].dtype or t.shape[0] != rows[0].shape[0] for t in rows):
+        raise ValueError(f"{name}: the inputs must be rows of one type with unit inner stride")
+
+
+def wkv(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, gate: torch.Tensor, w0: torch.Tensor, u: torch.Tensor,
+        gain: torch.Tensor, state: torch.Tensor, dim: int, vdim: int, eps: float, plain: bool = False) -> torch.Tensor:
+    """Decayed outer-product memory with a bonus ``u`` for the current token and decays ``exp(-exp(z + w0))`` per key channel, then
+    the RMS norm of every head, ``gain`` and ``silu(gate)``. r, k, z [B * S, H * D], v, gate [B * S, H * E] (rows may be strided);
+    w0, u [H * D], gain [H * E]; ``state`` [B, H, D, E] is updated. D and E are multiples of 8, ``dim`` / ``vdim`` the true sizes.
+    Returns [B * S, H * E]."""
+    _lib.require_cuda()
+    B, H, D, E = state.shape
+    _check_recurrent(state, (r, k, v, z, gate), (w0, u, gain), "wkv")
+    T = r.shape[0]
+    if T % B or r.shape[1] != H * D or k.shape != r.shape or z.shape != r.shape or v.shape[1] != H * E or gate.shape != v.shape \
+            or w0.numel() != H * D or u.numel() != H * D or gain.numel() != H * E:
+        raise ValueError("wkv: shape mismatch")
+    out = torch.empty((T, H * E), dtype=r.dtype, device=r.device)
+    _lib.call("b200_wkv", ptr(r), r.stride(0), ptr(k), k.stride(0), ptr(v), v.stride(0), ptr(z), z.stride(0), ptr(gate), gate.stride(0),
+              ptr(w0), ptr(u), ptr(gain), c_float(eps), ptr(state), ptr(out), B, T // B, H, dim, D, vdim, E, int(plain),
+              dtype_code(r.dtype), stream_ptr())
+    _count()
+    return out
+
+
+def gated_delta(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tensor, b: torch.Tensor, gate: torch.Tensor,
+                a_log: torch.Tensor, dt_bias: torch.Tensor, gain: torch.Tensor, state: torch.Tensor, dim: int, vdim: int, eps: float,
+                plain: bool = False) -> torch.Tensor:
+    """Gated delta rule on unit-length q (times dim ** -0.5) and k, then the RMS norm of every head, ``gain`` and ``silu(gate)``. q, k
+    [B * S, G * D], v, gate [B * S, H * E], a (decay) and b (step size) logits [B * S, H] (rows may be strided; a and b with one
+    pitch); a_log, dt_bias [H], gain [E]; ``state`` [B, H, D, E] is updated. Returns [B * S, H * E]."""
+    _lib.require_cuda()
+    B, H, D, E = state.shape
+    _check_recurrent(state, (q, k, v, a, b, gate), (a_log, dt_bias, gain), "gated_delta")
+    T, G = q.shape[0], q.shape[1] // D
+    if T % B or q.shape[1] != G * D or k.shape != q.shape or v.shape[1] != H * E or gate.shape != v.shape or a.shape[1] != H \
+            or b.shape != a.shape or a.stride(0) != b.stride(0) or a_log.numel() != H or dt_bias.numel() != H or gain.numel() != E:
+        raise ValueError("gated_delta: shape mismatch")
+    out = torch.empty((T, H * E), dtype=q.dtype, device=q.device)
+    _lib.call("b200_gated_delta", ptr(q), q.stride(0), ptr(k), k.stride(0), ptr(v), v.stride(0), ptr(a), ptr(b), a.stride(0), ptr(gate),
+              gate.stride(0), ptr(a_log), ptr(dt_bias), ptr(gain), c_float(eps), ptr(state), ptr(out), B, T // B, H, G, dim, D, vdim, E,
+              int(plain), dtype_code(q.dtype), stream_ptr())
+    _count()
+    return out
+
+
+# ---- grouped-query attention of any head size (csrc/kernels/gqa_attn.cu) ----------------------
+def head_norm_rope(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, heads: int, kv_heads: int, dim: int, gain_q: torch.Tensor | None,
+                   gain_k: torch.Tensor | None, eps: float, cos_sin: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor,
+                   k_cache: torch.Tensor, v_cache: torch.Tensor, q_scale: float = 1.0) -> torch.Tensor:
+    """Per-head RMS norm of q and k, interleaved rotary positions on their first ``cos_sin.shape[1]`` dimensions, ``q_scale`` on q, and
+    the write of k and v to ``slots``, in one kernel. q, k, v: column slices of one GEMM output, heads of equal (padded) size;
+    caches [..., kv_heads, D'] with D' at least that size (zeros behind). cos_sin fp32 [positions, rot]: (cos, sin) of pair 0, 1, ...
+    Returns q [T, heads, D']."""
+    _lib.require_cuda()
+    T, ld = q.shape[0], q.stride(0)
+    qk_in, v_in, qk_out, v_out = q.shape[1] // heads, v.shape[1] // kv_heads, k_cache.shape[-1], v_cache.shape[-1]
+    if k.shape[1] != kv_heads * qk_in or k.stride(0) != ld or v.stride(0) != ld or positions.dtype != torch.int32 \
+            or cos_sin.dtype != torch.float32 or not cos_sin.is_contiguous() or slots.dtype != torch.int64 \
+            or not (k_cache.is_contiguous() and v_cache.is_contiguous()) or k_cache.shape[-2] != kv_heads:
+        raise ValueError("head_norm_rope: shape/layout mismatch")
+    out = torch.empty((T, heads, qk_out), dtype=q.dtype, device=q.device)
+    _lib.call("b200_head_norm_rope", ptr(q), ptr(k), ptr(v), ld, ptr(gain_q), ptr(gain_k), ptr(cos_sin), ptr(positions), ptr(slots),
+              ptr(out), ptr(k_cache), ptr(v_cache), T, heads, kv_heads, dim, cos_sin.shape[1], qk_in, qk_out, v_in, v_out, c_float(eps),
+              c_float(q_scale), dtype_code(q.dtype), stream_ptr())
+    _count()
+    return out
+
+
+def gqa_attention_plain(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, kv_lens: torch.Tensor, block_table: torch.Tensor,
+                        tokens: int, scale: float, gate: torch.Tensor | None = None) -> torch.Tensor:
+    """Causal attention of the last `tokens` tokens of every sequence over paged keys, any head sizes (multiples of 4) and storage
+    type: q [B * tokens, H, dk], caches [blocks, page, G, dk] / [..., dv], kv_lens int32 [B] with the new tokens. ``gate``
+    [B * tokens, H]: every head's output times its sigmoid. Returns [B * tokens, H, dv]."""
+    _lib.require_cuda()
+    T, H, dk = q.shape
+    B, page, G, dv = kv_lens.numel(), k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
+    if T != B * tokens or k_cache.shape[3] != dk or not (q.is_contiguous() and k_cache.is_contiguous() and v_cache.is_contiguous()) \
+            or block_table.stride(1) != 1 or (gate is not None and (gate.shape != (T, H) or gate.stride(1) != 1 or gate.dtype != q.dtype)):
+        raise ValueError("gqa_attention_plain: shape/layout mismatch")
+    out = torch.empty((T, H, dv), dtype=q.dtype, device=q.device)
+    _lib.call("b200_gqa_attention_plain", ptr(q), ptr(k_cache), ptr(v_cache), ptr(block_table), block_table.stride(0), ptr(kv_lens), B,
+              tokens, H, G, dk, dv, page, c_float(scale), ptr(gate), gate.stride(0) if gate is not None else 0, ptr(out),
+              dtype_code(q.dtype), stream_ptr())
+    _count()
+    return out
 
 
 # ---- latent attention (csrc/kernels/latent_attn.cu, prefill_attn_sm100.cu) --------------------
@@ -544,8 +750,9 @@ def latent_prep(latent_in: torch.Tensor | None, gain: torch.Tensor | None, cache
     return act
 
 
-def head_linear(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
-    """Per-head GEMM ``y[t, h, :] = w[h] @ x[t, h, :]``: x [T, H, K] (unit inner stride), w [H, N, K] -> y [T, H, N]."""
+def head_linear(x: torch.Tensor, w: torch.Tensor, tanh: bool = False) -> torch.Tensor:
+    """Per-head GEMM ``y[t, h, :] = w[h] @ x[t, h, :]``: x [T, H, K] (unit inner stride), w [H, N, K] -> y [T, H, N]. With ``tanh`` of
+    tanh(x)."""
     _lib.require_cuda()
     T, H, K = x.shape
     N = w.shape[1]
@@ -554,7 +761,7 @@ def head_linear(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     y = torch.empty((T, H, N), dtype=x.dtype, device=x.device)
     ll = ctypes.c_longlong
     _lib.call("b200_head_linear", ptr(x), ptr(w), ptr(y), T, H, N, K, ll(x.stride(0)), ll(x.stride(1)), ll(y.stride(0)),
-              ll(y.stride(1)), dtype_code(x.dtype), stream_ptr())
+              ll(y.stride(1)), int(tanh), dtype_code(x.dtype), stream_ptr())
     _count()
     return y
 

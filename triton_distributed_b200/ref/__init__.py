@@ -13,5 +13,9 @@ from .moe import (ag_group_gemm_ref, grouped_gemm_ref, grouped_gemm_fp8_ref, deq
 from .attention import paged_decode_attention_ref, combine_partials_ref, sp_flash_decode_ref
 from .likosun import (depth_average_ref, gated_residual_ref, greedy_ref, latent_attention_ref, layer_norm_ref, likosun_layer_ref,
                       likosun_ref, rms_norm_ref, sink_softmax_ref, squared_relu_ref)
+from .sizilorn import (decayed_outer_ref, gated_attention_ref, gated_delta_mixer_ref, gated_delta_ref, gelu_tanh_ref, grouped_attention_ref,
+                       parallel_mixer_ref, rotate_pairs_ref, rotation_frequencies_ref, short_conv_ref, sigmoid_ref, sizilorn_greedy_ref,
+                       sizilorn_layer_ref, sizilorn_ref, softplus_ref, swish_ref, tanh_norm_ref, token_mix_ref, token_side_ref,
+                       unit_rms_ref, unit_vector_ref, wkv_mixer_ref)
 
 __all__ = [n for n in dir() if n.endswith("_ref")]
