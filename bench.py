@@ -16,6 +16,7 @@ timed after ``--warmup`` untimed ones. Rank 0 prints ONE JSON line.
 
 ``--workload likosun`` measures the Likosun decoder instead (one GPU): prefill and decode throughput next to a Qwen3-shaped
 model of equal size, and its kernels next to the like kernels (``triton_distributed_b200/benchmark/bench_likosun.py``).
+``--workload sizilorn`` does the same for the Sizilorn decoder (``triton_distributed_b200/benchmark/bench_sizilorn.py``).
 
 Launch: ``python bench.py`` (1 GPU) or
 ``python -m torch.distributed.run --nnodes=1 --nproc-per-node N --master-addr 127.0.0.1 --master-port P bench.py --gpus N``.
@@ -197,6 +198,18 @@ def _likosun_workload(args) -> None:
     print(json.dumps(out), flush=True)
 
 
+def _sizilorn_workload(args) -> None:
+    if args.gpus != 1 or int(os.environ.get("WORLD_SIZE", "1")) != 1:
+        raise SystemExit("--workload sizilorn runs on one GPU")
+    from triton_distributed_b200.benchmark import bench_sizilorn
+    sampler = ClockSampler(0)
+    sampler.start()
+    sampler.wait_first_sample(3.0)
+    out = bench_sizilorn.run(args.sizilorn_models, args.batch, args.prompt, args.steps, args.warmup, not args.no_kernels)
+    out["clocks"] = sampler.stop()
+    print(json.dumps(out), flush=True)
+
+
 def main() -> None:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
     ap.add_argument("--gpus", type=int, default=1)
@@ -215,9 +228,10 @@ def main() -> None:
     ap.add_argument("--ar-max-bytes", type=int, default=64 << 20)
     ap.add_argument("--settle-steps", type=int, default=24,
                     help="untimed decode steps right after graph capture (clocks, link state), before any timed phase")
-    ap.add_argument("--workload", choices=["qwen3", "likosun"], default="qwen3", help="likosun: the Likosun decoder next to a "
-                    "Qwen3-shaped model of equal size (one GPU)")
+    ap.add_argument("--workload", choices=["qwen3", "likosun", "sizilorn"], default="qwen3",
+                    help="likosun, sizilorn: that decoder next to a Qwen3-shaped model of equal size (one GPU)")
     ap.add_argument("--likosun-models", nargs="*", default=["likosun-1b", "likosun-7b", "likosun-20b"])
+    ap.add_argument("--sizilorn-models", nargs="*", default=["sizilorn-1b", "sizilorn-7b"])
     args = ap.parse_args()
     if args.impl == "reference":
         if int(os.environ.get("RANK", "0")) == 0:  # one line per job, also when launched as N ranks
@@ -228,6 +242,9 @@ def main() -> None:
 
     if args.workload == "likosun":
         _likosun_workload(args)
+        return
+    if args.workload == "sizilorn":
+        _sizilorn_workload(args)
         return
 
     import torch

@@ -24,7 +24,7 @@ from ..utils import perf_func_cold
 
 OPS = ["decode_step", "prefill_attn", "gemm_skinny_fused", "ag_gemm", "gemm_rs", "grouped_gemm", "grouped_gemm_fp8", "ag_group_gemm", "moe_reduce_rs", "allreduce_rmsnorm", "ep_dispatch_combine",
        "decode_attn", "sp_decode", "moe_sort", "sampling", "rmsnorm", "qk_norm_rope",
-       "latent_decode", "residual_norm"]
+       "latent_decode", "residual_norm", "wkv", "gated_delta"]
 
 
 def main() -> None:
@@ -182,6 +182,18 @@ def main() -> None:
         g = torch.ones(W, device=dev, dtype=dt)
         fn = lambda: ops.residual_norm(x, W, 0.5, a, gates[:, :W], g, b, gates[:, W:], g, states=states, weights=w, keep=True, gain=g, bias=g)
         info = {"bytes": T * W * (8 + 8 + 4 + 4.0 * n + 4 + 2)}
+    elif args.op in ("wkv", "gated_delta"):  # batch 8 x 512 tokens; 64 heads of 64, or 32 heads of 128
+        B, S = 8, 512
+        H, D = (64, 64) if args.op == "wkv" else (32, 128)
+        rows = [torch.randn(B * S, H * D, device=dev, dtype=dt) for _ in range(5)]
+        st, c = torch.zeros(B, H, D, D, device=dev), torch.ones(H * D, device=dev)
+        if args.op == "wkv":
+            fn = lambda: ops.wkv(*rows, c, c, c, st, D, D, 1e-6)
+        else:
+            ab = torch.randn(B * S, 2 * H, device=dev, dtype=dt)
+            fn = lambda: ops.gated_delta(rows[0][:, : H // 2 * D], rows[1][:, : H // 2 * D], rows[2], ab[:, :H], ab[:, H:], rows[3], c[:H], c[:H], c[:D],
+                                         st, D, D, 1e-6)
+        info = {"flops": (5.0 if args.op == "wkv" else 7.0) * B * S * H * D * D}
     else:  # qk_norm_rope
         T, Hq, Hkv, D = 16384, 64, 8, 128
         qkv = torch.randn(T, (Hq + 2 * Hkv) * D, device=dev, dtype=dt)

@@ -83,7 +83,10 @@ def _tensors(model):
     """Weight matrices a forward pass reads (not the embedding, of which a step reads a few rows, nor second layouts)."""
     yield getattr(model, "head", None) if hasattr(model, "head") else model.lm_head
     for layer in model.layers:
-        if hasattr(layer, "w_in"):
+        if hasattr(layer, "side_proj"):     # Sizilorn
+            yield from (layer.w_in, layer.left.wo, layer.right.wo) if layer.parallel else (layer.mixer.w_in, layer.mixer.w2, layer.mixer.wo)
+            yield from (layer.mlp.gate_up_proj, layer.mlp.down_proj, layer.side_gate, layer.side_proj)
+        elif hasattr(layer, "w_in"):
             yield from (layer.w_in, layer.attn.uk, layer.attn.uv, layer.attn.wo, layer.down)
         else:
             yield from (layer.attn.wqkv, layer.attn.wo, layer.mlp.gate_up_proj, layer.mlp.down_proj)
@@ -94,7 +97,7 @@ def _row(name: str, fn, nbytes: float, flops: float = 0.0, iters: int = 12) -> d
     _, _, times = utils.perf_func_cold(fn, iters, 3)
     us = min(times) * 1e3
     roof = max(nbytes / hbm, flops / tc) * 1e6
-    return {"kernel": name, "us": round(us, 2), "roofline_us": round(roof, 2), "of_roofline": round(roof / us, 3)}
+    return {"kernel": name, "us": round(us, 2), "roofline_us": float(f"{roof:.3g}"), "of_roofline": float(f"{roof / us:.3g}")}
 
 
 def kernels(name: str, batch: int = 8, prompt: int = 2048) -> list[dict]:

@@ -10,13 +10,16 @@ columns). Kernels by storage type and head size:
 from __future__ import annotations
 
 import math
+from typing import TYPE_CHECKING
 
 import torch
 
 from ... import ops
-from ...models.config import GatedAttentionSpec, RotarySpec
-from ...models.kv_cache import HybridCache
 from .latent_attn import pad_heads, pad_matrix, pad_up
+
+if TYPE_CHECKING:
+    from ...models.config import GatedAttentionSpec, RotarySpec
+    from ...models.kv_cache import HybridCache
 
 DECODE_HEAD = 128  # head size of the decode kernel
 

@@ -6,12 +6,16 @@ multiples of eight channels with zero weights.
 """
 from __future__ import annotations
 
+from typing import TYPE_CHECKING
+
 import torch
 
 from ... import ops
-from ...models.config import GatedDeltaSpec, WkvSpec
-from ...models.kv_cache import HybridCache
 from .latent_attn import pad_heads, pad_matrix, pad_up, pad_vector
+
+if TYPE_CHECKING:
+    from ...models.config import GatedDeltaSpec, WkvSpec
+    from ...models.kv_cache import HybridCache
 
 
 def _head_vector(v: torch.Tensor, heads: int, size: int) -> torch.Tensor:
