@@ -118,12 +118,13 @@ def test_linear_groups(dtype, T, K, rows):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("T,N,K", [(1, 40, 8), (33, 264, 64), (300, 128, 136), (5, 72, 264)])
-def test_head_linear_of_tanh(dtype, T, N, K):
+def test_tanh_linear(dtype, T, N, K):
     from triton_distributed_b200 import ops
     wide = torch.randn(T, K + 16, device="cuda").to(dtype)
-    w = torch.randn(1, N, K, device="cuda").to(dtype)
-    got = ops.head_linear(wide[:, None, 8:8 + K], w, tanh=True)[:, 0]
-    _close(got, torch.tanh(_d(wide[:, 8:8 + K])) @ _d(w[0]).t(), dtype, factor=1.5)
+    w = torch.randn(N, K, device="cuda").to(dtype)
+    want = torch.tanh(_d(wide[:, 8:8 + K])) @ _d(w).t()
+    _close(ops.tanh_linear(wide[:, 8:8 + K], w), want, dtype, factor=1.5)
+    _close(ops.head_linear(wide[:, None, 8:8 + K], w[None], tanh=True)[:, 0], want, dtype, factor=1.5)
 
 
 # ------------------------------------------------------------------------------------------------ carried inputs
@@ -254,7 +255,8 @@ def _delta_case(B, S, H, D, E, dtype):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("case", [_wkv_case, _delta_case], ids=["wkv", "delta"])
-@pytest.mark.parametrize("B,S,H,D,E", [(1, 35, 2, 8, 8), (2, 24, 4, 64, 64), (1, 33, 2, 20, 13), (1, 23, 2, 65, 128), (2, 25, 2, 128, 72), (1, 24, 1, 136, 24)])
+@pytest.mark.parametrize("B,S,H,D,E", [(1, 35, 2, 8, 8), (2, 24, 4, 64, 64), (1, 33, 2, 20, 13), (1, 23, 2, 65, 128), (2, 25, 2, 128, 72), (1, 24, 1, 136, 24),
+                                       (37, 21, 4, 24, 16), (37, 21, 4, 72, 100)])
 def test_recurrences(case, dtype, B, S, H, D, E):
     run, oracle = case(B, S, H, D, E, dtype)
     want, state = oracle()
@@ -264,7 +266,8 @@ def test_recurrences(case, dtype, B, S, H, D, E):
         _close(st, state, torch.float32, factor=3.0)
         for cut in _cuts(S)[1:]:
             o2, st2 = run(plain, cut)
-            assert torch.equal(o2, got) and torch.equal(st2, st), cut    # the same sums in the same order
+            _close(o2, got, dtype, factor=0.2 if plain else 1.0)
+            _close(st2, st, torch.float32, factor=0.1 if plain else 1.0)
 
 
 @pytest.mark.parametrize("plain", [False, True])

@@ -140,11 +140,10 @@ def kernels(name: str, batch: int = 8, prompt: int = 2048) -> list[dict]:
                    2.0 * T * w.numel())
         big = _row(f"linear of equal size, {tag}", lambda: ops.linear(xl, w), 2.0 * (w.numel() + xl.numel() + T * w.shape[0]), 2.0 * T * w.numel())
         pair(new, big)
-        low, w2 = rnd(T, m.decay_rank), rnd(1, N, m.decay_rank)
-        wl = rnd(N, m.decay_rank)
-        pair(_row(f"head_linear of tanh, rank {m.decay_rank}, {tag}", lambda: ops.head_linear(low[:, None], w2, tanh=True),
+        low, w2 = rnd(T, m.decay_rank), rnd(N, m.decay_rank)
+        pair(_row(f"tanh_linear, rank {m.decay_rank}, {tag}", lambda: ops.tanh_linear(low, w2),
                   2.0 * (low.numel() + w2.numel() + T * N), 2.0 * T * w2.numel()),
-             _row(f"linear of equal size, {tag}", lambda: ops.linear(low, wl), 2.0 * (low.numel() + w2.numel() + T * N), 2.0 * T * w2.numel()))
+             _row(f"linear of equal size, {tag}", lambda: ops.linear(low, w2), 2.0 * (low.numel() + w2.numel() + T * N), 2.0 * T * w2.numel()))
         del x
     ops.check_pipeline_status()
     torch.cuda.empty_cache()

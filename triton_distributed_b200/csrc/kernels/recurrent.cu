@@ -4,14 +4,14 @@
 //                                   with w_t = exp(-exp(z_t + w0)) per key channel and a bonus u for the current token
 //   gated delta rule (kDelta)       a = S^T k_t;  d = beta_t (v_t - g_t a);           S <- g_t S + k_t d^T;  o_t = S^T q_t
 //                                   with g_t = exp(-exp(A) softplus(a_t + dt)) and beta_t = sigmoid(b_t) per head, q and k
-//                                   scaled to unit length (q also by key_size^-0.5). S^T q is read from the old state together
-//                                   with S^T k: o_t = g_t S_old^T q_t + (k_t . q_t) d, so a token costs one pass over S.
+//                                   scaled to unit length (q also by key_size^-0.5)
 // Both end in the same way: o divided by its root mean square over the head, times a gain, times silu(gate).
 //
 // The columns of S never mix, and all of S stays in registers for the whole call. One CTA owns one head of one sequence; a
-// thread owns R rows x C columns, the threads that share columns are neighbouring lanes and reduce with shuffles. Tokens go
-// through shared memory in chunks of 16; the next chunk's copies are in flight while a chunk is computed. The order of
-// all sums is that of the tokens, whatever the call's length: results do not depend on how a sequence is cut.
+// thread owns R rows x 4 columns, the eight threads that share columns are neighbouring lanes and reduce with shuffles. Tokens go
+// through shared memory in chunks of 16; the next chunk's copies are in flight while a chunk is computed. All arithmetic is
+// fp32 on the CUDA cores (two products per instruction), so the fp32 pipe is what bounds a long call. To save its instructions
+// four tokens share a pass over S: what they owe each other is a 4 x 4 triangle of scalars (see the kernel).
 // Heads of up to 128 x 128 run this way (`recurrent_kernel`); larger ones keep S in global memory (`recurrent_plain_kernel`).
 //
 // In front of them: token_mix (h + (previous h - h) * mu for several mu at once) and short_conv (causal convolution over a few
@@ -26,7 +26,11 @@
 
 namespace b200 {
 
-__device__ __forceinline__ float silu(float z) { return z / (1.f + expf(-z)); }
+// exponential and quotient: the library's functions in the 32-bit mode, the short fp32 forms with 16-bit storage
+template <typename T>
+__device__ __forceinline__ float exp_t(float z) { return sizeof(T) == 4 ? expf(z) : __expf(z); }
+template <typename T>
+__device__ __forceinline__ float silu(float z) { return sizeof(T) == 4 ? z / (1.f + expf(-z)) : __fdividef(z, 1.f + __expf(-z)); }
 
 // ------------------------------------------------------------------------------------------------ token_mix
 constexpr int kMixMax = 8;       // mixes per call
@@ -67,6 +71,20 @@ __global__ void __launch_bounds__(128) token_mix_kernel(const TokenMixParams p) 
     }
     before = cur;
   }
+}
+
+// ------------------------------------------------------------------------------------------------ tanh of a column slice
+template <typename T>
+__global__ void __launch_bounds__(256) tanh_rows_kernel(const T* x, T* out, int rows, int cols, int ldx) {
+  const int groups = cols / 4;
+  const size_t at = blockIdx.x * static_cast<size_t>(blockDim.x) + threadIdx.x;
+  griddep_launch_dependents();
+  griddep_wait();
+  if (at >= static_cast<size_t>(rows) * groups) return;
+  const size_t t = at / groups;
+  const int c = static_cast<int>(at - t * groups) * 4;
+  const float4 v = load4(x + t * ldx + c);
+  store4(out + t * cols + c, make_float4(tanhf(v.x), tanhf(v.y), tanhf(v.z), tanhf(v.w)));
 }
 
 // ------------------------------------------------------------------------------------------------ short_conv
@@ -118,7 +136,7 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvParams p
     } else {
       for (int j = 0; j < n; ++j) tap(load4(p.taps + static_cast<size_t>(j) * p.C + c), input(t - n + 1 + j));
     }
-    store4(out + static_cast<size_t>(t) * p.C, make_float4(silu(acc.x), silu(acc.y), silu(acc.z), silu(acc.w)));
+    store4(out + static_cast<size_t>(t) * p.C, make_float4(silu<T>(acc.x), silu<T>(acc.y), silu<T>(acc.z), silu<T>(acc.w)));
   }
   if (t0 == 0)  // the last n - 1 inputs up to the end of the call; slot j only needs slots behind it, so ascending is safe
     for (int j = 0; j < n - 1; ++j) store4(last + static_cast<size_t>(j) * p.C, input(p.S - (n - 1) + j));
@@ -146,7 +164,8 @@ struct RecurrentParams {
 };
 
 __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
-__device__ __forceinline__ float wkv_decay(float z, float base) { return expf(-expf(z + base)); }
+template <typename T>
+__device__ __forceinline__ float wkv_decay(float z, float base) { return exp_t<T>(-exp_t<T>(z + base)); }
 __device__ __forceinline__ float delta_decay(float a, float A, float dt) { return expf(-expf(A) * softplus(a + dt)); }
 
 // eight elements global -> shared memory without registers; zeros where !in
@@ -168,27 +187,76 @@ __device__ __forceinline__ void store8(float* dst, const float (&f)[8]) {
 }
 
 constexpr int kRecTokens = 16;   // tokens per chunk
-constexpr int recurrent_smem(int dp, int elem) { return (6 * kRecTokens * dp + 4 * kRecTokens + 2 * dp) * 4 + 5 * kRecTokens * dp * elem; }
+constexpr int kRecGroup = 4;     // tokens per pass over the memory
+constexpr int kRecGroups = kRecTokens / kRecGroup;
+constexpr int recurrent_smem(int p, int elem) {
+  return (5 * kRecTokens * p + kRecGroups * p + 2 * p + kRecTokens * 8 + kRecGroups * 32 + 4 * kRecTokens) * 4 + 5 * kRecTokens * p * elem;
+}
 
-// kP: padded key and value size; a thread owns R rows (groups of four: rows 4 (lane % 8) + 32 i ...) and C = 4 columns.
-template <typename T, int kKind, int kP, int R>
-__global__ void __launch_bounds__(kP * kP / (R * 4), kP == 128 ? 2 : 4) recurrent_kernel(const RecurrentParams p) {
-  constexpr int C = 4, KG = kP / R, kThreads = kP * kP / (R * C), kWarps = kThreads / 32;
-  constexpr int kItems = kRecTokens * kP / 8;   // groups of eight elements of a chunk
-  static_assert(KG == 8 && kItems <= kThreads, "thread layout");
+// sums over the warp of N = 16 or 32 values; lane l is left with the sum of v[l % N]
+template <int N>
+__device__ __forceinline__ float warp_sums(float (&v)[N]) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int m = N / 2; m > 0; m >>= 1) {
+    const bool hi = (lane & m) != 0;
+#pragma unroll
+    for (int i = 0; i < m; ++i) v[i] = (hi ? v[i + m] : v[i]) + __shfl_xor_sync(0xffffffffu, hi ? v[i] : v[i + m], m);
+  }
+  return N == 32 ? v[0] : v[0] + __shfl_xor_sync(0xffffffffu, v[0], 16);
+}
+
+// V consecutive elements of shared memory as floats
+template <typename T, int V>
+__device__ __forceinline__ void load_few(const T* src, float (&f)[V]) {
+  if (V == 4) {
+    const float4 x = load4(src);
+    f[0] = x.x; f[1] = x.y; f[V - 2] = x.z; f[V - 1] = x.w;
+  } else if (sizeof(T) == 4) {
+    const float2 x = *reinterpret_cast<const float2*>(src);
+    f[0] = x.x; f[1] = x.y;
+  } else {
+    const uint32_t x = *reinterpret_cast<const uint32_t*>(src);
+    f[0] = to_float(reinterpret_cast<const T*>(&x)[0]); f[1] = to_float(reinterpret_cast<const T*>(&x)[1]);
+  }
+}
+template <int V>
+__device__ __forceinline__ void store_few(float* dst, const float (&f)[V]) {
+  if (V == 4) *reinterpret_cast<float4*>(dst) = make_float4(f[0], f[1], f[V - 2], f[V - 1]);
+  else *reinterpret_cast<float2*>(dst) = make_float2(f[0], f[1]);
+}
+
+// kP: padded key and value size; a thread owns R = kP / 8 rows (groups of four, eight lanes apart) and four columns.
+// Four tokens are taken in one pass over S. With S the memory in front of them, tokens 0..3:
+//   kWkv    o_i = S^T (r_i * prod_{l<i} w_l) + sum_{j<i} (sum_d r_i k_j prod_{j<l<i} w_l) v_j + (r_i . (u * k_i)) v_i
+//           S  <- diag(prod w) S + sum_j (k_j * prod_{l>j} w_l) v_j^T
+//   kDelta  with G_ij = prod_{j<l<=i} g_l, c_i = prod_{l<=i} g_l:
+//           d_i = beta_i (v_i - c_i S^T k_i - sum_{j<i} G_ij (k_j . k_i) d_j),   o_i = c_i S^T q_i + sum_{j<=i} G_ij (k_j . q_i) d_j
+//           S  <- c_3 S + sum_j G_3j k_j d_j^T
+// The scaled vectors and the sums over key channels are prepared per chunk, one warp per four tokens. Tokens behind the end of the
+// call count as w = g = 1, k = 0.
+template <typename T, int kKind, int kP>
+__global__ void __launch_bounds__(2 * kP, kP == 128 ? 2 : 4) recurrent_kernel(const RecurrentParams p) {
+  constexpr int R = kP / 8, C = 4, kThreads = 2 * kP, kWarps = kThreads / 32, V = kP / 32;
+  constexpr int kRaw = kRecTokens * kP;
+  static_assert(kWarps == 4 || kWarps == 8, "one warp per group of tokens");
   extern __shared__ __align__(16) float smf[];
-  float* sq = smf;                          // [tokens][kP]
-  float* sk = sq + kRecTokens * kP;
-  float* sw = sk + kRecTokens * kP;         // kWkv: decays per key channel
-  float* sv = sw + kRecTokens * kP;
-  float* sg = sv + kRecTokens * kP;         // silu(gate)
-  float* so = sg + kRecTokens * kP;
-  float* s_decay = so + kRecTokens * kP;    // kDelta: [tokens]
-  float* s_beta = s_decay + kRecTokens;
-  float* s_qk = s_beta + kRecTokens;        // kWkv: r . (u * k); kDelta: q . k
-  float* s_base = s_qk + 2 * kRecTokens;    // kWkv: w0 and u of the head
+  float* sq = smf;                            // [tokens][kP] read-out vectors
+  float* sk = sq + kRaw;                      // [tokens][kP]
+  float* sv = sk + kRaw;
+  float* sg = sv + kRaw;                      // silu(gate)
+  float* so = sg + kRaw;
+  float* sw = so + kRaw;                      // kWkv: [groups][kP] product of the decays
+  float* s_base = sw + kRecGroups * kP;       // kWkv: w0 and u of the head
   float* s_bonus = s_base + kP;
-  T* raw = reinterpret_cast<T*>(s_bonus + kP);   // [q, k, decay, v, gate][tokens][kP] of the next chunk as it lies in memory
+  float* s_n = s_bonus + kP;                  // [tokens][4] coefficients of o_i on v_j (kWkv) / d_j (kDelta)
+  float* s_m = s_n + kRecTokens * 4;          // kDelta: [tokens][4] coefficients of d_i on d_j
+  float* s_dot = s_m + kRecTokens * 4;        // [groups][32]
+  float* s_c = s_dot + kRecGroups * 32;       // kDelta: c_i, G_3i, beta_i, g_i per token
+  float* s_tail = s_c + kRecTokens;
+  float* s_beta = s_tail + kRecTokens;
+  float* s_g = s_beta + kRecTokens;
+  T* raw = reinterpret_cast<T*>(s_g + kRecTokens);   // [q, k, decay, v, gate][tokens][kP] of the next chunk as it lies in memory
   const int h = blockIdx.x, b = blockIdx.y, kh = h / p.per;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kg = lane & 7;
   const int col0 = (warp * 4 + (lane >> 3)) * C;
@@ -196,10 +264,7 @@ __global__ void __launch_bounds__(kP * kP / (R * 4), kP == 128 ? 2 : 4) recurren
   griddep_launch_dependents();
   // the state comes from an earlier call: it may be fetched into L2, but not read, before that call is known to be over
   for (int i = threadIdx.x * 32; i < p.Dp * p.Ep; i += kThreads * 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(state + i));
-  const int ic = threadIdx.x % (kP / 8) * 8, it = threadIdx.x / (kP / 8);   // this thread's elements of a chunk
-  const bool has_item = threadIdx.x < kItems;
-  T* mine_raw = raw + it * kP + ic;   // a thread converts the elements that it copied itself
-  constexpr int kRaw = kRecTokens * kP;
+  const int ic = threadIdx.x % (kP / 8) * 8, it = threadIdx.x / (kP / 8);   // this thread's eight elements of a chunk
   if (kKind == kWkv && threadIdx.x < kP) {
     const bool in = threadIdx.x < p.Dp;
     s_base[threadIdx.x] = in ? p.decay_base[h * p.Dp + threadIdx.x] : 0.f;
@@ -208,27 +273,26 @@ __global__ void __launch_bounds__(kP * kP / (R * 4), kP == 128 ? 2 : 4) recurren
   const float A = kKind == kDelta ? p.decay_base[h] : 0.f, dt = kKind == kDelta ? p.decay_bias[h] : 0.f;
   griddep_wait();
 
-  float ra = 0.f, rb = 0.f;
+  float ra = 0.f, rb = 0.f;   // kDelta: logits of token 4 * warp + lane of the next chunk
   const size_t row0 = static_cast<size_t>(b) * p.S;
   auto fetch = [&](int t0) {
-    if (has_item) {
-      const size_t row = row0 + t0 + it;
-      const bool in = t0 + it < p.S, ink = in && ic < p.Dp, inv = in && ic < p.Ep;
-      copy8<T>(mine_raw, p.q, row * p.ldq + kh * p.Dp + ic, ink);
-      copy8<T>(mine_raw + kRaw, p.k, row * p.ldk + kh * p.Dp + ic, ink);
-      if (kKind == kWkv) copy8<T>(mine_raw + 2 * kRaw, p.decay, row * p.ld_decay + h * p.Dp + ic, ink);
-      copy8<T>(mine_raw + 3 * kRaw, p.v, row * p.ldv + h * p.Ep + ic, inv);
-      copy8<T>(mine_raw + 4 * kRaw, p.gate, row * p.ldg + h * p.Ep + ic, inv);
-    }
+    const size_t row = row0 + t0 + it;
+    T* dst = raw + it * kP + ic;
+    const bool in = t0 + it < p.S, ink = in && ic < p.Dp, inv = in && ic < p.Ep;
+    copy8<T>(dst, p.q, row * p.ldq + kh * p.Dp + ic, ink);
+    copy8<T>(dst + kRaw, p.k, row * p.ldk + kh * p.Dp + ic, ink);
+    if (kKind == kWkv) copy8<T>(dst + 2 * kRaw, p.decay, row * p.ld_decay + h * p.Dp + ic, ink);
+    copy8<T>(dst + 3 * kRaw, p.v, row * p.ldv + h * p.Ep + ic, inv);
+    copy8<T>(dst + 4 * kRaw, p.gate, row * p.ldg + h * p.Ep + ic, inv);
     cp_async_commit();
-    if (kKind == kDelta && threadIdx.x < kRecTokens && t0 + static_cast<int>(threadIdx.x) < p.S) {
-      const size_t at = (row0 + t0 + threadIdx.x) * p.ld_decay + h;
+    const int tok = t0 + warp * kRecGroup + lane;
+    if (kKind == kDelta && warp < kRecGroups && lane < kRecGroup && tok < p.S) {
+      const size_t at = (row0 + tok) * p.ld_decay + h;
       ra = to_float(static_cast<const T*>(p.decay)[at]);
       rb = to_float(static_cast<const T*>(p.beta)[at]);
     }
   };
   fetch(0);
-  __syncthreads();   // s_base, s_bonus
 
   f32x2 s[R / 2][C];   // s[2 i + e][c] = rows 32 i + 4 kg + 2 e, + 1 of column col0 + c
 #pragma unroll
@@ -246,141 +310,259 @@ __global__ void __launch_bounds__(kP * kP / (R * 4), kP == 128 ? 2 : 4) recurren
     }
 
   for (int t0 = 0; t0 < p.S; t0 += kRecTokens) {
-    const int n = min(kRecTokens, p.S - t0);
-    // ---- registers -> shared memory. The products r . (u * k) and q . k and the lengths need sums over the kP / 8 threads of
-    // a token, which are neighbouring lanes.
+    const int n = min(kRecTokens, p.S - t0), n_groups = (n + kRecGroup - 1) / kRecGroup;
     cp_async_wait<0>();
-    if (has_item) {   // whole warps: kItems is a multiple of 32
-      float q8[8], k8[8], f[8];
-      load8(mine_raw, q8);
-      load8(mine_raw + kRaw, k8);
-      float x = 0.f, y = 0.f, z = 0.f;
-      if (kKind == kWkv) {
+    __syncthreads();   // the raw chunk of all threads; the last chunk's results have been read
+    // ---- prepare: warp w the vectors of group w (a lane owns V channels), values and gates by the other warps if there are any
+    if (warp < n_groups) {
+      float q[kRecGroup][V], k[kRecGroup][V];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) z = fmaf(q8[i] * s_bonus[ic + i], k8[i], z);
+      for (int i = 0; i < kRecGroup; ++i) {
+        load_few<T, V>(raw + (warp * kRecGroup + i) * kP + lane * V, q[i]);
+        load_few<T, V>(raw + kRaw + (warp * kRecGroup + i) * kP + lane * V, k[i]);
+      }
+      if (kKind == kWkv) {
+        float w[kRecGroup][V], x[16], total[V];
+#pragma unroll
+        for (int i = 0; i < kRecGroup; ++i) {
+          load_few<T, V>(raw + 2 * kRaw + (warp * kRecGroup + i) * kP + lane * V, w[i]);
+#pragma unroll
+          for (int e = 0; e < V; ++e) w[i][e] = warp * kRecGroup + i < n ? wkv_decay<T>(w[i][e], s_base[lane * V + e]) : 1.f;
+        }
+#pragma unroll
+        for (int i = 0; i < 16; ++i) x[i] = 0.f;
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          const float u = s_bonus[lane * V + e];
+#pragma unroll
+          for (int i = 0; i < kRecGroup; ++i) {
+            x[4 * i + i] = fmaf(q[i][e] * u, k[i][e], x[4 * i + i]);
+            float rw = q[i][e];   // r_i times the decays between the two tokens
+#pragma unroll
+            for (int j = i - 1; j >= 0; --j) {
+              x[4 * i + j] = fmaf(rw, k[j][e], x[4 * i + j]);
+              rw *= w[j][e];
+            }
+            q[i][e] = rw;         // now times the decays of all earlier tokens of the group
+          }
+          float after = 1.f;
+#pragma unroll
+          for (int j = kRecGroup - 1; j >= 0; --j) {
+            k[j][e] *= after;
+            after *= w[j][e];
+          }
+          total[e] = after;
+        }
+        store_few<V>(sw + warp * kP + lane * V, total);
+        const float dot = warp_sums<16>(x);
+        if (lane < 16) s_n[warp * 16 + lane] = dot;
       } else {
+        float x[32];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          x = fmaf(q8[i], q8[i], x);
-          y = fmaf(k8[i], k8[i], y);
-          z = fmaf(q8[i], k8[i], z);
+        for (int i = 0; i < 32; ++i) x[i] = 0.f;
+#pragma unroll
+        for (int e = 0; e < V; ++e)
+#pragma unroll
+          for (int i = 0; i < kRecGroup; ++i) {
+            x[16 + i] = fmaf(q[i][e], q[i][e], x[16 + i]);
+            x[20 + i] = fmaf(k[i][e], k[i][e], x[20 + i]);
+#pragma unroll
+            for (int j = 0; j < kRecGroup; ++j) x[4 * i + j] = fmaf(j <= i ? q[i][e] : k[i][e], k[j][e], x[4 * i + j]);  // k_j . q_i, or k_i . k_j
+          }
+        float* dot = s_dot + warp * 32;
+        const int tok = warp * kRecGroup + lane;
+        dot[lane] = warp_sums<32>(x);
+        if (lane < kRecGroup) {
+          s_g[tok] = tok < n ? delta_decay(ra, A, dt) : 1.f;
+          s_beta[tok] = tok < n ? 1.f / (1.f + expf(-rb)) : 0.f;
+        }
+        __syncwarp();
+        const float* g = s_g + warp * kRecGroup;
+        const float root = sqrtf(static_cast<float>(p.D));
+        if (lane < 16) {
+          const int i = lane >> 2, j = lane & 3, lo = min(i, j), hi = max(i, j);
+          float G = dot[lane] / sqrtf(dot[20 + j] + 1e-6f);
+          for (int l = lo + 1; l <= hi; ++l) G *= g[l];
+          if (j <= i) s_n[(warp * kRecGroup + i) * 4 + j] = G / (sqrtf(dot[16 + i] + 1e-6f) * root);
+          else s_m[(warp * kRecGroup + j) * 4 + i] = G / sqrtf(dot[20 + i] + 1e-6f);
+        } else if (lane < 16 + kRecGroup) {
+          const int i = lane - 16;
+          float c = 1.f, tail = 1.f;
+          for (int l = 0; l <= i; ++l) c *= g[l];
+          for (int l = i + 1; l < kRecGroup; ++l) tail *= g[l];
+          s_c[warp * kRecGroup + i] = c;
+          s_tail[warp * kRecGroup + i] = tail;
+        }
+#pragma unroll
+        for (int i = 0; i < kRecGroup; ++i) {
+          const float iq = 1.f / (sqrtf(dot[16 + i] + 1e-6f) * root), ik = 1.f / sqrtf(dot[20 + i] + 1e-6f);
+#pragma unroll
+          for (int e = 0; e < V; ++e) {
+            q[i][e] *= iq;
+            k[i][e] *= ik;
+          }
         }
       }
 #pragma unroll
-      for (int o = kP / 16; o > 0; o >>= 1) {
-        if (kKind == kDelta) {
-          x += __shfl_xor_sync(0xffffffffu, x, o);
-          y += __shfl_xor_sync(0xffffffffu, y, o);
-        }
-        z += __shfl_xor_sync(0xffffffffu, z, o);
+      for (int i = 0; i < kRecGroup; ++i) {
+        store_few<V>(sq + (warp * kRecGroup + i) * kP + lane * V, q[i]);
+        store_few<V>(sk + (warp * kRecGroup + i) * kP + lane * V, k[i]);
       }
-      if (kKind == kDelta) {
-        const float iq = 1.f / (sqrtf(x + 1e-6f) * sqrtf(static_cast<float>(p.D))), ik = 1.f / sqrtf(y + 1e-6f);
-        z *= iq * ik;
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          q8[i] *= iq;
-          k8[i] *= ik;
-        }
-      }
-      if (ic == 0) s_qk[it] = z;
-      store8(sq + it * kP + ic, q8);
-      store8(sk + it * kP + ic, k8);
-      if (kKind == kWkv) {
-        load8(mine_raw + 2 * kRaw, f);
-#pragma unroll
-        for (int i = 0; i < 8; ++i) f[i] = wkv_decay(f[i], s_base[ic + i]);
-        store8(sw + it * kP + ic, f);
-      }
-      load8(mine_raw + 3 * kRaw, f);
-      store8(sv + it * kP + ic, f);
-      load8(mine_raw + 4 * kRaw, f);
-#pragma unroll
-      for (int i = 0; i < 8; ++i) f[i] = silu(f[i]);
-      store8(sg + it * kP + ic, f);
     }
-    if (kKind == kDelta && threadIdx.x < kRecTokens) {
-      s_decay[threadIdx.x] = delta_decay(ra, A, dt);
-      s_beta[threadIdx.x] = 1.f / (1.f + expf(-rb));
+    if (kWarps == kRecGroups || warp >= kRecGroups) {
+      constexpr int kFirst = kThreads - 32 * kRecGroups;   // 128 threads, eight elements at a time
+#pragma unroll
+      for (int at = (threadIdx.x - kFirst) * 8; at < kRaw; at += 32 * kRecGroups * 8) {
+        float f[8];
+        load8(raw + 3 * kRaw + at, f);
+        store8(sv + at, f);
+        load8(raw + 4 * kRaw + at, f);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] = silu<T>(f[i]);
+        store8(sg + at, f);
+      }
     }
     __syncthreads();
     if (t0 + kRecTokens < p.S) fetch(t0 + kRecTokens);
     // ---- the tokens of the chunk
 #pragma unroll 1
-    for (int t = 0; t < n; ++t) {
-      // four rows of this thread out of a row vector of token t
-      auto four = [&](const float* x, int i) { return *reinterpret_cast<const ulonglong2*>(x + t * kP + 32 * i + 4 * kg); };
-      const float4 v4 = *reinterpret_cast<const float4*>(sv + t * kP + col0);
-      const float v[4] = {v4.x, v4.y, v4.z, v4.w};
-      float o[4], d[4];
-      if (kKind == kDelta) {
-        f32x2 oa[C], da[C], kv[R / 2];
+    for (int grp = 0; grp < n_groups; ++grp) {
+      const int tok = grp * kRecGroup;
+      // four rows of this thread out of a row vector
+      auto four = [&](const float* x, int i) { return *reinterpret_cast<const ulonglong2*>(x + 32 * i + 4 * kg); };
+      // per-token partial sums of this thread's rows with the memory
+      auto products = [&](const float* x, float (&o)[kRecGroup][C]) {
+        f32x2 acc[kRecGroup][C];
 #pragma unroll
-        for (int c = 0; c < C; ++c) oa[c] = da[c] = 0ull;
+        for (int t = 0; t < kRecGroup; ++t)
+#pragma unroll
+          for (int c = 0; c < C; ++c) acc[t][c] = 0ull;
+#pragma unroll
+        for (int i = 0; i < R / 4; ++i)
+#pragma unroll
+          for (int t = 0; t < kRecGroup; ++t) {
+            const ulonglong2 x2 = four(x + (tok + t) * kP, i);
+#pragma unroll
+            for (int c = 0; c < C; ++c) {
+              acc[t][c] = fma2(x2.x, s[2 * i][c], acc[t][c]);
+              acc[t][c] = fma2(x2.y, s[2 * i + 1][c], acc[t][c]);
+            }
+          }
+#pragma unroll
+        for (int t = 0; t < kRecGroup; ++t)
+#pragma unroll
+          for (int c = 0; c < C; ++c) o[t][c] = sum2(acc[t][c]);
+      };
+      const bool b2 = (kg & 4) != 0, b1 = (kg & 2) != 0, b0 = (kg & 1) != 0;
+      if (kKind == kWkv) {
+        float o[kRecGroup][C];
+        products(sq, o);
+        // sums over the eight lanes; lane kg is left with token kg >> 1 and a pair of columns
+        float x[2][C], y[C], z[2];
+#pragma unroll
+        for (int t = 0; t < 2; ++t)
+#pragma unroll
+          for (int c = 0; c < C; ++c) x[t][c] = (b2 ? o[t + 2][c] : o[t][c]) + __shfl_xor_sync(0xffffffffu, b2 ? o[t][c] : o[t + 2][c], 4);
+#pragma unroll
+        for (int c = 0; c < C; ++c) y[c] = (b1 ? x[1][c] : x[0][c]) + __shfl_xor_sync(0xffffffffu, b1 ? x[0][c] : x[1][c], 2);
+#pragma unroll
+        for (int c = 0; c < 2; ++c) z[c] = (b0 ? y[c + 2] : y[c]) + __shfl_xor_sync(0xffffffffu, b0 ? y[c] : y[c + 2], 1);
+        f32x2 v2[kRecGroup][C];
+#pragma unroll
+        for (int t = 0; t < kRecGroup; ++t) {
+          const float4 v = *reinterpret_cast<const float4*>(sv + (tok + t) * kP + col0);
+          v2[t][0] = pack2(v.x, v.x); v2[t][1] = pack2(v.y, v.y); v2[t][2] = pack2(v.z, v.z); v2[t][3] = pack2(v.w, v.w);
+        }
 #pragma unroll
         for (int i = 0; i < R / 4; ++i) {
-          const ulonglong2 q2 = four(sq, i), k2 = four(sk, i);
-          kv[2 * i] = k2.x;
-          kv[2 * i + 1] = k2.y;
+          const ulonglong2 w2 = four(sw + grp * kP, i);
 #pragma unroll
           for (int c = 0; c < C; ++c) {
-            da[c] = fma2(k2.x, s[2 * i][c], da[c]);
-            oa[c] = fma2(q2.x, s[2 * i][c], oa[c]);
-            da[c] = fma2(k2.y, s[2 * i + 1][c], da[c]);
-            oa[c] = fma2(q2.y, s[2 * i + 1][c], oa[c]);
+            s[2 * i][c] = mul2(w2.x, s[2 * i][c]);
+            s[2 * i + 1][c] = mul2(w2.y, s[2 * i + 1][c]);
+          }
+#pragma unroll
+          for (int t = 0; t < kRecGroup; ++t) {
+            const ulonglong2 k2 = four(sk + (tok + t) * kP, i);
+#pragma unroll
+            for (int c = 0; c < C; ++c) {
+              s[2 * i][c] = fma2(k2.x, v2[t][c], s[2 * i][c]);
+              s[2 * i + 1][c] = fma2(k2.y, v2[t][c], s[2 * i + 1][c]);
+            }
           }
         }
+        const int mine = tok + (kg >> 1), col = col0 + 2 * (kg & 1);
+        const float4 co = *reinterpret_cast<const float4*>(s_n + mine * 4);
+        const float f[kRecGroup] = {co.x, co.y, co.z, co.w};
 #pragma unroll
-        for (int c = 0; c < C; ++c) {
-          d[c] = sum2(da[c]);
-          o[c] = sum2(oa[c]);
+        for (int j = 0; j < kRecGroup; ++j) {
+          const float2 v = *reinterpret_cast<const float2*>(sv + (tok + j) * kP + col);
+          z[0] = fmaf(f[j], v.x, z[0]);
+          z[1] = fmaf(f[j], v.y, z[1]);
         }
-#pragma unroll
-        for (int m = 1; m < 8; m <<= 1)
-#pragma unroll
-          for (int c = 0; c < C; ++c) d[c] += __shfl_xor_sync(0xffffffffu, d[c], m);
-        const float g = s_decay[t], beta = s_beta[t];
-        const f32x2 g2 = pack2(g, g);
-#pragma unroll
-        for (int c = 0; c < C; ++c) {
-          d[c] = beta * (v[c] - g * d[c]);
-          const f32x2 d2 = pack2(d[c], d[c]);
-#pragma unroll
-          for (int i = 0; i < R / 2; ++i) s[i][c] = fma2(kv[i], d2, mul2(g2, s[i][c]));
-        }
+        *reinterpret_cast<float2*>(so + mine * kP + col) = make_float2(z[0], z[1]);
       } else {
-        f32x2 oa[C], v2[C];
+        // sums over the eight lanes; lanes kg and kg ^ 1 are left with column kg >> 1, all four tokens
+        auto column_sums = [&](const float (&o)[kRecGroup][C], float (&r)[kRecGroup]) {
+          float x[kRecGroup][2];
 #pragma unroll
-        for (int c = 0; c < C; ++c) {
-          oa[c] = 0ull;
-          v2[c] = pack2(v[c], v[c]);
-          d[c] = v[c];
+          for (int t = 0; t < kRecGroup; ++t)
+#pragma unroll
+            for (int c = 0; c < 2; ++c) x[t][c] = (b2 ? o[t][c + 2] : o[t][c]) + __shfl_xor_sync(0xffffffffu, b2 ? o[t][c] : o[t][c + 2], 4);
+#pragma unroll
+          for (int t = 0; t < kRecGroup; ++t) r[t] = (b1 ? x[t][1] : x[t][0]) + __shfl_xor_sync(0xffffffffu, b1 ? x[t][0] : x[t][1], 2);
+#pragma unroll
+          for (int t = 0; t < kRecGroup; ++t) r[t] += __shfl_xor_sync(0xffffffffu, r[t], 1);
+        };
+        float part[kRecGroup][C], a[kRecGroup], o[kRecGroup], d[kRecGroup];
+        products(sk, part);
+        column_sums(part, a);
+        products(sq, part);
+        column_sums(part, o);
+        const int col = col0 + (kg >> 1);
+#pragma unroll
+        for (int i = 0; i < kRecGroup; ++i) {
+          const float c = s_c[tok + i];
+          float t = sv[(tok + i) * kP + col] - c * a[i];
+#pragma unroll
+          for (int j = 0; j < i; ++j) t = fmaf(-s_m[(tok + i) * 4 + j], d[j], t);
+          d[i] = s_beta[tok + i] * t;
+          o[i] *= c;
+#pragma unroll
+          for (int j = 0; j <= i; ++j) o[i] = fmaf(s_n[(tok + i) * 4 + j], d[j], o[i]);
         }
+        so[(tok + (b0 ? 2 : 0)) * kP + col] = b0 ? o[2] : o[0];
+        so[(tok + (b0 ? 3 : 1)) * kP + col] = b0 ? o[3] : o[1];
+        f32x2 d2[kRecGroup][C];   // the weighted d of the thread's four columns
+#pragma unroll
+        for (int t = 0; t < kRecGroup; ++t) {
+          const float own = s_tail[tok + t] * d[t], near = __shfl_xor_sync(0xffffffffu, own, 2);
+          const float p0 = b1 ? near : own, p1 = b1 ? own : near;
+          const float f0 = __shfl_xor_sync(0xffffffffu, p0, 4), f1 = __shfl_xor_sync(0xffffffffu, p1, 4);
+          const float e[C] = {b2 ? f0 : p0, b2 ? f1 : p1, b2 ? p0 : f0, b2 ? p1 : f1};
+#pragma unroll
+          for (int c = 0; c < C; ++c) d2[t][c] = pack2(e[c], e[c]);
+        }
+        const float all = s_c[tok + kRecGroup - 1];
+        const f32x2 g2 = pack2(all, all);
 #pragma unroll
         for (int i = 0; i < R / 4; ++i) {
-          const ulonglong2 q2 = four(sq, i), k2 = four(sk, i), w2 = four(sw, i);
 #pragma unroll
           for (int c = 0; c < C; ++c) {
-            oa[c] = fma2(q2.x, s[2 * i][c], oa[c]);
-            s[2 * i][c] = fma2(w2.x, s[2 * i][c], mul2(k2.x, v2[c]));
-            oa[c] = fma2(q2.y, s[2 * i + 1][c], oa[c]);
-            s[2 * i + 1][c] = fma2(w2.y, s[2 * i + 1][c], mul2(k2.y, v2[c]));
+            s[2 * i][c] = mul2(g2, s[2 * i][c]);
+            s[2 * i + 1][c] = mul2(g2, s[2 * i + 1][c]);
+          }
+#pragma unroll
+          for (int t = 0; t < kRecGroup; ++t) {
+            const ulonglong2 k2 = four(sk + (tok + t) * kP, i);
+#pragma unroll
+            for (int c = 0; c < C; ++c) {
+              s[2 * i][c] = fma2(k2.x, d2[t][c], s[2 * i][c]);
+              s[2 * i + 1][c] = fma2(k2.y, d2[t][c], s[2 * i + 1][c]);
+            }
           }
         }
-#pragma unroll
-        for (int c = 0; c < C; ++c) o[c] = sum2(oa[c]);
       }
-      // ---- sum over the eight lanes of a column group; lane kg is left with column (kg >> 1) of the group (kg bit 2 picks the
-      // pair, bit 1 the member)
-      const bool hi2 = (kg & 4) != 0, hi1 = (kg & 2) != 0;
-      float k0 = hi2 ? o[2] : o[0], k1 = hi2 ? o[3] : o[1];
-      k0 += __shfl_xor_sync(0xffffffffu, hi2 ? o[0] : o[2], 4);
-      k1 += __shfl_xor_sync(0xffffffffu, hi2 ? o[1] : o[3], 4);
-      float r = hi1 ? k1 : k0;
-      r += __shfl_xor_sync(0xffffffffu, hi1 ? k0 : k1, 2);
-      r += __shfl_xor_sync(0xffffffffu, r, 1);
-      const float mine = hi2 ? (hi1 ? d[3] : d[2]) : (hi1 ? d[1] : d[0]);
-      if ((kg & 1) == 0) so[t * kP + col0 + (kg >> 1)] = fmaf(s_qk[t], mine, kKind == kDelta ? s_decay[t] * r : r);
     }
     __syncthreads();
     // ---- norm over the head, gain, gate: one warp per token
@@ -401,7 +583,6 @@ __global__ void __launch_bounds__(kP * kP / (R * 4), kP == 128 ? 2 : 4) recurren
               from_float<T>(o[i] * inv * p.gain[h * p.gain_stride + c] * sg[t * kP + c]);
       }
     }
-    __syncthreads();
   }
 #pragma unroll
   for (int i = 0; i < R / 4; ++i)
@@ -445,7 +626,7 @@ __global__ void __launch_bounds__(256) recurrent_plain_kernel(const RecurrentPar
       x = fmaf(q, q, x);
       y = fmaf(k, k, y);
       z = kKind == kWkv ? fmaf(q * p.bonus[h * p.Dp + i], k, z) : fmaf(q, k, z);
-      if (kKind == kWkv) sw[i] = wkv_decay(to_float(static_cast<const T*>(p.decay)[row * p.ld_decay + h * p.Dp + i]), p.decay_base[h * p.Dp + i]);
+      if (kKind == kWkv) sw[i] = wkv_decay<T>(to_float(static_cast<const T*>(p.decay)[row * p.ld_decay + h * p.Dp + i]), p.decay_base[h * p.Dp + i]);
     }
     z = cta_sum(z, red);
     float g = 1.f, beta = 1.f;
@@ -481,28 +662,28 @@ __global__ void __launch_bounds__(256) recurrent_plain_kernel(const RecurrentPar
     const float inv = 1.f / sqrtf(cta_sum(ss, red) / p.E + p.eps);
     for (int c = threadIdx.x; c < p.Ep; c += blockDim.x)
       static_cast<T*>(p.out)[row * p.H * p.Ep + h * p.Ep + c] = from_float<T>(
-          so[c] * inv * p.gain[h * p.gain_stride + c] * silu(to_float(static_cast<const T*>(p.gate)[row * p.ldg + h * p.Ep + c])));
+          so[c] * inv * p.gain[h * p.gain_stride + c] * silu<T>(to_float(static_cast<const T*>(p.gate)[row * p.ldg + h * p.Ep + c])));
   }
 }
 
-template <typename T, int kKind, int kP, int R>
+template <typename T, int kKind, int kP>
 static int launch_recurrent(const RecurrentParams& p, int B, cudaStream_t s) {
   static bool configured[64] = {false};
   int dev = 0;
   B200_CHECK_CUDA(cudaGetDevice(&dev));
   if (!configured[dev & 63]) {
-    B200_CHECK_CUDA(cudaFuncSetAttribute(recurrent_kernel<T, kKind, kP, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, recurrent_smem(kP, sizeof(T))));
+    B200_CHECK_CUDA(cudaFuncSetAttribute(recurrent_kernel<T, kKind, kP>, cudaFuncAttributeMaxDynamicSharedMemorySize, recurrent_smem(kP, sizeof(T))));
     configured[dev & 63] = true;
   }
-  B200_CHECK_CUDA(launch_pdl(recurrent_kernel<T, kKind, kP, R>, dim3(p.H, B), dim3(kP * kP / (R * 4)), recurrent_smem(kP, sizeof(T)), s, p));
+  B200_CHECK_CUDA(launch_pdl(recurrent_kernel<T, kKind, kP>, dim3(p.H, B), dim3(2 * kP), recurrent_smem(kP, sizeof(T)), s, p));
   return kOk;
 }
 
 template <typename T, int kKind>
 static int dispatch_recurrent(const RecurrentParams& p, int B, int plain, cudaStream_t s) {
   const int size = p.Dp > p.Ep ? p.Dp : p.Ep;
-  if (!plain && size <= 64) return launch_recurrent<T, kKind, 64, 8>(p, B, s);
-  if (!plain && size <= 128) return launch_recurrent<T, kKind, 128, 16>(p, B, s);
+  if (!plain && size <= 64) return launch_recurrent<T, kKind, 64>(p, B, s);
+  if (!plain && size <= 128) return launch_recurrent<T, kKind, 128>(p, B, s);
   const int smem = (3 * p.Dp + p.Ep) * 4;
   B200_REQUIRE(smem <= 48 * 1024, "heads of %d x %d are too large", p.Dp, p.Ep);
   B200_CHECK_CUDA(launch_pdl(recurrent_plain_kernel<T, kKind>, dim3(p.H, B), dim3(256), smem, s, p));
@@ -535,6 +716,17 @@ B200_API int b200_token_mix(const void* h, const void* mu, void* last, void* out
   B200_DISPATCH_FLOAT(dtype, switch (G) { B200_MIX(1) B200_MIX(2) B200_MIX(3) B200_MIX(4) B200_MIX(5) B200_MIX(6) B200_MIX(7) B200_MIX(8) });
 #undef B200_MIX
   return kOk;
+}
+
+// out [rows, cols] = tanh(x), x with row pitch ldx; cols and ldx: multiples of 4.
+B200_API int b200_tanh_rows(const void* x, void* out, int rows, int cols, int ldx, int dtype, void* stream) {
+  if (rows <= 0) return kOk;
+  B200_REQUIRE(cols >= 4 && cols % 4 == 0 && ldx % 4 == 0, "tanh_rows: columns (%d) and pitch (%d) must be multiples of 4", cols, ldx);
+  const size_t n = static_cast<size_t>(rows) * (cols / 4);
+  B200_DISPATCH_FLOAT(dtype, B200_CHECK_CUDA(launch_pdl(tanh_rows_kernel<T>, dim3(static_cast<unsigned>((n + 255) / 256)), dim3(256), 0,
+                                                        static_cast<cudaStream_t>(stream), static_cast<const T*>(x), static_cast<T*>(out),
+                                                        rows, cols, ldx));
+                      return kOk;);
 }
 
 // out = silu(sum_j taps[j] * x[t - n + 1 + j]); last [B, n - 1, C] carries the inputs before the call. C and ldx: multiples of 4.

@@ -41,7 +41,7 @@ class WkvMixer:
         mats = [pad_matrix(m, pad_up(m.shape[0], 128), width_pad) for m in mats]
         self.rows = [m.shape[0] for m in mats]
         self.w_in = torch.cat(mats).contiguous()
-        self.w2 = pad_heads(get("w2", rows=N), H, D, self.rank)[None].contiguous()   # [1, heads * dim, rank]
+        self.w2 = pad_heads(get("w2", rows=N), H, D, self.rank)   # [heads * dim, rank]
         self.w0, self.gain = _head_vector(get("w0", rows=N), H, D), _head_vector(get("norm", rows=N), H, D)
         self.u = _head_vector(get("u", rows=H), H, D)
         self.wo = pad_heads(get("o", cols=N).t().contiguous(), H, D, width_pad).t().contiguous()
@@ -55,7 +55,7 @@ class WkvMixer:
         mixes = ops.token_mix(h, self.mu, cache.state(layer_idx, "last"))
         r, k, v, gate, low = ops.linear_groups(mixes, self.w_in, self.rows).split(self.rows, dim=1)
         N = self.heads * self.dim
-        z = ops.head_linear(low[:, None, : self.rank], self.w2, tanh=True)[:, 0]
+        z = ops.tanh_linear(low[:, : self.rank], self.w2)
         o = ops.wkv(r[:, :N], k[:, :N], v[:, :N], z, gate[:, :N], self.w0, self.u, self.gain, cache.state(layer_idx, "memory"), self.spec.dim,
                     self.spec.dim, self.eps)
         return ops.linear(o, self.wo, out=out)

@@ -625,6 +625,18 @@ def token_mix(h: torch.Tensor, mu: torch.Tensor, last: torch.Tensor) -> torch.Te
     return out
 
 
+def tanh_linear(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """``tanh(x) @ w.T``, the second half of a low-rank map: x [T, K] (rows may be strided), w [N, K]. One launch for few tokens, tanh
+    and the tiled GEMM for many."""
+    if x.shape[0] <= 256:
+        return head_linear(x[:, None], w[None], tanh=True)[:, 0]
+    _check_2d(x, "x")
+    act = torch.empty(x.shape, dtype=x.dtype, device=x.device)
+    _lib.call("b200_tanh_rows", ptr(x), ptr(act), x.shape[0], x.shape[1], x.stride(0), dtype_code(x.dtype), stream_ptr())
+    _count()
+    return linear(act, w)
+
+
 def short_conv(x: torch.Tensor, taps: torch.Tensor, last: torch.Tensor) -> torch.Tensor:
     """Causal convolution per channel, then silu: x [B * S, C] (rows may be strided), taps fp32 [n, C] (the last weighs the current
     token), ``last`` [B, n - 1, C] the inputs before the call, replaced by the last ones of the call. Returns [B * S, C]."""
