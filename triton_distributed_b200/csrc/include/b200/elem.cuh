@@ -37,6 +37,21 @@ __device__ __forceinline__ void store4(__half* p, float4 v) {
   *reinterpret_cast<uint2*>(p) = make_uint2(pack_f16x2(v.x, v.y), pack_f16x2(v.z, v.w));
 }
 
+// Functions of fp32 values on their way into storage of type T: the math library's in the 32-bit mode; with 16-bit storage short
+// forms whose error (about 1e-6) is far below a rounding of the result.
+template <typename T>
+__device__ __forceinline__ float exp_t(float z) { return sizeof(T) == 4 ? expf(z) : __expf(z); }
+template <typename T>
+__device__ __forceinline__ float silu(float z) { return sizeof(T) == 4 ? z / (1.f + expf(-z)) : __fdividef(z, 1.f + __expf(-z)); }
+template <typename T>
+__device__ __forceinline__ float inv_sqrt(float z) { return sizeof(T) == 4 ? 1.f / sqrtf(z) : rsqrtf(z); }
+template <typename T>
+__device__ __forceinline__ float tanh_t(float z) {
+  if (sizeof(T) == 4) return tanhf(z);
+  const float e = __expf(-2.f * fabsf(z));   // tanh |z| = (1 - e) / (1 + e)
+  return copysignf(__fdividef(1.f - e, 1.f + e), z);
+}
+
 }  // namespace b200
 
 // Runs `...` with the type alias T bound to the element type of a dtype code (bf16, f16 or f32).

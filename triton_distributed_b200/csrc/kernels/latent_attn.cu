@@ -84,7 +84,8 @@ enum HeadLinearAct : int { kActNone = 0, kActTanh = 1 };   // applied to x on it
 template <bool BF16>
 __device__ __forceinline__ uint32_t tanh_pair(uint32_t v) {
   const float2 f = BF16 ? unpack_bf16x2(v) : unpack_f16x2(v);
-  return BF16 ? pack_bf16x2(tanhf(f.x), tanhf(f.y)) : pack_f16x2(tanhf(f.x), tanhf(f.y));
+  const float x = tanh_t<__half>(f.x), y = tanh_t<__half>(f.y);   // the same for both 16-bit types
+  return BF16 ? pack_bf16x2(x, y) : pack_f16x2(x, y);
 }
 
 constexpr int kHlTok = 4;  // token tiles of 8 per CTA

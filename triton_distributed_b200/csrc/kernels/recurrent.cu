@@ -26,12 +26,6 @@
 
 namespace b200 {
 
-// exponential and quotient: the library's functions in the 32-bit mode, the short fp32 forms with 16-bit storage
-template <typename T>
-__device__ __forceinline__ float exp_t(float z) { return sizeof(T) == 4 ? expf(z) : __expf(z); }
-template <typename T>
-__device__ __forceinline__ float silu(float z) { return sizeof(T) == 4 ? z / (1.f + expf(-z)) : __fdividef(z, 1.f + __expf(-z)); }
-
 // ------------------------------------------------------------------------------------------------ token_mix
 constexpr int kMixMax = 8;       // mixes per call
 constexpr int kMixTokens = 8;    // tokens per thread
@@ -84,7 +78,7 @@ __global__ void __launch_bounds__(256) tanh_rows_kernel(const T* x, T* out, int 
   const size_t t = at / groups;
   const int c = static_cast<int>(at - t * groups) * 4;
   const float4 v = load4(x + t * ldx + c);
-  store4(out + t * cols + c, make_float4(tanhf(v.x), tanhf(v.y), tanhf(v.z), tanhf(v.w)));
+  store4(out + t * cols + c, make_float4(tanh_t<T>(v.x), tanh_t<T>(v.y), tanh_t<T>(v.z), tanh_t<T>(v.w)));
 }
 
 // ------------------------------------------------------------------------------------------------ short_conv
@@ -190,7 +184,7 @@ constexpr int kRecTokens = 16;   // tokens per chunk
 constexpr int kRecGroup = 4;     // tokens per pass over the memory
 constexpr int kRecGroups = kRecTokens / kRecGroup;
 constexpr int recurrent_smem(int p, int elem) {
-  return (5 * kRecTokens * p + kRecGroups * p + 2 * p + kRecTokens * 8 + kRecGroups * 32 + 4 * kRecTokens) * 4 + 5 * kRecTokens * p * elem;
+  return (4 * kRecTokens * p + kRecGroups * p + 3 * p + kRecTokens * 8 + kRecGroups * 32 + 4 * kRecTokens) * 4 + 5 * kRecTokens * p * elem;
 }
 
 // sums over the warp of N = 16 or 32 values; lane l is left with the sum of v[l % N]
@@ -244,12 +238,12 @@ __global__ void __launch_bounds__(2 * kP, kP == 128 ? 2 : 4) recurrent_kernel(co
   float* sq = smf;                            // [tokens][kP] read-out vectors
   float* sk = sq + kRaw;                      // [tokens][kP]
   float* sv = sk + kRaw;
-  float* sg = sv + kRaw;                      // silu(gate)
-  float* so = sg + kRaw;
+  float* so = sv + kRaw;
   float* sw = so + kRaw;                      // kWkv: [groups][kP] product of the decays
   float* s_base = sw + kRecGroups * kP;       // kWkv: w0 and u of the head
   float* s_bonus = s_base + kP;
-  float* s_n = s_bonus + kP;                  // [tokens][4] coefficients of o_i on v_j (kWkv) / d_j (kDelta)
+  float* s_gain = s_bonus + kP;
+  float* s_n = s_gain + kP;                   // [tokens][4] coefficients of o_i on v_j (kWkv) / d_j (kDelta)
   float* s_m = s_n + kRecTokens * 4;          // kDelta: [tokens][4] coefficients of d_i on d_j
   float* s_dot = s_m + kRecTokens * 4;        // [groups][32]
   float* s_c = s_dot + kRecGroups * 32;       // kDelta: c_i, G_3i, beta_i, g_i per token
@@ -265,6 +259,7 @@ __global__ void __launch_bounds__(2 * kP, kP == 128 ? 2 : 4) recurrent_kernel(co
   // the state comes from an earlier call: it may be fetched into L2, but not read, before that call is known to be over
   for (int i = threadIdx.x * 32; i < p.Dp * p.Ep; i += kThreads * 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(state + i));
   const int ic = threadIdx.x % (kP / 8) * 8, it = threadIdx.x / (kP / 8);   // this thread's eight elements of a chunk
+  if (threadIdx.x < kP) s_gain[threadIdx.x] = threadIdx.x < p.Ep ? p.gain[h * p.gain_stride + threadIdx.x] : 0.f;
   if (kKind == kWkv && threadIdx.x < kP) {
     const bool in = threadIdx.x < p.Dp;
     s_base[threadIdx.x] = in ? p.decay_base[h * p.Dp + threadIdx.x] : 0.f;
@@ -313,7 +308,14 @@ __global__ void __launch_bounds__(2 * kP, kP == 128 ? 2 : 4) recurrent_kernel(co
     const int n = min(kRecTokens, p.S - t0), n_groups = (n + kRecGroup - 1) / kRecGroup;
     cp_async_wait<0>();
     __syncthreads();   // the raw chunk of all threads; the last chunk's results have been read
-    // ---- prepare: warp w the vectors of group w (a lane owns V channels), values and gates by the other warps if there are any
+    // ---- prepare: every thread its own values; warp w the vectors of group w, a lane V channels
+    float gate[8];   // of this thread's results
+    {
+      float f[8];
+      load8(raw + 3 * kRaw + it * kP + ic, f);
+      store8(sv + it * kP + ic, f);
+      load8(raw + 4 * kRaw + it * kP + ic, gate);
+    }
     if (warp < n_groups) {
       float q[kRecGroup][V], k[kRecGroup][V];
 #pragma unroll
@@ -409,19 +411,6 @@ __global__ void __launch_bounds__(2 * kP, kP == 128 ? 2 : 4) recurrent_kernel(co
         store_few<V>(sk + (warp * kRecGroup + i) * kP + lane * V, k[i]);
       }
     }
-    if (kWarps == kRecGroups || warp >= kRecGroups) {
-      constexpr int kFirst = kThreads - 32 * kRecGroups;   // 128 threads, eight elements at a time
-#pragma unroll
-      for (int at = (threadIdx.x - kFirst) * 8; at < kRaw; at += 32 * kRecGroups * 8) {
-        float f[8];
-        load8(raw + 3 * kRaw + at, f);
-        store8(sv + at, f);
-        load8(raw + 4 * kRaw + at, f);
-#pragma unroll
-        for (int i = 0; i < 8; ++i) f[i] = silu<T>(f[i]);
-        store8(sg + at, f);
-      }
-    }
     __syncthreads();
     if (t0 + kRecTokens < p.S) fetch(t0 + kRecTokens);
     // ---- the tokens of the chunk
@@ -434,17 +423,13 @@ __global__ void __launch_bounds__(2 * kP, kP == 128 ? 2 : 4) recurrent_kernel(co
       auto products = [&](const float* x, float (&o)[kRecGroup][C]) {
         f32x2 acc[kRecGroup][C];
 #pragma unroll
-        for (int t = 0; t < kRecGroup; ++t)
-#pragma unroll
-          for (int c = 0; c < C; ++c) acc[t][c] = 0ull;
-#pragma unroll
         for (int i = 0; i < R / 4; ++i)
 #pragma unroll
           for (int t = 0; t < kRecGroup; ++t) {
             const ulonglong2 x2 = four(x + (tok + t) * kP, i);
 #pragma unroll
             for (int c = 0; c < C; ++c) {
-              acc[t][c] = fma2(x2.x, s[2 * i][c], acc[t][c]);
+              acc[t][c] = i == 0 ? mul2(x2.x, s[0][c]) : fma2(x2.x, s[2 * i][c], acc[t][c]);
               acc[t][c] = fma2(x2.y, s[2 * i + 1][c], acc[t][c]);
             }
           }
@@ -520,31 +505,36 @@ __global__ void __launch_bounds__(2 * kP, kP == 128 ? 2 : 4) recurrent_kernel(co
         products(sq, part);
         column_sums(part, o);
         const int col = col0 + (kg >> 1);
+        float c4[4], beta[4], tail[4];
+        load_few<float, 4>(s_c + tok, c4);
+        load_few<float, 4>(s_beta + tok, beta);
+        load_few<float, 4>(s_tail + tok, tail);
 #pragma unroll
         for (int i = 0; i < kRecGroup; ++i) {
-          const float c = s_c[tok + i];
-          float t = sv[(tok + i) * kP + col] - c * a[i];
+          float m[4], e[4];
+          load_few<float, 4>(s_m + (tok + i) * 4, m);
+          load_few<float, 4>(s_n + (tok + i) * 4, e);
+          float t = fmaf(-c4[i], a[i], sv[(tok + i) * kP + col]);
 #pragma unroll
-          for (int j = 0; j < i; ++j) t = fmaf(-s_m[(tok + i) * 4 + j], d[j], t);
-          d[i] = s_beta[tok + i] * t;
-          o[i] *= c;
+          for (int j = 0; j < i; ++j) t = fmaf(-m[j], d[j], t);
+          d[i] = beta[i] * t;
+          o[i] *= c4[i];
 #pragma unroll
-          for (int j = 0; j <= i; ++j) o[i] = fmaf(s_n[(tok + i) * 4 + j], d[j], o[i]);
+          for (int j = 0; j <= i; ++j) o[i] = fmaf(e[j], d[j], o[i]);
         }
         so[(tok + (b0 ? 2 : 0)) * kP + col] = b0 ? o[2] : o[0];
         so[(tok + (b0 ? 3 : 1)) * kP + col] = b0 ? o[3] : o[1];
         f32x2 d2[kRecGroup][C];   // the weighted d of the thread's four columns
 #pragma unroll
         for (int t = 0; t < kRecGroup; ++t) {
-          const float own = s_tail[tok + t] * d[t], near = __shfl_xor_sync(0xffffffffu, own, 2);
+          const float own = tail[t] * d[t], near = __shfl_xor_sync(0xffffffffu, own, 2);
           const float p0 = b1 ? near : own, p1 = b1 ? own : near;
           const float f0 = __shfl_xor_sync(0xffffffffu, p0, 4), f1 = __shfl_xor_sync(0xffffffffu, p1, 4);
           const float e[C] = {b2 ? f0 : p0, b2 ? f1 : p1, b2 ? p0 : f0, b2 ? p1 : f1};
 #pragma unroll
           for (int c = 0; c < C; ++c) d2[t][c] = pack2(e[c], e[c]);
         }
-        const float all = s_c[tok + kRecGroup - 1];
-        const f32x2 g2 = pack2(all, all);
+        const f32x2 g2 = pack2(c4[kRecGroup - 1], c4[kRecGroup - 1]);
 #pragma unroll
         for (int i = 0; i < R / 4; ++i) {
 #pragma unroll
@@ -565,22 +555,23 @@ __global__ void __launch_bounds__(2 * kP, kP == 128 ? 2 : 4) recurrent_kernel(co
       }
     }
     __syncthreads();
-    // ---- norm over the head, gain, gate: one warp per token
-    for (int t = warp; t < n; t += kWarps) {
-      constexpr int kCols = kP / 32;
-      float o[kCols], ss = 0.f;
+    // ---- norm over the head, gain, gate: eight columns of a token per thread
+    {
+      float o[8], ss = 0.f;
+      load8(so + it * kP + ic, o);
 #pragma unroll
-      for (int i = 0; i < kCols; ++i) {
-        o[i] = so[t * kP + 32 * i + lane];
-        ss = fmaf(o[i], o[i], ss);
-      }
-      const float inv = 1.f / sqrtf(warp_sum(ss) / p.E + p.eps);
+      for (int i = 0; i < 8; ++i) ss = fmaf(o[i], o[i], ss);
 #pragma unroll
-      for (int i = 0; i < kCols; ++i) {
-        const int c = 32 * i + lane;
-        if (c < p.Ep)
-          static_cast<T*>(p.out)[(row0 + t0 + t) * p.H * p.Ep + h * p.Ep + c] =
-              from_float<T>(o[i] * inv * p.gain[h * p.gain_stride + c] * sg[t * kP + c]);
+      for (int m = kP / 16; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+      const float inv = inv_sqrt<T>(ss / p.E + p.eps);
+      if (it < n && ic < p.Ep) {
+        float f[8];
+        load8(s_gain + ic, f);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] *= o[i] * inv * silu<T>(gate[i]);
+        T* dst = static_cast<T*>(p.out) + (row0 + t0 + it) * p.H * p.Ep + h * p.Ep + ic;
+        store4(dst, make_float4(f[0], f[1], f[2], f[3]));
+        store4(dst + 4, make_float4(f[4], f[5], f[6], f[7]));
       }
     }
   }

@@ -128,10 +128,10 @@ __device__ __forceinline__ void norm_row(const NormParams& n, const Slice<kCl>& 
       if (c >= sl.end) continue;
       float4 o = v[u];
       if (n.kind == kNormTanh) {
-        o.x = tanhf(n.eps * o.x) * gain[u].x + bias[u].x;
-        o.y = tanhf(n.eps * o.y) * gain[u].y + bias[u].y;
-        o.z = tanhf(n.eps * o.z) * gain[u].z + bias[u].z;
-        o.w = tanhf(n.eps * o.w) * gain[u].w + bias[u].w;
+        o.x = tanh_t<T>(n.eps * o.x) * gain[u].x + bias[u].x;
+        o.y = tanh_t<T>(n.eps * o.y) * gain[u].y + bias[u].y;
+        o.z = tanh_t<T>(n.eps * o.z) * gain[u].z + bias[u].z;
+        o.w = tanh_t<T>(n.eps * o.w) * gain[u].w + bias[u].w;
       }
       store4(static_cast<T*>(n.h) + row * n.pitch + c, o);
     }
@@ -281,16 +281,21 @@ __global__ void __launch_bounds__(kRnThreads) residual_norm_kernel(const Residua
   norm_row<T, U, kCl>(p.norm, sl, t, x, gain, bias, red, stats);
 }
 
-// sum over the row of the squares of `v` and `w`, for the whole cluster
+// sums over the row of the squares of `v` and `w`, for the whole cluster
 template <int U, int kCl>
-__device__ __forceinline__ float2 row_squares(const float4 (&v)[U], const float4 (&w)[U], float* red, float2* shared_sums) {
-  float sv = 0.f, sw = 0.f;
+__device__ __forceinline__ float2 row_squares(const float4 (&v)[U], const float4 (&w)[U], float2* red, float2* shared_sums) {
+  float2 s = make_float2(0.f, 0.f);
 #pragma unroll
   for (int u = 0; u < U; ++u) {  // padding columns are zero
-    sv += (v[u].x * v[u].x + v[u].y * v[u].y) + (v[u].z * v[u].z + v[u].w * v[u].w);
-    sw += (w[u].x * w[u].x + w[u].y * w[u].y) + (w[u].z * w[u].z + w[u].w * w[u].w);
+    s.x += (v[u].x * v[u].x + v[u].y * v[u].y) + (v[u].z * v[u].z + v[u].w * v[u].w);
+    s.y += (w[u].x * w[u].x + w[u].y * w[u].y) + (w[u].z * w[u].z + w[u].w * w[u].w);
   }
-  float2 s = make_float2(block_sum(sv, red), block_sum(sw, red));
+  s = make_float2(warp_sum(s.x), warp_sum(s.y));
+  const int lane = threadIdx.x & 31;
+  if (lane == 0) red[threadIdx.x >> 5] = s;
+  __syncthreads();
+  s = lane < static_cast<int>(blockDim.x >> 5) ? red[lane] : make_float2(0.f, 0.f);
+  s = make_float2(warp_sum(s.x), warp_sum(s.y));
   if (kCl > 1) {
     const uint32_t me = cluster_ctarank();
     if (threadIdx.x < kCl) {
@@ -312,44 +317,41 @@ template <typename T, int U, int kCl>
 __global__ void __launch_bounds__(kRnThreads) residual_post_kernel(const PostParams p) {
   __shared__ float red[32];
   __shared__ float4 stats[kCl];
-  __shared__ float2 sums[kCl];
+  __shared__ float2 sums[kCl], red2[32];
   const size_t t = blockIdx.x / kCl;
   const int pitch = p.norm.pitch;
   const Slice<kCl> sl(pitch);
   griddep_launch_dependents();
-  float4 gain[U], bias[U], a[U], b[U];
+  float4 gain[U], bias[U], a[U], b[U], x[U];
   load_norm_weights<T, U, kCl>(p.norm, sl, gain, bias);
   if (kCl > 1) cluster_sync_all();  // every CTA of the cluster runs before any writes to another's shared memory
   griddep_wait();
 #pragma unroll
   for (int u = 0; u < U; ++u) {
     const int c = sl.col(u);
-    a[u] = b[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+    a[u] = b[u] = x[u] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (c >= sl.end) continue;
+    x[u] = load4(p.x + t * pitch + c);
     a[u] = load4(static_cast<const T*>(p.a) + t * pitch + c);
     if (p.b != nullptr) b[u] = load4(static_cast<const T*>(p.b) + t * pitch + c);
   }
-  const float2 ss = row_squares<U, kCl>(a, b, red, sums);
+  const float2 ss = row_squares<U, kCl>(a, b, red2, sums);
   const float ia = p.mult / sqrtf(ss.x / p.norm.width + p.eps), ib = p.mult / sqrtf(ss.y / p.norm.width + p.eps);
 #pragma unroll
   for (int u = 0; u < U; ++u) {
     const int c = sl.col(u);
-    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (c < sl.end) {
-      x = load4(p.x + t * pitch + c);
-      const float4 ga = load4(static_cast<const T*>(p.gain_a) + c);
-      x.x = fmaf(a[u].x * ia, ga.x, x.x); x.y = fmaf(a[u].y * ia, ga.y, x.y);
-      x.z = fmaf(a[u].z * ia, ga.z, x.z); x.w = fmaf(a[u].w * ia, ga.w, x.w);
-      if (p.b != nullptr) {
-        const float4 gb = load4(static_cast<const T*>(p.gain_b) + c);
-        x.x = fmaf(b[u].x * ib, gb.x, x.x); x.y = fmaf(b[u].y * ib, gb.y, x.y);
-        x.z = fmaf(b[u].z * ib, gb.z, x.z); x.w = fmaf(b[u].w * ib, gb.w, x.w);
-      }
-      store4(p.x + t * pitch + c, x);
+    if (c >= sl.end) continue;
+    const float4 ga = load4(static_cast<const T*>(p.gain_a) + c);
+    x[u].x = fmaf(a[u].x * ia, ga.x, x[u].x); x[u].y = fmaf(a[u].y * ia, ga.y, x[u].y);
+    x[u].z = fmaf(a[u].z * ia, ga.z, x[u].z); x[u].w = fmaf(a[u].w * ia, ga.w, x[u].w);
+    if (p.b != nullptr) {
+      const float4 gb = load4(static_cast<const T*>(p.gain_b) + c);
+      x[u].x = fmaf(b[u].x * ib, gb.x, x[u].x); x[u].y = fmaf(b[u].y * ib, gb.y, x[u].y);
+      x[u].z = fmaf(b[u].z * ib, gb.z, x[u].z); x[u].w = fmaf(b[u].w * ib, gb.w, x[u].w);
     }
-    a[u] = x;
+    store4(p.x + t * pitch + c, x[u]);
   }
-  norm_row<T, U, kCl>(p.norm, sl, t, a, gain, bias, red, stats);
+  norm_row<T, U, kCl>(p.norm, sl, t, x, gain, bias, red, stats);
 }
 
 static int check_norm(const NormParams& n) {

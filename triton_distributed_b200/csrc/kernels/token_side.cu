@@ -5,8 +5,9 @@
 
 namespace b200 {
 
+template <typename T>
 __device__ __forceinline__ float gelu_tanh(float z) {
-  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  return 0.5f * z * (1.f + tanh_t<T>(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
 struct TokenSideParams {
@@ -35,7 +36,7 @@ __global__ void __launch_bounds__(256) token_side_kernel(const TokenSideParams p
   const float z[4] = {g.x, g.y, g.z, g.w};
   float o[4];
 #pragma unroll
-  for (int i = 0; i < 4; ++i) o[i] = ok && c + i < p.dim ? gelu_tanh(z[i]) * to_float(e[i]) : 0.f;
+  for (int i = 0; i < 4; ++i) o[i] = ok && c + i < p.dim ? gelu_tanh<T>(z[i]) * to_float(e[i]) : 0.f;
   store4(static_cast<T*>(p.act) + t * p.pitch + c, make_float4(o[0], o[1], o[2], o[3]));
 }
 
