@@ -12,7 +12,8 @@
 // through shared memory in chunks of 16; the next chunk's copies are in flight while a chunk is computed. All arithmetic is
 // fp32 on the CUDA cores (two products per instruction), so the fp32 pipe is what bounds a long call. To save its instructions
 // four tokens share a pass over S: what they owe each other is a 4 x 4 triangle of scalars (see the kernel).
-// Heads of up to 128 x 128 run this way (`recurrent_kernel`); larger ones keep S in global memory (`recurrent_plain_kernel`).
+// Heads of up to 128 x 128 run this way (`recurrent_kernel`; calls of one token `recurrent_step_kernel`); larger ones keep S in
+// global memory (`recurrent_plain_kernel`).
 //
 // In front of them: token_mix (h + (previous h - h) * mu for several mu at once) and short_conv (causal convolution over a few
 // tokens per channel, silu), both of which carry the last inputs of a sequence from call to call.
@@ -596,6 +597,133 @@ __device__ __forceinline__ float cta_sum(float v, float* red) {
   return warp_sum((threadIdx.x & 31) < (blockDim.x >> 5) ? red[threadIdx.x & 31] : 0.f);
 }
 
+// One token per sequence: bound by reading and writing S once. The layout of recurrent_kernel, one token at a time; q and k keep
+// their length, which enters as a factor.
+template <typename T, int kKind, int kP>
+__global__ void __launch_bounds__(2 * kP) recurrent_step_kernel(const RecurrentParams p) {
+  constexpr int R = kP / 8, kWarps = kP / 16, kThreads = 2 * kP;
+  __shared__ __align__(16) float sq[kP], sk[kP], sw[kP], sv[kP], so[kP];
+  __shared__ float red[3][kWarps];
+  const int h = blockIdx.x, b = blockIdx.y, kh = h / p.per;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kg = lane & 7;
+  const int col0 = (warp * 4 + (lane >> 3)) * 4, ch = threadIdx.x;
+  float* state = p.state + (static_cast<size_t>(b) * p.H + h) * p.Dp * p.Ep;
+  griddep_launch_dependents();
+  // the state comes from an earlier call: it may be fetched into L2, but not read, before that call is known to be over
+  for (int i = threadIdx.x * 32; i < p.Dp * p.Ep; i += kThreads * 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(state + i));
+  const float base = kKind == kWkv && ch < p.Dp ? p.decay_base[h * p.Dp + ch] : 0.f, bonus = kKind == kWkv && ch < p.Dp ? p.bonus[h * p.Dp + ch] : 0.f;
+  const float gain = ch < p.Ep ? p.gain[h * p.gain_stride + ch] : 0.f;
+  griddep_wait();
+  float q = 0.f, k = 0.f, z = 0.f, v = 0.f, gate = 0.f, g = 1.f, beta = 1.f;
+  const size_t row = b;
+  if (ch < p.Dp) {
+    q = to_float(static_cast<const T*>(p.q)[row * p.ldq + kh * p.Dp + ch]);
+    k = to_float(static_cast<const T*>(p.k)[row * p.ldk + kh * p.Dp + ch]);
+    if (kKind == kWkv) z = to_float(static_cast<const T*>(p.decay)[row * p.ld_decay + h * p.Dp + ch]);
+  }
+  if (ch < p.Ep) {
+    v = to_float(static_cast<const T*>(p.v)[row * p.ldv + h * p.Ep + ch]);
+    gate = to_float(static_cast<const T*>(p.gate)[row * p.ldg + h * p.Ep + ch]);
+  }
+  if (kKind == kDelta) {
+    g = to_float(static_cast<const T*>(p.decay)[row * p.ld_decay + h]);
+    beta = to_float(static_cast<const T*>(p.beta)[row * p.ld_decay + h]);
+  }
+  float4 s[R];   // s[4 i + e] = row 32 i + 4 kg + e, columns col0 ...
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int r = 32 * (i >> 2) + 4 * kg + (i & 3);
+    s[i] = r < p.Dp && col0 < p.Ep ? *reinterpret_cast<const float4*>(state + static_cast<size_t>(r) * p.Ep + col0) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  if (ch < kP) {
+    sq[ch] = q;
+    sk[ch] = k;
+    sv[ch] = v;
+    if (kKind == kWkv) sw[ch] = wkv_decay<T>(z, base);
+  }
+  // sums over the key channels
+  const float x = warp_sum(kKind == kWkv ? q * bonus * k : q * k);
+  const float y = kKind == kDelta ? warp_sum(q * q) : 0.f, w = kKind == kDelta ? warp_sum(k * k) : 0.f;
+  if (lane == 0) {
+    red[0][warp] = x;
+    red[1][warp] = y;
+    red[2][warp] = w;
+  }
+  __syncthreads();
+  float qk = 0.f, qq = 0.f, kk = 0.f;
+#pragma unroll
+  for (int i = 0; i < kP / 32; ++i) {
+    qk += red[0][i];
+    if (kKind == kDelta) {
+      qq += red[1][i];
+      kk += red[2][i];
+    }
+  }
+  float iq = 1.f, ik = 1.f;
+  if (kKind == kDelta) {
+    iq = 1.f / (sqrtf(qq + 1e-6f) * sqrtf(static_cast<float>(p.D)));
+    ik = 1.f / sqrtf(kk + 1e-6f);
+    g = delta_decay(g, p.decay_base[h], p.decay_bias[h]);
+    beta = 1.f / (1.f + expf(-beta));
+  }
+  const float4 v4 = *reinterpret_cast<const float4*>(sv + col0);
+  float o[4] = {0.f, 0.f, 0.f, 0.f}, d[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < R / 4; ++i) {
+    float qr[4], kr[4];
+    load_few<float, 4>(sq + 32 * i + 4 * kg, qr);
+    if (kKind == kDelta) load_few<float, 4>(sk + 32 * i + 4 * kg, kr);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float4 t = s[4 * i + e];
+      o[0] = fmaf(qr[e], t.x, o[0]); o[1] = fmaf(qr[e], t.y, o[1]); o[2] = fmaf(qr[e], t.z, o[2]); o[3] = fmaf(qr[e], t.w, o[3]);
+      if (kKind == kDelta) {
+        d[0] = fmaf(kr[e], t.x, d[0]); d[1] = fmaf(kr[e], t.y, d[1]); d[2] = fmaf(kr[e], t.z, d[2]); d[3] = fmaf(kr[e], t.w, d[3]);
+      }
+    }
+  }
+#pragma unroll
+  for (int m = 1; m < 8; m <<= 1)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      o[c] += __shfl_xor_sync(0xffffffffu, o[c], m);
+      if (kKind == kDelta) d[c] += __shfl_xor_sync(0xffffffffu, d[c], m);
+    }
+  const float vv[4] = {v4.x, v4.y, v4.z, v4.w};
+#pragma unroll
+  for (int c = 0; c < 4; ++c) {
+    d[c] = kKind == kDelta ? beta * fmaf(-g * ik, d[c], vv[c]) : vv[c];
+    o[c] = iq * fmaf(ik * qk, d[c], g * o[c]);
+    d[c] *= ik;
+  }
+  if (kg == 0) *reinterpret_cast<float4*>(so + col0) = make_float4(o[0], o[1], o[2], o[3]);
+#pragma unroll
+  for (int i = 0; i < R / 4; ++i) {
+    float kr[4], wr[4];
+    load_few<float, 4>(sk + 32 * i + 4 * kg, kr);
+    if (kKind == kWkv) load_few<float, 4>(sw + 32 * i + 4 * kg, wr);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int r = 32 * i + 4 * kg + e;
+      const float f = kKind == kWkv ? wr[e] : g;
+      const float4 t = s[4 * i + e];
+      if (r < p.Dp && col0 < p.Ep)
+        *reinterpret_cast<float4*>(state + static_cast<size_t>(r) * p.Ep + col0) =
+            make_float4(fmaf(kr[e], d[0], f * t.x), fmaf(kr[e], d[1], f * t.y), fmaf(kr[e], d[2], f * t.z), fmaf(kr[e], d[3], f * t.w));
+    }
+  }
+  __syncthreads();
+  // ---- norm over the head, gain, gate
+  const float mine = ch < kP ? so[ch] : 0.f, part = warp_sum(mine * mine);
+  if (lane == 0) red[0][warp] = part;
+  __syncthreads();
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < kP / 32; ++i) ss += red[0][i];
+  if (ch < p.Ep)
+    static_cast<T*>(p.out)[row * p.H * p.Ep + h * p.Ep + ch] = from_float<T>(mine * inv_sqrt<T>(ss / p.E + p.eps) * gain * silu<T>(gate));
+}
+
 // Heads of any size: the state stays in global memory, a thread walks the rows of its columns.
 template <typename T, int kKind>
 __global__ void __launch_bounds__(256) recurrent_plain_kernel(const RecurrentParams p) {
@@ -659,6 +787,10 @@ __global__ void __launch_bounds__(256) recurrent_plain_kernel(const RecurrentPar
 
 template <typename T, int kKind, int kP>
 static int launch_recurrent(const RecurrentParams& p, int B, cudaStream_t s) {
+  if (p.S == 1) {
+    B200_CHECK_CUDA(launch_pdl(recurrent_step_kernel<T, kKind, kP>, dim3(p.H, B), dim3(2 * kP), 0, s, p));
+    return kOk;
+  }
   static bool configured[64] = {false};
   int dev = 0;
   B200_CHECK_CUDA(cudaGetDevice(&dev));
